@@ -74,12 +74,32 @@ class RunEntry:
     ``writes_cache`` False when the entry only reads a cache another entry filled.
     ``add_embedding`` the embedding's output (the stream as it was before the first entry)
                     is added to the stream before this entry runs.
+    ``join_embedding`` the stream and the embedding's output pass the configuration's
+                    ``stream_join_spec()`` before this entry runs.
     """
 
     layer: int
     cache_layer: int
     writes_cache: bool = True
     add_embedding: bool = False
+    join_embedding: bool = False
+
+
+def looped_run_order(n_layers: int, loop: Optional[Dict[str, int]], first_of_pass) -> List[RunEntry]:
+    """Layers 0 .. n_layers - 1 in order, with layers ``start`` .. ``stop`` - 1 of ``loop`` run
+    ``times`` times in a row (the same weights; every pass has caches of its own: the first pass
+    the layers', further ones numbered after the last layer).  ``first_of_pass(pass number)``
+    gives the further fields of a pass's first entry."""
+    if loop is None:
+        return [RunEntry(i, i) for i in range(n_layers)]
+    a, b = loop["start"], loop["stop"]
+    order = [RunEntry(i, i) for i in range(a)]
+    for rep in range(loop["times"]):
+        for i in range(a, b):
+            cache = i if rep == 0 else n_layers + (rep - 1) * (b - a) + (i - a)
+            order.append(RunEntry(i, cache, True, **(first_of_pass(rep) if i == a else {})))
+    return order + [RunEntry(i, i) for i in range(b, n_layers)]
+
 
 
 class ModelConfig:
@@ -108,6 +128,10 @@ class ModelConfig:
 
     def position_spec(self) -> PartSpec:
         return PartSpec("none")
+
+    def stream_join_spec(self) -> Optional[PartSpec]:
+        """How entries with ``join_embedding`` join the stream with the embedding's output."""
+        return None
 
     def final_norm_spec(self) -> PartSpec:
         raise NotImplementedError
@@ -158,10 +182,25 @@ def _require_bool(raw: Dict[str, Any], key: str, default: bool) -> bool:
     return value
 
 
+def config_int(d, key: str, where: str, minimum: int = 1) -> int:
+    """``d[key]``, an integer that is at least ``minimum``; ``where`` names ``d`` in the error."""
+    v = d.get(key) if isinstance(d, dict) else None
+    if isinstance(v, bool) or not isinstance(v, int) or v < minimum:
+        raise ConfigError(f"config.json: {where}.{key} must be an integer >= {minimum}, got {v!r}")
+    return v
+
+
+def config_number(d, key: str, where: str) -> float:
+    v = d.get(key) if isinstance(d, dict) else None
+    if isinstance(v, bool) or not isinstance(v, (int, float)):
+        raise ConfigError(f"config.json: {where}.{key} must be a number, got {v!r}")
+    return float(v)
+
+
 def replace(config, **changes):
     """``dataclasses.replace`` that re-validates."""
     return type(config).from_dict({**config.to_dict(), **changes})
 
 
-__all__ = ["ConfigError", "PartSpec", "LayerSpec", "RunEntry", "ModelConfig",
-           "replace", "dataclasses"]
+__all__ = ["ConfigError", "PartSpec", "LayerSpec", "RunEntry", "ModelConfig", "looped_run_order",
+           "config_int", "config_number", "replace", "dataclasses"]

@@ -26,25 +26,12 @@ import copy
 from dataclasses import dataclass, field
 from typing import Any, Dict, List
 
-from .base import ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry
+from .base import (ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry,
+                   config_int as _int, config_number as _num)
 
 _TYPES = ("parallel", "attention")
 #: the distance bias of ``attention`` layers: slope_h = 2^(-SLOPE_BITS * (h + 1) / heads)
 SLOPE_BITS = 8.0
-
-
-def _int(d, key: str, where: str, minimum: int = 1) -> int:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, int) or v < minimum:
-        raise ConfigError(f"config.json: {where}.{key} must be an integer >= {minimum}, got {v!r}")
-    return v
-
-
-def _num(d, key: str, where: str) -> float:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, (int, float)):
-        raise ConfigError(f"config.json: {where}.{key} must be a number, got {v!r}")
-    return float(v)
 
 
 def _check_attention(mx, where: str, rotary: bool) -> None:

@@ -24,23 +24,10 @@ import copy
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
-from .base import ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry
+from .base import (ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry,
+                   config_int as _int, config_number as _num, looped_run_order)
 
 _MIXERS = ("attention", "retention")
-
-
-def _int(d: Dict[str, Any], key: str, where: str, minimum: int = 1) -> int:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, int) or v < minimum:
-        raise ConfigError(f"config.json: {where}.{key} must be an integer >= {minimum}, got {v!r}")
-    return v
-
-
-def _num(d: Dict[str, Any], key: str, where: str) -> float:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, (int, float)):
-        raise ConfigError(f"config.json: {where}.{key} must be a number, got {v!r}")
-    return float(v)
 
 
 @dataclass(frozen=True)
@@ -177,16 +164,8 @@ class PezaraxConfig(ModelConfig):
         """Layers in order; the looped span ``times`` times in a row.  The first pass uses the
         layers' own caches, every further pass caches numbered after the last layer, and its
         first entry has the embedding's output added before it."""
-        n = len(self.layers)
-        if self.loop is None:
-            return [RunEntry(i, i) for i in range(n)]
-        a, b, times = self.loop["start"], self.loop["stop"], self.loop["times"]
-        order = [RunEntry(i, i) for i in range(a)]
-        for rep in range(times):
-            for i in range(a, b):
-                cache = i if rep == 0 else n + (rep - 1) * (b - a) + (i - a)
-                order.append(RunEntry(i, cache, True, add_embedding=rep > 0 and i == a))
-        return order + [RunEntry(i, i) for i in range(b, n)]
+        return looped_run_order(len(self.layers), self.loop,
+                                lambda rep: {"add_embedding": rep > 0})
 
     def embedding_spec(self) -> PartSpec:
         return PartSpec("scaled_token_embedding", {"weights": "embed", "vocab": self.vocab,

@@ -20,24 +20,11 @@ import copy
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
-from .base import ConfigError, LayerSpec, ModelConfig, PartSpec
+from .base import (ConfigError, LayerSpec, ModelConfig, PartSpec,
+                   config_int as _int, config_number as _num)
 
 _MIXERS = ("latent_attention",)
 _MLP_KINDS = ("dense", "moe")
-
-
-def _int(d: Dict[str, Any], key: str, where: str, minimum: int = 1) -> int:
-    v = d.get(key)
-    if isinstance(v, bool) or not isinstance(v, int) or v < minimum:
-        raise ConfigError(f"config.json: {where}.{key} must be an integer >= {minimum}, got {v!r}")
-    return v
-
-
-def _num(d: Dict[str, Any], key: str, where: str) -> float:
-    v = d.get(key)
-    if isinstance(v, bool) or not isinstance(v, (int, float)):
-        raise ConfigError(f"config.json: {where}.{key} must be a number, got {v!r}")
-    return float(v)
 
 
 @dataclass(frozen=True)

@@ -34,7 +34,8 @@ import copy
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional
 
-from .base import ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry
+from .base import (ConfigError, LayerSpec, ModelConfig, PartSpec, RunEntry,
+                   config_int as _int, config_number as _num)
 
 _TYPES = ("parallel", "latent_attention", "parallel_2")
 #: constants the design fixes
@@ -42,20 +43,6 @@ LRU_DECAY_CONSTANT = 8.0           # log a = -8 * r * softplus(lambda)
 MLP_ACT_SLOPE = 1.702              # g * sigmoid(1.702 g)
 MLP_UP_SHIFT = 1.0                 # ... * (u + 1)
 NORM_OFFSET = 1.0                  # norms multiply by 1 + w
-
-
-def _int(d, key: str, where: str, minimum: int = 1) -> int:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, int) or v < minimum:
-        raise ConfigError(f"config.json: {where}.{key} must be an integer >= {minimum}, got {v!r}")
-    return v
-
-
-def _num(d, key: str, where: str) -> float:
-    v = d.get(key) if isinstance(d, dict) else None
-    if isinstance(v, bool) or not isinstance(v, (int, float)):
-        raise ConfigError(f"config.json: {where}.{key} must be a number, got {v!r}")
-    return float(v)
 
 
 def _check_rot(rot, most: int, where: str, yarn: bool) -> None:

@@ -6,7 +6,11 @@
 //     of the branch alone with the stream added after it (alpha * x + norm(y)),
 //     optionally with a copy of the result in the activation type for the next product;
 //   * the gated pair of a feed-forward: f(g) * (u + shift) with optional clamps and an
-//     optional per-(token, group) scale (a router's weights);
+//     optional per-(token, group) scale (a router's weights); f is a sigmoid-weighted unit or the
+//     tanh form of gelu;
+//   * a layer or root-mean-square norm of a branch joined to the stream, followed in the same
+//     kernel by the next branch's norm of the sum (layers with a norm before and after a branch);
+//   * a cap on logits, cap * tanh(z / cap);
 //   * a router: logits in 32-bit, the largest `top`, softmax over those.
 // All arithmetic is 32-bit; reduction trees depend on the row's width only.
 #include "common.cuh"
@@ -131,13 +135,19 @@ __global__ void rms_norm_kernel(RmsArgs a) {
 }
 
 // --------------------------------------------------------------------- gated pair
-// out[t, out_col + i] = g' * sigmoid(act_alpha * g') * (u' + up_shift) * scale[t, i / group]
-// with g' = min(g, limit) and u' = clamp(u, -limit, limit) when limit > 0.
+// out[t, out_col + i] = f(g') * (u' + up_shift) * scale[t, i / group]
+// with f(g) = g * sigmoid(act_alpha * g) (act 0) or the tanh form of gelu (act 1), and
+// g' = min(g, limit), u' = clamp(u, -limit, limit) when limit > 0.
+__device__ __forceinline__ float gated_unit(float g, float act_alpha, int act) {
+    return act == 1 ? prb_activate(g, PRB_ACT_GELU_TANH) : g * sigmoidf_(act_alpha * g);
+}
+
 template <typename O>
 __global__ void gated_pair_kernel(O* __restrict__ out, long out_ld, int out_col,
                                   const float* __restrict__ in, long in_ld, int gate_col, int up_col,
                                   int n, int n_rows, float limit, float act_alpha, float up_shift,
-                                  const float* __restrict__ scale, long scale_ld, int group) {
+                                  const float* __restrict__ scale, long scale_ld, int group,
+                                  int act) {
     prb_grid_launch_dependents();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= (size_t)n_rows * n) return;
@@ -148,7 +158,7 @@ __global__ void gated_pair_kernel(O* __restrict__ out, long out_ld, int out_col,
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
     }
-    float v = g * sigmoidf_(act_alpha * g) * (u + up_shift);
+    float v = gated_unit(g, act_alpha, act) * (u + up_shift);
     if (scale) v *= scale[(size_t)t * scale_ld + i / group];
     out[(size_t)t * out_ld + out_col + i] = prb_from_float<O>(v);
 }
@@ -159,7 +169,8 @@ template <typename O>
 __global__ void gated_pair4_kernel(O* __restrict__ out, long out_ld, int out_col,
                                    const float* __restrict__ in, long in_ld, int gate_col, int up_col,
                                    int n, int n_rows, float limit, float act_alpha, float up_shift,
-                                   const float* __restrict__ scale, long scale_ld, int group) {
+                                   const float* __restrict__ scale, long scale_ld, int group,
+                                   int act) {
     prb_grid_launch_dependents();
     const int n4 = n / 4;
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -175,7 +186,7 @@ __global__ void gated_pair4_kernel(O* __restrict__ out, long out_ld, int out_col
             g[k] = fminf(g[k], limit);
             u[k] = fminf(fmaxf(u[k], -limit), limit);
         }
-        v[k] = g[k] * sigmoidf_(act_alpha * g[k]) * (u[k] + up_shift) * sc;
+        v[k] = gated_unit(g[k], act_alpha, act) * (u[k] + up_shift) * sc;
     }
     O* o = out + (size_t)t * out_ld + out_col + i;
     if constexpr (sizeof(O) == 4) {
@@ -186,6 +197,93 @@ __global__ void gated_pair4_kernel(O* __restrict__ out, long out_ld, int out_col
         pk.x = *reinterpret_cast<const uint32_t*>(&lo);
         pk.y = *reinterpret_cast<const uint32_t*>(&hi);
         *reinterpret_cast<uint2*>(o) = pk;
+    }
+}
+
+// ------------------------------------------ a norm after a branch, and the next one before
+// One row (a CTA):  x <- x + mult * norm_1(y);  then what the next product reads of the new x:
+// norm_2(x) (next 1), or x itself (next 2), in the activation type, rows `out_ld` apart; or
+// nothing (next 0).  A norm is (v - mean) / sqrt(variance + eps) * w + b (centred; b may be
+// null) or v / sqrt(mean(v^2) + eps) * w.  The variance is the mean of the squared deviations
+// (two passes over values that stay in registers, NV a thread).
+struct NormPairArgs {
+    void* out;              // or null (next 0)
+    long out_ld;
+    float* x;               // [n_rows, width], in place
+    const float* y;         // [n_rows, width]
+    const float* w1;
+    const float* b1;        // or null
+    const float* w2;
+    const float* b2;
+    int n_rows, width, centred1, centred2, next;
+    float mult, eps1, eps2;
+};
+
+template <int NV>
+__device__ __forceinline__ float row_inverse_deviation(float (&v)[NV], int width, bool centred, float eps,
+                                                       float* scratch) {
+    if (centred) {
+        float s = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) s += v[j];      // (places beyond the row hold zero)
+        const float mean = prb_block_sum(s, scratch) / (float)width;
+#pragma unroll
+        for (int j = 0; j < NV; ++j)
+            v[j] = (int)threadIdx.x + j * (int)blockDim.x < width ? v[j] - mean : 0.0f;
+    }
+    float q = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) q = fmaf(v[j], v[j], q);
+    return 1.0f / sqrtf(prb_block_sum(q, scratch) / (float)width + eps);
+}
+
+template <typename O, int NV>
+__global__ void norm_pair_kernel(NormPairArgs a) {
+    __shared__ float scratch[32];
+    prb_grid_launch_dependents();
+    const int r = blockIdx.x;
+    if (r >= a.n_rows) return;
+    float* x = a.x + (size_t)r * a.width;
+    const float* y = a.y + (size_t)r * a.width;
+    float v[NV], xv[NV], w[NV], b[NV], w2[NV], b2[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {                   // everything is asked for at once
+        const int i = threadIdx.x + j * blockDim.x;
+        const bool in = i < a.width;
+        v[j] = in ? y[i] : 0.0f;
+        xv[j] = in ? x[i] : 0.0f;
+        w[j] = in ? a.w1[i] : 0.0f;
+        b[j] = in && a.b1 ? a.b1[i] : 0.0f;
+        w2[j] = in && a.next == 1 ? a.w2[i] : 0.0f;
+        b2[j] = in && a.next == 1 && a.b2 ? a.b2[i] : 0.0f;
+    }
+    const float inv = row_inverse_deviation<NV>(v, a.width, a.centred1 != 0, a.eps1, scratch);
+    O* out = reinterpret_cast<O*>(a.out) + (size_t)r * a.out_ld;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        xv[j] = fmaf(a.mult, fmaf(v[j] * inv, w[j], b[j]), xv[j]);
+        if (i >= a.width) continue;
+        x[i] = xv[j];
+        if (a.next == 2) out[i] = prb_from_float<O>(xv[j]);
+    }
+    if (a.next != 1) return;
+    const float inv2 = row_inverse_deviation<NV>(xv, a.width, a.centred2 != 0, a.eps2, scratch);
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = threadIdx.x + j * blockDim.x;
+        if (i < a.width) out[i] = prb_from_float<O>(fmaf(xv[j] * inv2, w2[j], b2[j]));
+    }
+}
+
+// ------------------------------------------------------------------- a cap on logits
+__global__ void tanh_cap_kernel(float* __restrict__ z, long ld, int n, long total, float cap) {
+    prb_grid_launch_dependents();
+    for (long e = (long)blockIdx.x * blockDim.x + threadIdx.x; e < total;
+         e += (long)gridDim.x * blockDim.x) {
+        const long r = e / n;
+        float* p = z + r * ld + (e - r * n);
+        *p = cap * tanhf(*p / cap);
     }
 }
 
@@ -315,11 +413,48 @@ PRB_API int prb_rms_norm(void* out, float* x_out, const float* x, const float* y
     return 0;
 }
 
+// x <- x + mult * norm_1(y), then norm_2(x) or a copy of x in the activation type.
+PRB_API int prb_norm_pair(void* out, long out_ld, float* x, const float* y, const float* w1,
+                          const float* b1, const float* w2, const float* b2, int n_rows, int width,
+                          int centred1, int centred2, int next, float mult, float eps1, float eps2,
+                          int out_dtype, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0 || width > 1024 * 16) return PRB_E_SIZE;
+    if (next < 0 || next > 2 || w1 == nullptr || (next != 0 && out == nullptr) || (next == 1 && w2 == nullptr))
+        return PRB_E_ARG;
+    NormPairArgs a{out, out_ld, x, y, w1, b1, w2, b2, n_rows, width, centred1, centred2, next, mult,
+                   eps1, eps2};
+    // values a thread holds: 4 while 1,024 threads allow it
+    const int per = width <= 4096 ? 4 : 16;
+    int threads = ((width + per - 1) / per + 31) / 32 * 32;
+    if (threads < 64) threads = 64;
+#define NORM_PAIR(OT)                                                                                do {                                                                                                 if (per == 4) norm_pair_kernel<OT, 4><<<n_rows, threads, 0, stream>>>(a);                        else norm_pair_kernel<OT, 16><<<n_rows, threads, 0, stream>>>(a);                            } while (0)
+    if (out_dtype == PRB_F32) NORM_PAIR(float);
+    else if (out_dtype == PRB_BF16) NORM_PAIR(__nv_bfloat16);
+    else return PRB_E_DTYPE;
+#undef NORM_PAIR
+    PRB_LAUNCH_CHECK();
+    return 0;
+}
+
+// z[r, :n] = cap * tanh(z[r, :n] / cap) in place, rows `ld` apart.
+PRB_API int prb_tanh_cap(float* z, long ld, int n_rows, int n, float cap, cudaStream_t stream) {
+    if (n_rows <= 0 || n <= 0) return 0;
+    if (!(cap > 0.0f) || ld < n) return PRB_E_ARG;
+    const long total = (long)n_rows * n;
+    long blocks = (total + 255) / 256;
+    if (blocks > (long)prb_sm_count() * 16) blocks = (long)prb_sm_count() * 16;
+    tanh_cap_kernel<<<(unsigned)blocks, 256, 0, stream>>>(z, ld, n, total, cap);
+    PRB_LAUNCH_CHECK();
+    return 0;
+}
+
 PRB_API int prb_gated_pair(void* out, long out_ld, int out_col, const float* in, long in_ld,
                            int gate_col, int up_col, int n, int n_rows, float limit,
                            float act_alpha, float up_shift, const float* scale, long scale_ld,
-                           int group, int out_dtype, cudaStream_t stream) {
+                           int group, int act, int out_dtype, cudaStream_t stream) {
     if (n <= 0 || n_rows <= 0) return 0;
+    if (act < 0 || act > 1) return PRB_E_ARG;
     if (scale != nullptr && group <= 0) return PRB_E_ARG;
     const size_t total = (size_t)n * n_rows;
     const size_t esz = out_dtype == PRB_F32 ? 4 : 2;
@@ -330,11 +465,11 @@ PRB_API int prb_gated_pair(void* out, long out_ld, int out_col, const float* in,
         if (out_dtype == PRB_F32)
             gated_pair4_kernel<float><<<blocks4, 256, 0, stream>>>(
                 (float*)out, out_ld, out_col, in, in_ld, gate_col, up_col, n, n_rows, limit,
-                act_alpha, up_shift, scale, scale_ld, group);
+                act_alpha, up_shift, scale, scale_ld, group, act);
         else
             gated_pair4_kernel<__nv_bfloat16><<<blocks4, 256, 0, stream>>>(
                 (__nv_bfloat16*)out, out_ld, out_col, in, in_ld, gate_col, up_col, n, n_rows, limit,
-                act_alpha, up_shift, scale, scale_ld, group);
+                act_alpha, up_shift, scale, scale_ld, group, act);
         PRB_LAUNCH_CHECK();
         return 0;
     }
@@ -342,11 +477,11 @@ PRB_API int prb_gated_pair(void* out, long out_ld, int out_col, const float* in,
     if (out_dtype == PRB_F32)
         gated_pair_kernel<float><<<blocks, 256, 0, stream>>>(
             (float*)out, out_ld, out_col, in, in_ld, gate_col, up_col, n, n_rows, limit, act_alpha,
-            up_shift, scale, scale_ld, group);
+            up_shift, scale, scale_ld, group, act);
     else if (out_dtype == PRB_BF16)
         gated_pair_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(
             (__nv_bfloat16*)out, out_ld, out_col, in, in_ld, gate_col, up_col, n, n_rows, limit,
-            act_alpha, up_shift, scale, scale_ld, group);
+            act_alpha, up_shift, scale, scale_ld, group, act);
     else
         return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();

@@ -136,7 +136,16 @@ def _declare(h: ctypes.CDLL) -> None:
     h.prb_rms_norm.argtypes = [P, P, P, P, P, L, P, P, P, P, I, I, I, F, F, I, I, P, P]
     h.prb_gate_mul.argtypes = [P, L, P, L, P, L, I, I, I, P]
     h.prb_gate_mul.restype = c_int
-    h.prb_gated_pair.argtypes = [P, L, I, P, L, I, I, I, I, F, F, F, P, L, I, I, P]
+    h.prb_gated_pair.argtypes = [P, L, I, P, L, I, I, I, I, F, F, F, P, L, I, I, I, P]
+    h.prb_norm_pair.argtypes = [P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, F, I, P]
+    h.prb_norm_pair.restype = c_int
+    h.prb_tanh_cap.argtypes = [P, L, I, I, F, P]
+    h.prb_tanh_cap.restype = c_int
+    h.prb_rotary_angles.argtypes = [P, P, P, P, I, I, P]
+    h.prb_rotary_angles.restype = c_int
+    h.prb_wattn_prepare_heads.argtypes = [P, P, P, L, I, I, I] + [P] * 7 + \
+        [I, P, I, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, I, I, I, I, P, P]
+    h.prb_wattn_prepare_heads.restype = c_int
     h.prb_route.argtypes = [P, P, P, P, L, P, P, I, I, I, I, I, P]
     h.prb_latent_prepare.argtypes = [P, L, P, P, L, I, I, P, P, P, P, P, I, I, I, I, I, I, I, F,
                                      I, I, F, P, P, P]
@@ -148,12 +157,12 @@ def _declare(h: ctypes.CDLL) -> None:
     h.prb_latent_mma_rows.argtypes = []
     h.prb_latent_attention.argtypes = [P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P]
     h.prb_latent_unfold.argtypes = [P, L, P, P, P, L, I, I, I, I, I, I, I, P]
-    h.prb_embed_scaled.argtypes = [P, P, P, P, I, I, I, F, I, P, P]
+    h.prb_embed_scaled.argtypes = [P, P, P, P, I, I, I, F, I, P, L, P, P]
     h.prb_route_scores.argtypes = [P, P, P, P, L, P, I, I, I, I, I, I, F, I, I, P]
     h.prb_routed_act.argtypes = [P, L, P, L, I, I, I, P, L, I, I, I, I, P]
     h.prb_retention_lanes.argtypes = [I]
     h.prb_retention_scan.argtypes = [P, P, L, I, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I,
-                                     P, P, I, P, P]
+                                     P, P, I, P, P, P]
     h.prb_retention_segment.argtypes = []
     h.prb_retention_segment.restype = c_int
     h.prb_retention_max_segments.argtypes = [I, I]
@@ -177,7 +186,7 @@ def _declare(h: ctypes.CDLL) -> None:
     h.prb_retention_step_supports.argtypes = [I, I]
     h.prb_retention_step_supports.restype = c_int
     h.prb_retention_step.argtypes = [P, L, P, L, I, I, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I,
-                                     F, F, I, P, P]
+                                     F, F, I, P, P, P]
     h.prb_retention_step.restype = c_int
     h.prb_tmix_lanes.argtypes = [I]
     h.prb_tmix_shift.argtypes = [P, L, P, L, P, P, P, P, P, P, I, I, I, I, I, P, P]
@@ -190,14 +199,14 @@ def _declare(h: ctypes.CDLL) -> None:
                                          I, I, I, I, I, I, I, I, I, P, P, P, I, P, P]
     h.prb_tmix_finish.argtypes = [P, L, P, L, P, L, I, P, P, I, I, I, F, F, I, P]
     h.prb_wattn_prepare.argtypes = [P, P, P, L, I, I, I, P, P, P, P, P, I, I, I, I, I, I, F, F, I,
-                                    I, I, I, I, P, P, P, P, P, P]
+                                    I, I, I, P, P, P]
     h.prb_wattn.argtypes = [P, L, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, I, I, F, F, I, I,
-                            P, I, P, P]
+                            P, I, F, P, P]
     h.prb_wattn_tile_rows.argtypes = [I, I, I, I]
     h.prb_wattn_single_supports.argtypes = [I, I, I, I]
     h.prb_wattn_single.argtypes = list(h.prb_wattn.argtypes)
     h.prb_wattn_tile.argtypes = [P, L, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, I, I, I, F,
-                                 F, I, I, P, I, P, P]
+                                 F, I, I, P, I, F, P, P]
     h.prb_lru_max_taps.argtypes = []
     h.prb_lru_conv.argtypes = [P, P, L, I, P, P, P, P, P, P, P, P, I, I, I, I, I, P]
     h.prb_lru_gates.argtypes = [P, P, P, P, P, P, P, I, I, I, I, P]
@@ -987,11 +996,16 @@ def gate_mul(out, inp, gate) -> None:
                               gate.stride(0), n_rows, n, dtype_code(out.dtype), _stream()), what)
 
 
+GATED_ACT_CODES = {"sigmoid": 0, "gelu_tanh": 1}
+
+
 def gated_pair(out, inp, gate_col: int, up_col: int, n: int, out_col: int = 0, limit: float = 0.0,
-               act_alpha: float = 1.0, up_shift: float = 0.0, scale=None, group: int = 1) -> None:
+               act_alpha: float = 1.0, up_shift: float = 0.0, scale=None, group: int = 1,
+               act: str = "sigmoid") -> None:
     """out[t, out_col + i] = g * sigmoid(act_alpha * g) * (u + up_shift) (* scale[t, i // group])
     for i < n, with g = inp[t, gate_col + i] and u = inp[t, up_col + i] (float32), g capped at
-    ``limit`` and u clamped to +-``limit`` when ``limit`` > 0."""
+    ``limit`` and u clamped to +-``limit`` when ``limit`` > 0.  ``act`` "gelu_tanh": the tanh form
+    of gelu(g) in the place of g * sigmoid(act_alpha * g)."""
     what = "gated_pair"
     if not inp.is_cuda or inp.dtype != torch.float32 or inp.stride(1) != 1:
         raise KernelArgumentError(f"{what}: inp must be float32 on CUDA with unit inner stride")
@@ -1006,7 +1020,76 @@ def gated_pair(out, inp, gate_col: int, up_col: int, n: int, out_col: int = 0, l
                                 int(gate_col), int(up_col), int(n), inp.shape[0], float(limit),
                                 float(act_alpha), float(up_shift), _p(scale),
                                 0 if scale is None else scale.stride(0), int(group),
-                                dtype_code(out.dtype), _stream()), what)
+                                GATED_ACT_CODES[act], dtype_code(out.dtype), _stream()), what)
+
+
+def norm_pair(x, y, mult: float, weight, bias, eps: float, centred: bool, out=None, next_norm=None) -> None:
+    """x <- x + mult * norm(y) in place (x, y float32 [T, width]; ``centred``: a layer norm with
+    ``weight`` and ``bias``, else a root-mean-square norm with ``weight``), and in the same kernel,
+    with ``out`` (float32 or bfloat16, rows may be further apart than width): ``next_norm`` =
+    (weight, bias or None, eps, centred) of the new x, or, without ``next_norm``, x itself."""
+    what = "norm_pair"
+    _need(x, torch.float32, "x", what)
+    _need(y, torch.float32, "y", what)
+    n, width = x.shape
+    if tuple(y.shape) != (n, width):
+        raise KernelArgumentError(f"{what}: x and y differ in shape")
+    w2 = b2 = None
+    eps2, centred2, mode = 0.0, False, 0
+    if next_norm is not None:
+        if out is None:
+            raise KernelArgumentError(f"{what}: a following norm needs somewhere to go")
+        w2, b2, eps2, centred2 = next_norm
+        mode = 1
+    elif out is not None:
+        mode = 2
+    for name, t in (("weight", weight), ("bias", bias), ("next weight", w2), ("next bias", b2)):
+        if t is not None:
+            _need(t, torch.float32, name, what)
+            if t.numel() != width:
+                raise KernelArgumentError(f"{what}: {name} must hold {width} numbers")
+    if out is not None and (not out.is_cuda or out.stride(1) != 1 or out.shape[0] < n or
+                            out.shape[1] < width):
+        raise KernelArgumentError(f"{what}: out has the wrong shape")
+    _check(lib().prb_norm_pair(_p(out), 0 if out is None else out.stride(0), _p(x), _p(y), _p(weight),
+                               _p(bias), _p(w2), _p(b2), n, width, int(bool(centred)),
+                               int(bool(centred2)), mode, float(mult), float(eps), float(eps2),
+                               dtype_code(x.dtype if out is None else out.dtype), _stream()), what)
+
+
+def tanh_cap(z, cap: float) -> None:
+    """z <- cap * tanh(z / cap) in place; z float32 [rows, n], rows may be further apart."""
+    what = "tanh_cap"
+    if not z.is_cuda or z.dtype != torch.float32 or z.dim() != 2 or z.stride(1) != 1:
+        raise KernelArgumentError(f"{what}: z must be float32 rows on CUDA with unit inner stride")
+    if not cap > 0.0:
+        raise KernelArgumentError(f"{what}: the cap must be positive")
+    _check(lib().prb_tanh_cap(_p(z), z.stride(0), z.shape[0], z.shape[1], float(cap), _stream()), what)
+
+
+def rotary_angles(out, positions, freq, freq_lo) -> None:
+    """out[t, i] = (cos, sin) of positions[t] * (freq[i] + freq_lo[i]), the product in 64-bit; out
+    float32 [T, n, 2]."""
+    what = "rotary_angles"
+    _need(out, torch.float32, "out", what)
+    _need(positions, torch.int32, "positions", what)
+    _need(freq, torch.float32, "freq", what)
+    n, half = out.shape[0], out.shape[1]
+    if out.dim() != 3 or out.shape[2] != 2 or positions.numel() < n or freq.numel() < half:
+        raise KernelArgumentError(f"{what}: shapes do not fit")
+    _check(lib().prb_rotary_angles(_p(out), _p(positions), _p(freq), _p(_freq_lo(freq_lo, 2 * half, what)),
+                                   n, half, _stream()), what)
+
+
+def _angles(angles, rows: int, rot_dims: int, what: str):
+    """``angles``: float32 [>= rows, rot_dims / 2, 2] (cosine and sine, see :func:`rotary_angles`),
+    or None: the kernel computes them from its frequencies."""
+    if angles is not None:
+        _need(angles, torch.float32, "angles", what)
+        if angles.dim() != 3 or angles.shape[0] < rows or angles.shape[1] != rot_dims // 2 or \
+                angles.shape[2] != 2:
+            raise KernelArgumentError(f"{what}: angles must be [rows, {rot_dims // 2}, 2]")
+    return angles
 
 
 def route(scale, chosen, chosen_w, x, w, bias, top: int) -> None:
@@ -1230,9 +1313,10 @@ def latent_attention_mma(out, qa, cache, block_table, seq_of_token, positions, i
 
 
 # ------------------------------------------------- scaled embedding, routing by scores
-def embed_scaled(out, tokens, table, scale: float, keep=None, status=None) -> None:
+def embed_scaled(out, tokens, table, scale: float, keep=None, status=None, pair=None) -> None:
     """out[t] = table[tokens[t]] * scale (float32 [T, width]); ``keep`` receives the same rows
-    a second time (a stream that is joined by its own beginning again later)."""
+    a second time (a stream that is joined by its own beginning again later); ``pair``, in the
+    table's type and at least 2 * width wide, the row twice side by side."""
     what = "embed_scaled"
     _need(out, torch.float32, "out", what)
     _need(tokens, torch.int32, "tokens", what)
@@ -1244,9 +1328,13 @@ def embed_scaled(out, tokens, table, scale: float, keep=None, status=None) -> No
         _need(keep, torch.float32, "keep", what)
         if keep.shape[0] < n or keep.shape[1] != width:
             raise KernelArgumentError(f"{what}: keep has the wrong shape")
+    if pair is not None and (not pair.is_cuda or pair.dtype != table.dtype or pair.stride(1) != 1 or
+                             pair.shape[0] < n or pair.shape[1] < 2 * width):
+        raise KernelArgumentError(f"{what}: pair has the wrong shape or type")
     _check(lib().prb_embed_scaled(_p(out), _p(keep), _p(tokens), _p(table), n, width,
-                                  table.shape[0], float(scale), dtype_code(table.dtype),
-                                  _p(status), _stream()), what)
+                                  table.shape[0], float(scale), dtype_code(table.dtype), _p(pair),
+                                  0 if pair is None else pair.stride(0), _p(status), _stream()),
+           what)
 
 
 SCORE_CODES = {"sigmoid": 0, "identity": 1, "softmax": 2}
@@ -1334,10 +1422,12 @@ def retention_step_supports(dim: int, vdim: int) -> bool:
 
 def retention_step(out, proj, q_col: int, k_col: int, v_col: int, g_col: int, state, q_start,
                    state_slot, positions, decay, freq, n_requests: int, heads: int, dim: int,
-                   vdim: int, rot_dims: int, k_scale: float, eps: float, status=None) -> None:
+                   vdim: int, rot_dims: int, k_scale: float, eps: float, status=None,
+                   angles=None) -> None:
     """Rotation, recurrence and finish (:func:`retention_scan` and :func:`retention_finish`) of
     a step of few tokens in ONE launch, a CTA per (head, request); ``proj`` is not changed.
-    ``g_col`` < 0: no gate.  out in the activation type, rows may be wider than heads * vdim."""
+    ``g_col`` < 0: no gate.  out in the activation type, rows may be wider than heads * vdim.
+    ``angles``: the step's table of cosines and sines (:func:`rotary_angles`), or None."""
     what = "retention_step"
     _need(state, torch.float32, "state", what)
     _need(decay, torch.float32, "decay", what)
@@ -1359,7 +1449,8 @@ def retention_step(out, proj, q_col: int, k_col: int, v_col: int, g_col: int, st
                                     _p(state_slot), _p(positions), _p(decay), _p(freq), n,
                                     int(n_requests), state.shape[0], heads, dim, vdim,
                                     int(rot_dims), float(k_scale), float(eps),
-                                    dtype_code(out.dtype), _p(status), _stream()), what)
+                                    dtype_code(out.dtype), _p(_angles(angles, n, rot_dims, what)),
+                                    _p(status), _stream()), what)
 
 
 def retention_lanes(dim: int) -> int:
@@ -1379,7 +1470,8 @@ def retention_max_segments(t_cap: int, b_cap: int) -> int:
 
 def retention_scan(o_raw, proj, q_col: int, k_col: int, v_col: int, state, q_start, state_slot,
                    positions, decay, freq, n_requests: int, heads: int, dim: int, vdim: int,
-                   rot_dims: int, k_scale: float, cols: int, status=None, segments=None) -> None:
+                   rot_dims: int, k_scale: float, cols: int, status=None, segments=None,
+                   angles=None) -> None:
     """o_raw[t, h] = S_t^T q_t with S_t = decay_h S_(t-1) + k_t v_t^T per request and head, over
     the step's tokens in order, from and back to ``state`` [slots, heads, vdim, dim] float32
     (zero at position 0).  proj float32 [T, ld] holds q, k (heads * dim) and v (heads * vdim)
@@ -1417,7 +1509,8 @@ def retention_scan(o_raw, proj, q_col: int, k_col: int, v_col: int, state, q_sta
                                     int(v_col), _p(state), _p(q_start), _p(state_slot),
                                     _p(positions), _p(decay), _p(freq), n, int(n_requests),
                                     state.shape[0], heads, dim, vdim, int(rot_dims), float(k_scale),
-                                    int(cols), _p(seg_own), _p(seg_start), n_seg, _p(status),
+                                    int(cols), _p(seg_own), _p(seg_start), n_seg,
+                                    _p(_angles(angles, n, rot_dims, what)), _p(status),
                                     _stream()), what)
     # (the rotation is a launch of its own; the segmented scan is three)
     add_launches((1 if rot_dims > 0 or float(k_scale) != 1.0 else 0) + (2 if n_seg else 0))
@@ -1668,16 +1761,24 @@ def tmix_finish(out, raw, proj, g_col: int, norm_w, seq_of_token, heads: int, vd
 def wattn_prepare(q_out, cache, proj, q_col: int, k_col: int, v_col: int, q_norm, k_norm, slots,
                   positions, freq, heads: int, kv_heads: int, dim: int, vdim: int, rot_dims: int,
                   eps: float, temp_coef: float, temp_every: int, status=None, head_norm=None,
-                  biases=None, freq_lo=None) -> None:
+                  biases=None, freq_lo=None, angles=None, interleaved: bool = False,
+                  keys_are_values: bool = False, conv=None) -> None:
     """Queries and keys of the step's tokens as the attention reads them: a root-mean-square
     norm over the whole projection (``q_norm`` / ``k_norm``: float32 weights, or None), or per
     head (``head_norm`` "before": before the rotation, ``q_norm`` / ``k_norm`` of ``dim`` numbers
     shared by the heads; "after": after the rotation, without weights), ``biases`` = (q, k, v)
     float32 vectors (or None each) that join the projection first, the
     query's temperature 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1) (``temp_every`` 0:
-    none), the rotation of each head's first ``rot_dims`` coordinates (rotate-half).  Queries go
+    none), the rotation of each head's first ``rot_dims`` coordinates (rotate-half, or
+    ``interleaved`` pairs; from ``angles``, see :func:`rotary_angles`, or from ``freq``).  Queries go
     to q_out float32 [T, heads * dim]; keys and values to the tokens' cache rows [k | v]
-    (cache [pages, kv_heads, page size, dim + vdim]; ``slots`` None: nothing is cached)."""
+    (cache [pages, kv_heads, page size, dim + vdim]; ``slots`` None: nothing is cached).
+
+    ``conv`` = (q taps [heads * dim, n], k taps [kv_heads * dim, n], state [slots, n - 1, (heads +
+    kv_heads) * dim], seq_of_token, q_start, state_slot, requests): a causal convolution over
+    time on every channel of q and k, before norm and rotation.  ``requests`` 0: every request
+    of the step brings one token; else how many requests to bring the state up to date for.
+    ``keys_are_values``: there is no value projection; a key before norm and rotation is its value."""
     what = "wattn_prepare"
     _need(q_out, torch.float32, "q_out", what)
     _need(cache, None, "cache", what)
@@ -1689,11 +1790,12 @@ def wattn_prepare(q_out, cache, proj, q_col: int, k_col: int, v_col: int, q_norm
     pages, kvh, page_size, rowlen = cache.shape
     if kvh != kv_heads or rowlen != dim + vdim or q_out.shape[1] != heads * dim or \
             proj.shape[0] < n or q_col + heads * dim > proj.shape[1] or \
-            freq.numel() < max(1, rot_dims // 2):
+            freq.numel() < max(1, rot_dims // 2) or (keys_are_values and vdim != dim):
         raise KernelArgumentError(f"{what}: shapes do not fit")
     if slots is not None:
         _need(slots, torch.int32, "slots", what)
-        if k_col + kv_heads * dim > proj.shape[1] or v_col + kv_heads * vdim > proj.shape[1]:
+        if k_col + kv_heads * dim > proj.shape[1] or \
+                (not keys_are_values and v_col + kv_heads * vdim > proj.shape[1]):
             raise KernelArgumentError(f"{what}: key or value columns outside the projection")
     if head_norm not in (None, "before", "after"):
         raise KernelArgumentError(f"{what}: head_norm is None, 'before' or 'after'")
@@ -1713,13 +1815,49 @@ def wattn_prepare(q_out, cache, proj, q_col: int, k_col: int, v_col: int, q_norm
             _need(t, torch.float32, name, what)
             if t.numel() != size:
                 raise KernelArgumentError(f"{what}: the {name} must hold {size} numbers")
-    _check(lib().prb_wattn_prepare(_p(q_out), _p(cache), _p(proj), proj.stride(0), int(q_col),
-                                   int(k_col), int(v_col), _p(q_norm), _p(k_norm), _p(slots),
-                                   _p(positions), _p(freq), n, heads, kv_heads, dim, vdim,
-                                   int(rot_dims), float(eps), float(temp_coef), int(temp_every),
-                                   page_size, pages, dtype_code(cache.dtype), mode, _p(bq),
-                                   _p(bk), _p(bv), _p(_freq_lo(freq_lo, rot_dims, what)),
-                                   _p(status), _stream()), what)
+    lo = _freq_lo(freq_lo, rot_dims, what)
+    if mode < 2 and biases is None and not interleaved and not keys_are_values and conv is None and \
+            (mode == 1 or angles is None):
+        # (norms over whole projections, or none)
+        _check(lib().prb_wattn_prepare(_p(q_out), _p(cache), _p(proj), proj.stride(0), int(q_col),
+                                       int(k_col), int(v_col), _p(q_norm), _p(k_norm), _p(slots),
+                                       _p(positions), _p(freq), n, heads, kv_heads, dim, vdim,
+                                       int(rot_dims), float(eps), float(temp_coef), int(temp_every),
+                                       page_size, pages, dtype_code(cache.dtype), _p(lo), _p(status),
+                                       _stream()), what)
+        return
+    if mode == 1:
+        raise KernelArgumentError(f"{what}: a norm over whole projections goes with neither biases, "
+                                  f"a convolution, interleaved pairs nor keys as values")
+    wq = wk = state = seq = q_start = state_slot = None
+    taps = n_slots = requests = 0
+    if conv is not None:
+        wq, wk, state, seq, q_start, state_slot, requests = conv
+        taps = wq.shape[1]
+        _need(wq, torch.float32, "q taps", what)
+        _need(wk, torch.float32, "k taps", what)
+        for name, t in (("seq_of_token", seq), ("q_start", q_start), ("state_slot", state_slot)):
+            _need(t, torch.int32, name, what)
+        if tuple(wq.shape) != (heads * dim, taps) or tuple(wk.shape) != (kv_heads * dim, taps) or \
+                seq.numel() < n or q_start.numel() < requests + 1 or state_slot.numel() < requests:
+            raise KernelArgumentError(f"{what}: the convolution's shapes do not fit")
+        n_slots = state.shape[0]
+        if taps > 1:
+            _need(state, torch.float32, "convolution state", what)
+            if tuple(state.shape[1:]) != (taps - 1, (heads + kv_heads) * dim):
+                raise KernelArgumentError(f"{what}: the convolution's state has the wrong shape")
+        else:
+            state = None
+    _check(lib().prb_wattn_prepare_heads(
+        _p(q_out), _p(cache), _p(proj), proj.stride(0), int(q_col), int(k_col),
+        -1 if keys_are_values else int(v_col), _p(q_norm), _p(k_norm), _p(bq), _p(bk), _p(bv), _p(wq),
+        _p(wk), taps, _p(state), n_slots, _p(seq), _p(q_start), _p(state_slot), int(requests),
+        _p(slots), _p(positions), _p(freq), _p(lo), _p(_angles(angles, n, rot_dims, what)), n, heads,
+        kv_heads, dim, vdim, int(rot_dims), int(bool(interleaved)), mode, float(eps),
+        float(temp_coef), int(temp_every), page_size, pages, dtype_code(cache.dtype), _p(status),
+        _stream()), what)
+    if taps > 1 and requests > 0:
+        add_launches(1)
 
 
 def wattn_tile_rows(heads: int, kv_heads: int, dim: int, vdim: int) -> int:
@@ -1736,10 +1874,11 @@ def wattn_single_supports(heads: int, kv_heads: int, dim: int, vdim: int) -> boo
 def wattn(out, q, cache, block_table, seq_of_token, positions, heads: int, dim: int, vdim: int,
           window: int, keep_first: int, scale: float, gate=None, slopes=None,
           out_scale: float = 1.0, status=None, tile_rows: int = 0, single: bool = False,
-          sinks=None, gate_per_value: bool = False) -> None:
+          sinks=None, gate_per_value: bool = False, softcap: float = 0.0) -> None:
     """Softmax attention over cache rows [k | v]: a query at position i sees key j <= i with
     i - j < window (``window`` 0: all) or j < keep_first; score (q . k) * scale - slopes[h] * (i
-    - j); ``sinks`` (float32 [heads]): exp(sinks[h]) joins the softmax's denominator once,
+    - j), with ``softcap`` > 0 softcap * tanh((q . k) * scale / softcap) in the place of the
+    first term; ``sinks`` (float32 [heads]): exp(sinks[h]) joins the softmax's denominator once,
     without a key or a value; head h's result times sigmoid(gate[t, h]) (``gate``: float32, may
     be a column slice; ``gate_per_value``: [rows, heads * vdim], a gate per value coordinate) times
     ``out_scale``.  32-bit arithmetic; out in the cache's type.  ``tile_rows`` > 0: the
@@ -1780,7 +1919,7 @@ def wattn(out, q, cache, block_table, seq_of_token, positions, heads: int, dim: 
               _p(positions), _p(gate), gate_ld, _p(slopes), n, heads, kv_heads, dim, vdim,
               page_size, block_table.shape[1], pages, int(window or 0), int(keep_first or 0))
     tail = (float(scale), float(out_scale), dtype_code(cache.dtype), dtype_code(out.dtype),
-            _p(sinks), gate_per, _p(status), _stream())
+            _p(sinks), gate_per, float(softcap or 0.0), _p(status), _stream())
     if single:
         _check(lib().prb_wattn_single(*common, *tail), what)
     elif tile_rows > 0:

@@ -39,12 +39,25 @@ struct ScanArgs {
     float* seg_start;         // [segments, heads, vdim, dim]: the states at the segments' starts
 };
 
+// Cosine and sine of pair w at token t: from the step's table, if it has one, else computed.
+__device__ __forceinline__ void ret_angle(const float2* angles, int t, int half, int w, float pos,
+                                          const float* freq, float& sn, float& cs) {
+    if (angles != nullptr) {
+        const float2 v = angles[(size_t)t * half + w];
+        cs = v.x;
+        sn = v.y;
+    } else {
+        prb_sincos_angle(pos, freq[w], &sn, &cs);
+    }
+}
+
 // q and k of every token of the step, in place in the projection's 32-bit result: the first
 // rot_dims coordinates of every head turned by the token's position (rotate-half layout), k
 // times k_scale afterwards.  A CTA per token.
 __global__ void retention_rotate_kernel(float* __restrict__ proj, long ld, int q_col, int k_col,
                                         const int* __restrict__ positions,
-                                        const float* __restrict__ freq, int n_tokens, int heads,
+                                        const float* __restrict__ freq,
+                                        const float2* __restrict__ angles, int n_tokens, int heads,
                                         int dim, int rot_dims, float k_scale) {
     prb_grid_launch_dependents();
     const int t = blockIdx.x;
@@ -59,7 +72,7 @@ __global__ void retention_rotate_kernel(float* __restrict__ proj, long ld, int q
         float* kr = row + k_col + h * dim;
         if (w < half) {
             float sn, cs;
-            sincosf(pos * freq[w], &sn, &cs);
+            ret_angle(angles, t, half, w, pos, freq, sn, cs);
             const float q0 = qr[w], q1 = qr[w + half], k0 = kr[w], k1 = kr[w + half];
             qr[w] = q0 * cs - q1 * sn;
             qr[w + half] = q1 * cs + q0 * sn;
@@ -241,6 +254,7 @@ __global__ void retention_carry_kernel(ScanArgs a) {
 struct StepArgs {
     ScanArgs scan;            // cols == vdim
     const float* freq;
+    const float2* angles;     // [T, rot_dims / 2] cosine and sine, or null: computed from freq
     int rot_dims;
     float k_scale, eps;
     void* out;                // [T, out_ld] in O
@@ -289,7 +303,7 @@ __global__ void retention_step_kernel(StepArgs sa) {
         for (int w = threadIdx.x; w < units; w += blockDim.x) {
             if (w < half) {
                 float sn, cs;
-                sincosf(pos * sa.freq[w], &sn, &cs);
+                ret_angle(sa.angles, t, half, w, pos, sa.freq, sn, cs);
                 const float q0 = qr[w], q1 = qr[w + half], k0 = kr[w], k1 = kr[w + half];
                 qs[w] = q0 * cs - q1 * sn;
                 qs[w + half] = q1 * cs + q0 * sn;
@@ -419,7 +433,8 @@ PRB_API int prb_retention_scan(float* o_raw, float* proj, long ld, int q_col, in
                                const int* positions, const float* decay, const float* freq,
                                int n_tokens, int n_requests, int n_slots, int heads, int dim,
                                int vdim, int rot_dims, float k_scale, int cols, float* seg_own,
-                               float* seg_start, int segments, int* status, cudaStream_t stream) {
+                               float* seg_start, int segments, const void* angles, int* status,
+                              cudaStream_t stream) {
     if (n_tokens <= 0 || n_requests <= 0) return 0;
     const int lanes = prb_retention_lanes(dim);
     if (heads <= 0 || heads > 65535 || n_requests > 65535 || dim <= 0 || vdim <= 0 || lanes == 0 ||
@@ -433,7 +448,7 @@ PRB_API int prb_retention_scan(float* o_raw, float* proj, long ld, int q_col, in
         const int work = heads * (dim - rot_dims / 2);
         const int rt = work >= 256 ? 256 : ((work + 31) / 32) * 32;
         retention_rotate_kernel<<<n_tokens, rt, 0, stream>>>(proj, ld, q_col, k_col, positions, freq,
-                                                             n_tokens, heads, dim, rot_dims, k_scale);
+                                                             (const float2*)angles, n_tokens, heads, dim, rot_dims, k_scale);
         PRB_LAUNCH_CHECK();
     }
     // threads: cols * lanes rounded up to whole warps, at most 1,024
@@ -497,7 +512,8 @@ PRB_API int prb_retention_step(void* out, long out_ld, const float* proj, long l
                                const int* state_slot, const int* positions, const float* decay,
                                const float* freq, int n_tokens, int n_requests, int n_slots,
                                int heads, int dim, int vdim, int rot_dims, float k_scale, float eps,
-                               int out_dtype, int* status, cudaStream_t stream) {
+                               int out_dtype, const void* angles, int* status,
+                               cudaStream_t stream) {
     if (n_tokens <= 0 || n_requests <= 0) return 0;
     const int lanes = prb_retention_lanes(dim);
     if (heads <= 0 || heads > 65535 || n_requests > 65535 || dim <= 0 || vdim <= 0 ||
@@ -509,7 +525,7 @@ PRB_API int prb_retention_step(void* out, long out_ld, const float* proj, long l
     StepArgs sa{ScanArgs{nullptr, proj, ld, q_col, k_col, v_col, state, q_start, state_slot,
                          positions, decay, n_tokens, n_slots, heads, dim, vdim, vdim, lanes, status,
                          n_requests, 0, nullptr, nullptr},
-                freq, rot_dims, k_scale, eps, out, out_ld, g_col};
+                freq, (const float2*)angles, rot_dims, k_scale, eps, out, out_ld, g_col};
     const size_t smem = (size_t)(2 * lanes * ni + vdim) * sizeof(float);
     const dim3 grid(heads, n_requests);
     if (out_dtype == PRB_F32) {

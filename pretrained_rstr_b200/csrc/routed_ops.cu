@@ -14,21 +14,26 @@ namespace {
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // ------------------------------------------------------------------ scaled embedding
+// `pair` (optional): the row once more in the table's type, twice side by side ([row | row],
+// `pair_ld` elements a token): the input of a product that joins the stream with its beginning.
 template <typename W>
 __global__ void embed_scaled_kernel(float* __restrict__ out, float* __restrict__ keep,
                                     const int* __restrict__ tokens, const W* __restrict__ table,
-                                    int n_tokens, int width, int vocab, float scale, int* status) {
+                                    int n_tokens, int width, int vocab, float scale,
+                                    W* __restrict__ pair, long pair_ld, int* status) {
     prb_grid_launch_dependents();
     const int t = blockIdx.x;
     if (t >= n_tokens) return;
     const int tok = tokens[t];
     float* o = out + (size_t)t * width;
     float* k = keep ? keep + (size_t)t * width : nullptr;
+    W* pr = pair ? pair + (size_t)t * pair_ld : nullptr;
     if (tok < 0 || tok >= vocab) {
         if (threadIdx.x == 0) prb_set_status(status, PRB_S_TOKEN_RANGE, t, tok, vocab);
         for (int i = threadIdx.x; i < width; i += blockDim.x) {
             o[i] = 0.0f;
             if (k) k[i] = 0.0f;
+            if (pr) pr[i] = pr[width + i] = prb_from_float<W>(0.0f);
         }
         return;
     }
@@ -37,6 +42,7 @@ __global__ void embed_scaled_kernel(float* __restrict__ out, float* __restrict__
         const float v = prb_to_float<W>(e[i]) * scale;
         o[i] = v;
         if (k) k[i] = v;
+        if (pr) pr[i] = pr[width + i] = prb_from_float<W>(v);
     }
 }
 
@@ -254,16 +260,19 @@ __global__ void route_act_kernel(O* __restrict__ out, long out_ld, const float* 
 
 PRB_API int prb_embed_scaled(float* out, float* keep, const int* tokens, const void* table,
                              int n_tokens, int width, int vocab, float scale, int table_dtype,
-                             int* status, cudaStream_t stream) {
+                             void* pair, long pair_ld, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (width <= 0 || vocab <= 0) return PRB_E_SIZE;
+    if (pair != nullptr && pair_ld < 2L * width) return PRB_E_ARG;
     const int threads = width >= 256 ? 256 : ((width + 31) / 32) * 32;
     if (table_dtype == PRB_F32)
         embed_scaled_kernel<float><<<n_tokens, threads, 0, stream>>>(
-            out, keep, tokens, (const float*)table, n_tokens, width, vocab, scale, status);
+            out, keep, tokens, (const float*)table, n_tokens, width, vocab, scale, (float*)pair,
+            pair_ld, status);
     else if (table_dtype == PRB_BF16)
         embed_scaled_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
-            out, keep, tokens, (const __nv_bfloat16*)table, n_tokens, width, vocab, scale, status);
+            out, keep, tokens, (const __nv_bfloat16*)table, n_tokens, width, vocab, scale,
+            (__nv_bfloat16*)pair, pair_ld, status);
     else
         return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();

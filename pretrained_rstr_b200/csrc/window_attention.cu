@@ -2,13 +2,14 @@
 // key/value heads, key and value heads of different sizes, a sliding window that may keep a
 // sequence's first tokens visible, a bias that grows with the distance of query and key, a
 // root-mean-square norm over the whole query (and key) projection, a query temperature that
-// grows with the position, a norm per head before or after the rotation, biases, rotary
-// positions on a head's first coordinates, a learned sink per head in the softmax's
-// denominator, and a gate per head or per value coordinate on the result.  Every option is a
-// parameter; a mixer that leaves one out passes 0 / null.
+// grows with the position, rotary positions on a head's first coordinates, a cap on scores, a
+// sink per head in the softmax's denominator, and a gate per head or per value coordinate on
+// the result.  Every option is a parameter; a mixer that leaves one out passes 0 / null.
+// (What acts on queries and keys head by head before they are attended to, norms per head,
+// biases, a short convolution, is in window_attention_prepare.cu.)
 //
 //   visible(i, j) = j <= i and (i - j < window or j < keep_first)         (window 0: all j <= i)
-//   score(i, j)   = (q_i . k_j) * scale - slope_h * (i - j)
+//   score(i, j)   = (q_i . k_j) * scale, capped by cap * tanh(score / cap), - slope_h * (i - j)
 //   w(i, j)       = exp(score(i, j)) / (sum_j' exp(score(i, j')) + exp(sink_h))
 //   o_i           = (sum_j w(i, j) v_j) * sigmoid(gate_i,h or gate_i,h,c) * out_scale
 //
@@ -38,6 +39,10 @@ constexpr int WA_SEG = 256;         // keys scored at a time
 constexpr int WA_MAX_V = 4;         // value coordinates a thread owns at most (vdim <= 512)
 constexpr int NO_WINDOW = 1 << 30;
 
+// A cap on scores (0: none).
+__device__ __forceinline__ float wa_cap(float s, float cap) {
+    return cap > 0.0f ? cap * tanhf(s / cap) : s;
+}
 __device__ __forceinline__ float wa_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // A learned sink joins a finished softmax: the denominator l (taken against the maximum m)
@@ -89,70 +94,6 @@ __device__ __forceinline__ void wa_project(const float* __restrict__ src, int n_
     }
 }
 
-// The same with a norm per HEAD (norm_mode 2: before the rotation, with a weight of `dim`
-// numbers that all heads share; 3: after the rotation, without a weight) and a bias that joins
-// the projection first.  A warp takes a head: its sum of squares is a warp's, whatever the
-// number of heads.
-template <typename D, typename F>
-__device__ __forceinline__ void wa_project_heads(const float* __restrict__ src,
-                                                 const float* __restrict__ bias, int n_heads,
-                                                 int dim, int rot_dims, int norm_mode,
-                                                 const float* __restrict__ norm_w, float eps,
-                                                 float factor, float pos,
-                                                 const float* __restrict__ freq,
-                                                 const float* __restrict__ freq_lo, F dst) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    const int half = rot_dims / 2;
-    const int units = half + (dim - rot_dims);
-    for (int hd = warp; hd < n_heads; hd += nwarps) {
-        const float* s = src + hd * dim;
-        const float* bb = bias ? bias + hd * dim : nullptr;
-        float inv = 1.0f;
-        if (norm_mode == 2) {
-            float ss = 0.0f;
-            for (int i = lane; i < dim; i += 32) {
-                const float v = s[i] + (bb ? bb[i] : 0.0f);
-                ss = fmaf(v, v, ss);
-            }
-            inv = 1.0f / sqrtf(prb_warp_sum(ss) / (float)dim + eps);
-        } else if (norm_mode == 3) {
-            float ss = 0.0f;
-            for (int u = lane; u < units; u += 32) {
-                if (u < half) {
-                    float sn, cs;
-                    prb_sincos_angle(pos, freq[u], &sn, &cs, freq_lo ? freq_lo[u] : 0.0f);
-                    const float a = s[u] + (bb ? bb[u] : 0.0f);
-                    const float b = s[u + half] + (bb ? bb[u + half] : 0.0f);
-                    const float ra = a * cs - b * sn, rb = b * cs + a * sn;
-                    ss = fmaf(ra, ra, fmaf(rb, rb, ss));
-                } else {
-                    const int i = u - half + rot_dims;
-                    const float v = s[i] + (bb ? bb[i] : 0.0f);
-                    ss = fmaf(v, v, ss);
-                }
-            }
-            inv = 1.0f / sqrtf(prb_warp_sum(ss) / (float)dim + eps);
-        }
-        const float pre = norm_mode == 2 ? inv : 1.0f;
-        const float post = (norm_mode == 3 ? inv : 1.0f) * factor;
-        const float* nw = norm_mode == 2 ? norm_w : nullptr;
-        D* d = dst(hd);
-        for (int u = lane; u < units; u += 32) {
-            if (u < half) {
-                float sn, cs;
-                prb_sincos_angle(pos, freq[u], &sn, &cs, freq_lo ? freq_lo[u] : 0.0f);
-                const float a = (s[u] + (bb ? bb[u] : 0.0f)) * pre * (nw ? nw[u] : 1.0f);
-                const float b = (s[u + half] + (bb ? bb[u + half] : 0.0f)) * pre * (nw ? nw[u + half] : 1.0f);
-                d[u] = prb_from_float<D>((a * cs - b * sn) * post);
-                d[u + half] = prb_from_float<D>((b * cs + a * sn) * post);
-            } else {
-                const int i = u - half + rot_dims;
-                d[i] = prb_from_float<D>((s[i] + (bb ? bb[i] : 0.0f)) * pre * (nw ? nw[i] : 1.0f) * post);
-            }
-        }
-    }
-}
-
 template <typename C>
 __global__ void wattn_prepare_kernel(float* __restrict__ q_out, C* __restrict__ cache,
                                      const float* __restrict__ proj, long ld, int q_col, int k_col,
@@ -162,9 +103,6 @@ __global__ void wattn_prepare_kernel(float* __restrict__ q_out, C* __restrict__ 
                                      const float* __restrict__ freq, int n_tokens, int heads,
                                      int kv_heads, int dim, int vdim, int rot_dims, float eps,
                                      float temp_coef, int temp_every, int page_size, int num_pages,
-                                     int norm_mode, const float* __restrict__ q_bias,
-                                     const float* __restrict__ k_bias,
-                                     const float* __restrict__ v_bias,
                                      const float* __restrict__ freq_lo, int* status) {
     __shared__ float scratch[32];
     prb_grid_launch_dependents();
@@ -176,13 +114,8 @@ __global__ void wattn_prepare_kernel(float* __restrict__ q_out, C* __restrict__ 
     float temp = 1.0f;
     if (temp_every > 0) temp = 1.0f + temp_coef * logf((float)((p + 1) / temp_every) + 1.0f);
     float* qo = q_out + (size_t)t * heads * dim;
-    const bool per_head = norm_mode >= 2 || q_bias != nullptr || k_bias != nullptr;
-    if (per_head)
-        wa_project_heads<float>(row + q_col, q_bias, heads, dim, rot_dims, norm_mode, q_norm, eps,
-                                temp, pos, freq, freq_lo, [&](int hd) { return qo + hd * dim; });
-    else
-        wa_project<float>(row + q_col, heads, dim, rot_dims, q_norm, eps, temp, pos, freq, freq_lo, scratch,
-                          [&](int hd) { return qo + hd * dim; });
+    wa_project<float>(row + q_col, heads, dim, rot_dims, q_norm, eps, temp, pos, freq, freq_lo, scratch,
+                      [&](int hd) { return qo + hd * dim; });
     if (slots == nullptr) return;
     const int slot = slots[t];
     if (slot < 0) return;
@@ -194,16 +127,11 @@ __global__ void wattn_prepare_kernel(float* __restrict__ q_out, C* __restrict__ 
     const int rowlen = dim + vdim;
     C* base = cache + (((size_t)page * kv_heads) * page_size + off) * rowlen;
     const size_t head_step = (size_t)page_size * rowlen;
-    if (per_head)
-        wa_project_heads<C>(row + k_col, k_bias, kv_heads, dim, rot_dims, norm_mode, k_norm, eps,
-                            1.0f, pos, freq, freq_lo, [&](int hd) { return base + hd * head_step; });
-    else
-        wa_project<C>(row + k_col, kv_heads, dim, rot_dims, k_norm, eps, 1.0f, pos, freq, freq_lo, scratch,
-                      [&](int hd) { return base + hd * head_step; });
+    wa_project<C>(row + k_col, kv_heads, dim, rot_dims, k_norm, eps, 1.0f, pos, freq, freq_lo, scratch,
+                  [&](int hd) { return base + hd * head_step; });
     for (int u = threadIdx.x; u < kv_heads * vdim; u += blockDim.x) {
         const int g = u / vdim, j = u - g * vdim;
-        base[g * head_step + dim + j] =
-            prb_from_float<C>(row[v_col + u] + (v_bias ? v_bias[u] : 0.0f));
+        base[g * head_step + dim + j] = prb_from_float<C>(row[v_col + u]);
     }
 }
 
@@ -216,7 +144,7 @@ wattn_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ q,
              const float* __restrict__ gate, long gate_ld, const float* __restrict__ slopes,
              int n_tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
              int max_pages, int num_pages, int window, int keep_first, float scale,
-             float out_scale, const float* __restrict__ sinks, int gate_per, int* status) {
+             float out_scale, const float* __restrict__ sinks, int gate_per, float softcap, int* status) {
     extern __shared__ float smem[];
     __shared__ float scratch[32];
     float* qs = smem;                        // [dim]
@@ -268,7 +196,7 @@ wattn_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ q,
                 const C* kp = cache + (((size_t)page * kv_heads + g) * page_size + (j % page_size)) * rowlen;
                 float a = 0.0f;
                 for (int d = 0; d < dim; ++d) a = fmaf(qs[d], prb_to_float<C>(kp[d]), a);
-                s = a * scale - slope * (float)(pos - j);
+                s = wa_cap(a * scale, softcap) - slope * (float)(pos - j);
             }
             wgt[i] = s;
             mx = fmaxf(mx, s);
@@ -337,7 +265,7 @@ wattn_tile_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ q,
                   const float* __restrict__ gate, long gate_ld, const float* __restrict__ slopes,
                   int n_tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
                   int max_pages, int num_pages, int window, int keep_first, int tq, float scale,
-                  float out_scale, const float* __restrict__ sinks, int gate_per, int* status) {
+                  float out_scale, const float* __restrict__ sinks, int gate_per, float softcap, int* status) {
     extern __shared__ __align__(16) float smem[];
     __shared__ int pages_s[WT_KB];
     prb_grid_launch_dependents();
@@ -488,7 +416,7 @@ wattn_tile_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ q,
                 e[x] = 0.0f;
                 if (!act[x]) continue;
                 const bool vis = j < j_end && j <= pi[x] && (pi[x] - j < win || j < keep_first);
-                const float tt = vis ? s[x] - slope[x] * (float)(pi[x] - j) : -INFINITY;
+                const float tt = vis ? wa_cap(s[x], softcap) - slope[x] * (float)(pi[x] - j) : -INFINITY;
                 const float nm = fmaxf(m[x], prb_warp_max(tt));
                 const float f = expf(m[x] - nm);                   // (exp(-inf) = 0)
                 e[x] = vis ? expf(tt - nm) : 0.0f;
@@ -589,7 +517,7 @@ wattn_single_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ 
                     const float* __restrict__ gate, long gate_ld, const float* __restrict__ slopes,
                     int n_tokens, int heads, int kv_heads, int dim, int vdim, int page_size,
                     int max_pages, int num_pages, int window, int keep_first, float scale,
-                    float out_scale, const float* __restrict__ sinks, int gate_per, int* status) {
+                    float out_scale, const float* __restrict__ sinks, int gate_per, float softcap, int* status) {
     extern __shared__ __align__(16) float smem[];
     __shared__ long long rows_s[WT_WARPS * WT_KB];   // a staged key's row of the cache, or -1
     prb_grid_launch_dependents();
@@ -723,7 +651,7 @@ wattn_single_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ 
         for (int x = 0; x < PPW; ++x) {
             e[x] = 0.0f;
             if (x >= hg) continue;
-            const float tt = vis ? s[x] - slope[x] * (float)(p - j) : -INFINITY;
+            const float tt = vis ? wa_cap(s[x], softcap) - slope[x] * (float)(p - j) : -INFINITY;
             const float nm = fmaxf(m[x], prb_warp_max(tt));
             if (nm == -INFINITY) continue;           // (no key of the block is seen)
             const float f = expf(m[x] - nm);         // (exp(-inf) = 0)
@@ -821,11 +749,9 @@ PRB_API int prb_wattn_prepare(float* q_out, void* cache, const float* proj, long
                               const int* slots, const int* positions, const float* freq,
                               int n_tokens, int heads, int kv_heads, int dim, int vdim, int rot_dims,
                               float eps, float temp_coef, int temp_every, int page_size,
-                              int num_pages, int cache_dtype, int norm_mode, const float* q_bias,
-                              const float* k_bias, const float* v_bias, const float* freq_lo,
-                              int* status, cudaStream_t stream) {
+                              int num_pages, int cache_dtype, const float* freq_lo, int* status,
+                              cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (norm_mode < 0 || norm_mode > 3) return PRB_E_ARG;
     if (heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rot_dims < 0 || rot_dims % 2 ||
         rot_dims > dim || page_size <= 0)
         return PRB_E_SIZE;
@@ -833,12 +759,12 @@ PRB_API int prb_wattn_prepare(float* q_out, void* cache, const float* proj, long
         wattn_prepare_kernel<float><<<n_tokens, 256, 0, stream>>>(
             q_out, (float*)cache, proj, ld, q_col, k_col, v_col, q_norm, k_norm, slots, positions,
             freq, n_tokens, heads, kv_heads, dim, vdim, rot_dims, eps, temp_coef, temp_every,
-            page_size, num_pages, norm_mode, q_bias, k_bias, v_bias, freq_lo, status);
+            page_size, num_pages, freq_lo, status);
     else if (cache_dtype == PRB_BF16)
         wattn_prepare_kernel<__nv_bfloat16><<<n_tokens, 256, 0, stream>>>(
             q_out, (__nv_bfloat16*)cache, proj, ld, q_col, k_col, v_col, q_norm, k_norm, slots,
             positions, freq, n_tokens, heads, kv_heads, dim, vdim, rot_dims, eps, temp_coef,
-            temp_every, page_size, num_pages, norm_mode, q_bias, k_bias, v_bias, freq_lo, status);
+            temp_every, page_size, num_pages, freq_lo, status);
     else
         return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();
@@ -850,7 +776,7 @@ PRB_API int prb_wattn(void* out, long out_ld, const float* q, const void* cache,
                       const float* gate, long gate_ld, const float* slopes, int n_tokens, int heads,
                       int kv_heads, int dim, int vdim, int page_size, int max_pages, int num_pages,
                       int window, int keep_first, float scale, float out_scale, int cache_dtype,
-                      int out_dtype, const float* sinks, int gate_per, int* status,
+                      int out_dtype, const float* sinks, int gate_per, float softcap, int* status,
                       cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || heads > 65535 || dim <= 0 ||
@@ -864,7 +790,7 @@ PRB_API int prb_wattn(void* out, long out_ld, const float* q, const void* cache,
     wattn_kernel<CT, OT><<<grid, WA_THREADS, smem, stream>>>(                                    \
         (OT*)out, out_ld, q, (const CT*)cache, block_table, seq_of_token, positions, gate,       \
         gate_ld, slopes, n_tokens, heads, kv_heads, dim, vdim, page_size, max_pages, num_pages,  \
-        window, keep_first, scale, out_scale, sinks, gate_per, status)
+        window, keep_first, scale, out_scale, sinks, gate_per, softcap, status)
     if (cache_dtype == PRB_F32 && out_dtype == PRB_F32) WATTN(float, float);
     else if (cache_dtype == PRB_BF16 && out_dtype == PRB_BF16) WATTN(__nv_bfloat16, __nv_bfloat16);
     else return PRB_E_DTYPE;
@@ -888,7 +814,7 @@ PRB_API int prb_wattn_tile(void* out, long out_ld, const float* q, const void* c
                            int heads, int kv_heads, int dim, int vdim, int page_size, int max_pages,
                            int num_pages, int window, int keep_first, int tq, float scale,
                            float out_scale, int cache_dtype, int out_dtype, const float* sinks,
-                           int gate_per, int* status, cudaStream_t stream) {
+                           int gate_per, float softcap, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     const int most = prb_wattn_tile_rows(heads, kv_heads, dim, vdim);
     if (most <= 0 || kv_heads > 65535 || page_size <= 0 || max_pages <= 0 || window < 0 ||
@@ -905,7 +831,7 @@ PRB_API int prb_wattn_tile(void* out, long out_ld, const float* q, const void* c
         wattn_tile_kernel<CT, OT, VCN><<<grid, WT_WARPS * 32, smem, stream>>>(                   \
             (OT*)out, out_ld, q, (const CT*)cache, block_table, seq_of_token, positions, gate,   \
             gate_ld, slopes, n_tokens, heads, kv_heads, dim, vdim, page_size, max_pages,         \
-            num_pages, window, keep_first, tq, scale, out_scale, sinks, gate_per, status);       \
+            num_pages, window, keep_first, tq, scale, out_scale, sinks, gate_per, softcap, status);       \
     } while (0)
 #define WATT(CT, OT)                                                                             \
     do {                                                                                         \
@@ -936,7 +862,7 @@ PRB_API int prb_wattn_single(void* out, long out_ld, const float* q, const void*
                              int heads, int kv_heads, int dim, int vdim, int page_size,
                              int max_pages, int num_pages, int window, int keep_first, float scale,
                              float out_scale, int cache_dtype, int out_dtype, const float* sinks,
-                             int gate_per, int* status, cudaStream_t stream) {
+                             int gate_per, float softcap, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (cache_dtype != PRB_F32 && cache_dtype != PRB_BF16) return PRB_E_DTYPE;
     const int csize = cache_dtype == PRB_F32 ? 4 : 2;
@@ -976,7 +902,7 @@ PRB_API int prb_wattn_single(void* out, long out_ld, const float* q, const void*
                            (const CT*)cache, block_table, seq_of_token, positions, gate,         \
                            gate_ld, slopes, n_tokens, heads, kv_heads, dim, vdim, page_size,     \
                            max_pages, num_pages, window, keep_first, scale, out_scale, sinks,    \
-                           gate_per, status);                                                    \
+                           gate_per, softcap, status);                                                    \
     } while (0)
 #define WS1(CT, OT, VCN)                                                                         \
     do {                                                                                         \

@@ -179,7 +179,8 @@ class ModelRunner:
                 count = view.host_counts.get(name) or 0
                 view.launch[name] = min(view.caps[array], -(-count // step) * step)
                 bounds.append(view.launch[name])
-        key = (lay.t_cap, lay.b_cap, rows_cap, filled, reach, tuple(bounds))
+        # (parts may run other kernels when every request brings one token)
+        key = (lay.t_cap, lay.b_cap, rows_cap, filled, reach, tuple(bounds), ctx.max_q_len > 1)
         ctx.launch_tokens, ctx.launch_rows = lay.t_cap, rows_cap
         self._counts_from_device(ctx)
         ctx.max_context = reach

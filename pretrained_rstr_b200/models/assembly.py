@@ -27,12 +27,16 @@ from ..parts.linear import LazyNorm
 
 class Model:
     def __init__(self, config, runtime, embedding, position, blocks, order, final_norm, head,
-                 width: int, vocab: int):
+                 width: int, vocab: int, join=None):
         self.config, self.runtime = config, runtime
         self.embedding, self.position = embedding, position
         self.blocks, self.order = blocks, order
         self.final_norm, self.head = final_norm, head
         self.width, self.vocab = width, vocab
+        self.join = join                    # joins the stream with the embedding's output, or None
+        if join is None and any(e.join_embedding for e in order):
+            raise ValueError("run order: an entry joins the stream with the embedding's output, and "
+                             "the configuration names no way to (stream_join_spec)")
         self.max_positions = config.max_positions
         #: optional ``tap(run index, x)`` called after every block (measurements and tests; a
         #: model with a tap is not replayed from CUDA graphs)
@@ -45,7 +49,7 @@ class Model:
         self._caches: List[LayerCache] = []
         # a step can be replayed as a CUDA graph only if every part launches the same
         # kernels whatever the step holds (parts say so with ``graph_safe = True``)
-        parts = [embedding, position, final_norm, head]
+        parts = [embedding, position, final_norm, head] + ([join] if join is not None else [])
         for blk in blocks:
             parts += [blk, blk.mixer, blk.feed_forward, *blk.norms.values()]
         self.graph_safe = all(getattr(p, "graph_safe", False) for p in parts)
@@ -119,6 +123,18 @@ class Model:
             self.embedding.bind_state(own)
 
     # --------------------------------------------------------------------- forward
+    def _reader_after(self, at: int, stream):
+        """What reads the stream after run entry ``at``: a norm, the join's buffer, or None (not
+        known, or the last entry, after which only wanted rows are read)."""
+        if at + 1 >= len(self.order):
+            return None
+        following = self.order[at + 1]
+        if following.join_embedding:
+            return stream
+        if following.add_embedding:
+            return None
+        return getattr(self.blocks[following.layer], "entry_norm", None)
+
     def forward(self, ctx) -> torch.Tensor:
         """Run the step's tokens through the model; returns float32 logits [rows, vocab]
         for ``ctx.logit_rows`` (a view of scratch memory whose rows are padded to a multiple
@@ -129,16 +145,35 @@ class Model:
         if any(e.add_embedding for e in self.order):
             # the stream's beginning is kept for the entries that add it again
             x0 = ctx.scratch("embedding_output", (ctx.token_capacity, self.width), torch.float32)[:t]
+        # [stream | embedding's output] in the activation type, for the entries that join the two
+        pair = self.join.buffer(ctx, t) if any(e.join_embedding for e in self.order) else None
+        kept = {}
         if x0 is not None and getattr(self.embedding, "keeps_copy", False):
-            self.embedding.forward(ctx, self.position, x, keep=x0)
-        else:
-            self.embedding.forward(ctx, self.position, x)
-            if x0 is not None:
-                ops.bias_act(x0, x, None, None, None)
-        for entry, cache in zip(self.order, self._caches):
+            kept["keep"] = x0
+        if pair is not None and getattr(self.embedding, "keeps_pair", False):
+            kept["pair"] = pair
+        self.embedding.forward(ctx, self.position, x, **kept)
+        if x0 is not None and "keep" not in kept:
+            ops.bias_act(x0, x, None, None, None)
+        if pair is not None and "pair" not in kept:
+            pair[:, :self.width].copy_(x)
+            pair[:, self.width:2 * self.width].copy_(x)
+        # what a block has left of the stream for whoever reads it next: (the reader, a tensor);
+        # the reader is the next block's first norm, or the join's buffer
+        stream = None if pair is None else pair[:, :self.width]
+        ctx.stream_left = (stream, stream)
+        for at, (entry, cache) in enumerate(zip(self.order, self._caches)):
             block = self.blocks[entry.layer]
             if entry.add_embedding:
                 ops.bias_act(x, x, None, x0, None)             # x += x0, in 32-bit
+                ctx.stream_left = None
+            if entry.join_embedding:
+                if ctx.stream_left is None or ctx.stream_left[0] is not stream:
+                    stream.copy_(x)
+                self.join.forward(ctx, pair, x)
+                ctx.stream_left = None
+            ctx.arrived, ctx.stream_left = ctx.stream_left, None
+            ctx.wanted_after = self._reader_after(at, stream)
             block.forward(ctx, x, cache)
             ctx.last_block = block             # (a block may leave something for its successor)
             if self.tap is not None:
@@ -182,6 +217,8 @@ def build_model(config, store, runtime) -> Model:
     embedding = build_part("embedding", config.embedding_spec(), store, runtime)
     final_norm = build_part("norm", config.final_norm_spec(), store, runtime)
     head = build_part("head", config.head_spec(), store, runtime)
+    join_spec = config.stream_join_spec()
+    join = None if join_spec is None else build_part("stream_join", join_spec, store, runtime)
     order = config.run_order()
     for e in order:
         if not (0 <= e.layer < len(blocks)) or e.cache_layer < 0:
@@ -189,4 +226,4 @@ def build_model(config, store, runtime) -> Model:
                              f"the model has {len(blocks)}")
     emb = config.embedding_spec().params
     return Model(config, runtime, embedding, position, blocks, order, final_norm, head,
-                 width=emb["width"], vocab=config.head_spec().params["vocab"])
+                 width=emb["width"], vocab=config.head_spec().params["vocab"], join=join)

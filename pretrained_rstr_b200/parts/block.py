@@ -214,7 +214,69 @@ class BranchNormBlock(Block):
         ctx.stream_copy_by = self
 
 
+class SandwichBlock(Block):
+    """x <- x + m * norm_1b(mixer(norm_1(x))); x <- x + m * norm_2b(feed_forward(norm_2(x))): a norm
+    before and a norm after each branch, and a constant m (``params["residual_mult"]``) on what
+    joins the stream.  A layer without a feed-forward has the first half only.
+
+    A branch's second norm, the sum and the NEXT branch's first norm are one kernel, also across
+    layers: ``ctx.wanted_after`` says what reads the stream next (a norm, or a buffer that takes
+    a copy of it), and what this block leaves for it is ``ctx.stream_left``."""
+    graph_safe = True
+
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Dict[str, Norm],
+                 width: int, runtime, params=None, store=None):
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.norms = dict(norms)
+        self.width, self.runtime = width, runtime
+        self.mult = float((params or {}).get("residual_mult", 1.0))
+        self.has_ff = not getattr(feed_forward, "is_none", False)
+        wanted = {"mixer", "mixer_after"} | ({"feed_forward", "feed_forward_after"} if self.has_ff else set())
+        if set(norms) != wanted:
+            raise ValueError(f"sandwich wants the norms {sorted(wanted)}, got {sorted(norms)}")
+        for part in (mixer, feed_forward):
+            if not getattr(part, "can_overwrite", False):
+                raise ValueError(f"sandwich: {type(part).__name__} cannot hand over its result apart "
+                                 f"from the stream")
+        for name in ("mixer_after", "feed_forward_after"):
+            if name in norms and getattr(norms[name], "pair", lambda: None)() is None:
+                raise ValueError("sandwich needs norms with a weight per coordinate after the branches")
+        #: the norm this block reads the stream through first
+        self.entry_norm = norms["mixer"]
+
+    def forward(self, ctx, x, cache: LayerCache) -> None:
+        t = x.shape[0]
+        cap = ctx.token_capacity
+        y = ctx.scratch("branch_result", (cap, self.width), torch.float32)[:t]
+        h = ctx.scratch("block_normed", (cap, self.width), self.runtime.dtype)[:t]
+        arrived = getattr(ctx, "arrived", None)
+        ready = arrived is not None and arrived[0] is self.entry_norm
+        h_in = arrived[1] if ready else PreNormBlock._normed(ctx, self.mixer, self.entry_norm, x, h)
+        self.mixer.forward(ctx, h_in, y, cache, accumulate=False)
+        after = getattr(ctx, "wanted_after", None)
+        if self.has_ff:
+            norm = self.norms["feed_forward"]
+            ready = self._join(x, y, "mixer_after", norm, h)
+            h_in = h if ready else PreNormBlock._normed(ctx, self.feed_forward, norm, x, h)
+            self.feed_forward.forward(ctx, h_in, y, accumulate=False)
+        if self._join(x, y, "feed_forward_after" if self.has_ff else "mixer_after", after, h):
+            ctx.stream_left = (after, h)
+
+    def _join(self, x, y, name: str, reader, h) -> bool:
+        """x <- x + m * norm(y), and what ``reader`` wants of the new x: a norm's result in ``h``,
+        or a copy in the buffer it is.  True if that has been done."""
+        weight, bias, eps, centred = self.norms[name].pair()
+        if isinstance(reader, torch.Tensor):
+            ops.norm_pair(x, y, self.mult, weight, bias, eps, centred, out=reader)
+            return True
+        following = getattr(reader, "pair", lambda: None)()
+        ops.norm_pair(x, y, self.mult, weight, bias, eps, centred,
+                      out=None if following is None else h, next_norm=following)
+        return following is not None
+
+
 register_part("arrangement", "pre_norm", PreNormBlock)
+register_part("arrangement", "sandwich", SandwichBlock)
 register_part("arrangement", "branch_norm", BranchNormBlock)
 register_part("arrangement", "post_norm_gated", PostNormGatedBlock)
 register_part("arrangement", "parallel", ParallelBlock)

@@ -25,9 +25,12 @@ class TokenEmbedding(Embedding):
 
 class ScaledTokenEmbedding(Embedding):
     """x[t] = table[token[t]] * scale.  ``keeps_copy``: the rows can be left a second time in
-    ``keep`` (for a run order that adds the embedding's output to the stream again)."""
+    ``keep`` (for a run order that adds the embedding's output to the stream again);
+    ``keeps_pair``: and, in the activation type, twice side by side in ``pair`` (for one that joins
+    the stream and the embedding's output in a matrix product)."""
     graph_safe = True
     keeps_copy = True
+    keeps_pair = True
 
     def __init__(self, table: torch.Tensor, vocab: int, width: int, scale: float, runtime):
         if tuple(table.shape) != (vocab, width):
@@ -36,10 +39,11 @@ class ScaledTokenEmbedding(Embedding):
         self.table = table.to(runtime.dtype).contiguous()
         self.vocab, self.width, self.scale = vocab, width, float(scale)
 
-    def forward(self, ctx, position, x, keep=None) -> None:
+    def forward(self, ctx, position, x, keep=None, pair=None) -> None:
         if position.table() is not None:
             raise ValueError("scaled_token_embedding adds no position table")
-        ops.embed_scaled(x, ctx.tokens, self.table, self.scale, keep=keep, status=ctx.status)
+        ops.embed_scaled(x, ctx.tokens, self.table, self.scale, keep=keep, status=ctx.status,
+                         pair=pair)
 
 
 class TokenPairEmbedding(Embedding):

@@ -54,7 +54,8 @@ class NoFeedForward(FeedForward):
 class GatedMLP(FeedForward):
     """down(f(gate(h)) * (up(h) + up_shift)) with f(g) = g * sigmoid(act_alpha * g); with
     ``limit`` > 0 the gate's result is capped at ``limit`` and up's clamped to +-``limit``
-    first.  (act_alpha 1, shift 0, no limit: the usual SiLU-gated feed-forward.)  Gate and up
+    first.  (act_alpha 1, shift 0, no limit: the usual SiLU-gated feed-forward.)  ``activation``
+    "gelu_tanh": f is the tanh form of gelu instead.  Gate and up
     are one matrix product, in which rows of an arrangement may ride along
     (:meth:`fuse_input_rows`); its float32 result feeds the activation unrounded."""
     graph_safe = True
@@ -62,7 +63,7 @@ class GatedMLP(FeedForward):
     accepts_lazy_norm = True      # the first matrix product may compute the norm itself
 
     def __init__(self, gate, up, down, width: int, inner: int, limit: float, act_alpha: float,
-                 up_shift: float, runtime):
+                 up_shift: float, runtime, activation: str = "sigmoid"):
         from .latent_attention import FusedInput
         for name, t, shape in (("gate", gate, (inner, width)), ("up", up, (inner, width)),
                                ("down", down, (width, inner))):
@@ -75,6 +76,9 @@ class GatedMLP(FeedForward):
         self.width, self.inner = width, inner
         self.limit, self.act_alpha, self.up_shift = float(limit), float(act_alpha), float(up_shift)
         self.runtime = runtime
+        if activation not in ops.GATED_ACT_CODES:
+            raise ValueError(f"gated_mlp: unknown activation {activation!r}")
+        self.activation = activation
 
     def fuse_input_rows(self, name: str, weight) -> str:
         return self.input.add(name, weight)
@@ -88,7 +92,7 @@ class GatedMLP(FeedForward):
         cols = self.input.cols
         a = ctx.scratch_zero("gated_act", (ctx.token_capacity, self.down.n_in), self.runtime.dtype)[:t]
         ops.gated_pair(a, proj, cols["gate"][0], cols["up"][0], self.inner, limit=self.limit,
-                       act_alpha=self.act_alpha, up_shift=self.up_shift)
+                       act_alpha=self.act_alpha, up_shift=self.up_shift, act=self.activation)
         self.down.forward(ctx, a, x, resid=x if accumulate else None)
 
 
@@ -246,7 +250,7 @@ def _gated_mlp(p, store, rt) -> GatedMLP:
     w = p["weights"]
     return GatedMLP(store.get(w["gate"]), store.get(w["up"]), store.get(w["down"]), p["width"],
                     p["inner"], p.get("limit", 0.0), p.get("act_alpha", 1.0),
-                    p.get("up_shift", 0.0), rt)
+                    p.get("up_shift", 0.0), rt, p.get("activation", "sigmoid"))
 
 
 register_part("feed_forward", "dense_mlp", _dense_mlp)

@@ -4,6 +4,7 @@ from __future__ import annotations
 
 import torch
 
+from ..csrc import ops
 from .interfaces import Head
 from .linear import Linear
 from .registry import register_part
@@ -23,12 +24,24 @@ class TiedHead(Head):
 
 
 class LinearHead(TiedHead):
-    """A head with a matrix of its own, [vocab, width], no bias."""
+    """A head with a matrix of its own, [vocab, width], no bias.  ``softcap`` > 0: the logits are
+    softcap * tanh(logits / softcap)."""
+
+    def __init__(self, table: torch.Tensor, vocab: int, width: int, runtime, softcap: float = 0.0):
+        super().__init__(table, vocab, width, runtime)
+        self.softcap = float(softcap or 0.0)
+        if self.softcap < 0.0:
+            raise ValueError(f"linear_head: a cap of {self.softcap} on the logits")
+
+    def forward(self, ctx, h, logits) -> None:
+        super().forward(ctx, h, logits)
+        if self.softcap > 0.0:
+            ops.tanh_cap(logits, self.softcap)
 
 
 register_part("head", "linear_head",
               lambda p, store, rt: LinearHead(store.get(p["weights"], rt.dtype), p["vocab"],
-                                              p["width"], rt))
+                                              p["width"], rt, p.get("softcap", 0.0)))
 register_part("head", "tied_head",
               lambda p, store, rt: TiedHead(store.get(p["weights"] + ".weight", rt.dtype),
                                             p["vocab"], p["width"], rt))

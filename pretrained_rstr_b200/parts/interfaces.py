@@ -55,6 +55,18 @@ class Norm:
         raise NotImplementedError
 
 
+class StreamJoin:
+    """Joins the stream with the embedding's output before a run entry that asks for it."""
+
+    def buffer(self, ctx, rows: int) -> torch.Tensor:
+        """[rows, >= 2 width] in the activation type: [stream | embedding's output]."""
+        raise NotImplementedError
+
+    def forward(self, ctx, pair: torch.Tensor, x: torch.Tensor) -> None:
+        """x [rows, width] float32 <- the join of the buffer's two halves."""
+        raise NotImplementedError
+
+
 class Mixer:
     def kv_spec(self) -> Optional[KVSpec]:
         return None

@@ -21,11 +21,20 @@ class LayerNorm(Norm):
         self.eps = float(eps)
         self.size = size
 
+    def pair(self):
+        """(weight, bias, eps, centred): what a kernel that norms on the way needs to know."""
+        return self.gamma, self.beta, self.eps, True
+
     def forward(self, ctx, x, out, rows=None) -> None:
         ops.layernorm(out, x, self.gamma, self.beta, self.eps, rows=rows, status=ctx.status)
 
 
 def _layer_norm(params, store, runtime) -> LayerNorm:
+    """``weights``: a name with ``.weight`` and (unless ``bias`` is False) ``.bias`` behind it; or
+    ``weight`` and ``bias``: the two tensors' full names."""
+    if "weight" in params:
+        beta = store.get(params["bias"]) if params.get("bias") else None
+        return LayerNorm(store.get(params["weight"]), beta, params["eps"], params["size"])
     name = params["weights"]
     beta = store.get(name + ".bias") if params.get("bias", True) else None
     return LayerNorm(store.get(name + ".weight"), beta, params["eps"], params["size"])
@@ -54,6 +63,10 @@ class RMSNorm(Norm):
         self.gamma = self.weight if self.gain is None else None
         self.beta = None
         self.centred = False
+
+    def pair(self):
+        """(weight, None, eps, centred), or None for a norm with one learned number."""
+        return None if self.gamma is None else (self.gamma, None, self.eps, False)
 
     def forward(self, ctx, x, out, rows=None) -> None:
         ops.rms_norm(x, out=out, gain=self.gain, weight=self.weight, rows=rows, eps=self.eps,

@@ -1,9 +1,14 @@
-"""Frequencies of rotary positions in the rotate-half layout: coordinate i < dims / 2 pairs
-with i + dims / 2 and the pair at position p turns by p * base^(-2 i / dims).  The mixers'
-kernels compute the angles in 32-bit from this table and the tokens' positions."""
+"""Frequencies of rotary positions: pair i of dims / 2 at position p turns by p * base^(-2 i /
+dims); pair i is (i, i + dims / 2) in the rotate-half layout and (2i, 2i + 1) in the interleaved
+one.  Kernels compute the angles from these tables and the tokens' positions, or read the
+step's table of cosines and sines (:class:`RotaryAngles`)."""
 from __future__ import annotations
 
+import hashlib
+
 import torch
+
+from ..csrc import ops
 
 
 def rotary_frequencies(base: float, dims: int, device, divide_by: float = 1.0,
@@ -57,3 +62,43 @@ def yarn_frequencies(base: float, dims: int, factor: float, original: float, fas
     if with_lo:
         return split_frequencies(freq, device), 0.1 * math.log(factor) + 1.0
     return table, 0.1 * math.log(factor) + 1.0
+
+
+def banded_frequencies(base: float, dims: int, factor: float, low: float, high: float,
+                       original: float):
+    """Frequencies scaled by their wavelength l = 2 pi / f (Llama 3.1's scaling): f where l <
+    original / high, f / factor where l > original / low, and between the two the blend (1 - s) f /
+    factor + s f with s = (original / l - low) / (high - low).  A list of 64-bit numbers."""
+    import math
+    out = []
+    for i in range(dims // 2):
+        f = float(base) ** (-2.0 * i / dims)
+        wave = 2.0 * math.pi / f
+        if wave < original / high:
+            out.append(f)
+        elif wave > original / low:
+            out.append(f / factor)
+        else:
+            s = (original / wave - low) / (high - low)
+            out.append((1.0 - s) * f / factor + s * f)
+    return out
+
+
+class RotaryAngles:
+    """Cosines and sines of every token's angles, computed once per step and shared by all layers,
+    heads and passes whose frequencies are the same."""
+
+    def __init__(self, freq, freq_lo):
+        self.freq, self.freq_lo = freq, freq_lo
+        mark = hashlib.sha256(freq.cpu().numpy().tobytes() + freq_lo.cpu().numpy().tobytes())
+        self.key = f"rotary_angles_{mark.hexdigest()[:16]}"
+
+    def table(self, ctx, rows: int):
+        """float32 [rows, pairs, 2] of this step."""
+        done = ctx.__dict__.setdefault("rotary_done", {})
+        out = done.get(self.key)
+        if out is None:
+            out = ctx.scratch(self.key, (ctx.token_capacity, self.freq.numel(), 2), torch.float32)[:rows]
+            ops.rotary_angles(out, ctx.positions, self.freq, self.freq_lo)
+            done[self.key] = out
+        return out

@@ -10,6 +10,7 @@ Categories and what a factory returns (interfaces in :mod:`.interfaces`):
 ``position``      :class:`PositionEncoding`  factory(params, store, runtime)
 ``embedding``     :class:`Embedding`    factory(params, store, runtime)
 ``head``          :class:`Head`         factory(params, store, runtime)
+``stream_join``   :class:`StreamJoin`    factory(params, store, runtime)
 ``arrangement``   :class:`Block`        factory(mixer, feed_forward, norms by name, width, runtime);
                                         the block keeps ``mixer``, ``feed_forward`` and ``norms``
 """
@@ -17,7 +18,8 @@ from __future__ import annotations
 
 from typing import Any, Callable, Dict
 
-_CATEGORIES = ("mixer", "feed_forward", "norm", "position", "embedding", "head", "arrangement")
+_CATEGORIES = ("mixer", "feed_forward", "norm", "position", "embedding", "head", "stream_join",
+               "arrangement")
 _PARTS: Dict[str, Dict[str, Callable[..., Any]]] = {c: {} for c in _CATEGORIES}
 
 

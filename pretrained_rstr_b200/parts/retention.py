@@ -12,7 +12,8 @@ and is per-request STATE of the cache manager (a slot per live request), so a pr
 cut anywhere and decoding is the same kernel with one token; long portions are cut into
 segments that run side by side, joined by the states at their starts.  Projections Q, K, V and G are
 one matrix product whose 32-bit result feeds the recurrence unrounded.  Sizes, decays, the
-rotation's base and reach, the key scale and eps are parameters.
+rotation's base and reach, the key scale and eps are parameters; the angles' cosines and sines
+come from a table the step computes once.
 """
 from __future__ import annotations
 
@@ -22,7 +23,7 @@ from ..csrc import ops
 from .interfaces import LayerCache, Mixer, StateSpec
 from .latent_attention import FusedInput
 from .linear import padded_linear
-from .positions_rotary import rotary_frequencies
+from .positions_rotary import RotaryAngles, rotary_frequencies
 from .registry import register_part
 
 
@@ -63,7 +64,9 @@ class Retention(Mixer):
         self.out = padded_linear(need("out", (self.width, self.heads * self.vdim)), runtime)
         dev = runtime.device
         self.decay = torch.tensor(decay, dtype=torch.float64).to(torch.float32).to(dev)
-        self.freq = rotary_frequencies(float(p.get("rot_base", 10000.0)), self.rot_dims, dev)
+        self.freq, lo = rotary_frequencies(float(p.get("rot_base", 10000.0)), self.rot_dims, dev,
+                                           with_lo=True)
+        self.rotary = RotaryAngles(self.freq, lo) if self.rot_dims else None
         self.sm_count = ops.sm_count() if torch.cuda.is_available() else 148
         self.one_launch = torch.cuda.is_available() and ops.retention_step_supports(self.dim, self.vdim)
 
@@ -90,6 +93,7 @@ class Retention(Mixer):
         proj = self._proj = self.input.run(ctx, h)
         cols = self.input.cols
         requests = ctx.layout.b_cap
+        angles = self.rotary.table(ctx, t) if self.rotary else None
         gated = ctx.scratch_zero("retention_gated", (cap, self.out.n_in), self.runtime.dtype)[:t]
         if ctx.layout.t_cap <= ops.retention_segment() and self.one_launch:
             # a step of few tokens: rotation, recurrence and finish in one launch
@@ -97,7 +101,7 @@ class Retention(Mixer):
                                cols["gate"][0] if self.gated else -1, cache.state["retention"],
                                ctx.q_start, ctx.state_slot, ctx.positions, self.decay, self.freq,
                                requests, self.heads, self.dim, self.vdim, self.rot_dims,
-                               self.k_scale, self.eps, ctx.status)
+                               self.k_scale, self.eps, ctx.status, angles=angles)
             self.out.forward(ctx, gated, x, resid=x if accumulate else None)
             return
         raw = ctx.scratch("retention_raw", (cap, self.heads * self.vdim), torch.float32)[:t]
@@ -115,7 +119,7 @@ class Retention(Mixer):
                            cache.state["retention"], ctx.q_start, ctx.state_slot, ctx.positions,
                            self.decay, self.freq, requests, self.heads, self.dim, self.vdim,
                            self.rot_dims, self.k_scale, self._columns_per_cta(lists), ctx.status,
-                           segments=segments)
+                           segments=segments, angles=angles)
         ops.retention_finish(gated, raw, proj if self.gated else None,
                              cols["gate"][0] if self.gated else 0, ctx.seq_of_token, self.heads,
                              self.vdim, self.eps)
