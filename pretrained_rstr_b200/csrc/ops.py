@@ -202,6 +202,11 @@ def _declare(h: ctypes.CDLL) -> None:
                                     I, I, I, P, P, P]
     h.prb_wattn.argtypes = [P, L, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, I, I, F, F, I, I,
                             P, I, F, P, P]
+    h.prb_wattn_bf16_supports.argtypes = [I, I, I, I]
+    h.prb_wattn_bf16_supports.restype = c_int
+    h.prb_wattn_bf16.argtypes = [P, L, P, P, P, P, P, P, L, P, I, I, I, I, I, I, I, I, I, I, I, F, F,
+                                 P, I, F, P, P]
+    h.prb_wattn_bf16.restype = c_int
     h.prb_wattn_tile_rows.argtypes = [I, I, I, I]
     h.prb_wattn_single_supports.argtypes = [I, I, I, I]
     h.prb_wattn_single.argtypes = list(h.prb_wattn.argtypes)
@@ -1871,10 +1876,18 @@ def wattn_single_supports(heads: int, kv_heads: int, dim: int, vdim: int) -> boo
     return bool(lib().prb_wattn_single_supports(heads, kv_heads, dim, vdim))
 
 
+def wattn_bf16_supports(heads: int, kv_heads: int, dim: int, vdim: int):
+    """(whether the tensor-core kernel for portions, whether the single-token kernel for
+    bfloat16 cache rows takes these sizes)."""
+    bits = int(lib().prb_wattn_bf16_supports(heads, kv_heads, dim, vdim))
+    return bool(bits & 1), bool(bits & 2)
+
+
 def wattn(out, q, cache, block_table, seq_of_token, positions, heads: int, dim: int, vdim: int,
           window: int, keep_first: int, scale: float, gate=None, slopes=None,
           out_scale: float = 1.0, status=None, tile_rows: int = 0, single: bool = False,
-          sinks=None, gate_per_value: bool = False, softcap: float = 0.0) -> None:
+          sinks=None, gate_per_value: bool = False, softcap: float = 0.0,
+          bf16_kernels: bool = False) -> None:
     """Softmax attention over cache rows [k | v]: a query at position i sees key j <= i with
     i - j < window (``window`` 0: all) or j < keep_first; score (q . k) * scale - slopes[h] * (i
     - j), with ``softcap`` > 0 softcap * tanh((q . k) * scale / softcap) in the place of the
@@ -1884,7 +1897,10 @@ def wattn(out, q, cache, block_table, seq_of_token, positions, heads: int, dim: 
     ``out_scale``.  32-bit arithmetic; out in the cache's type.  ``tile_rows`` > 0: the
     tiled kernel (a CTA per that many consecutive token rows and key/value head).  ``single``:
     the kernel for steps of single tokens (a CTA per (token, key/value head) whose warps share
-    out the key blocks; sizes that :func:`wattn_single_supports` takes)."""
+    out the key blocks; sizes that :func:`wattn_single_supports` takes).  ``bf16_kernels``: the
+    kernels for bfloat16 cache rows instead (sizes that :func:`wattn_bf16_supports` takes):
+    products on tensor cores with 32-bit operands as pairs of bfloat16 numbers, everything
+    else in 32-bit."""
     what = "wattn"
     _need(q, torch.float32, "q", what)
     _need(cache, None, "cache", what)
@@ -1918,6 +1934,13 @@ def wattn(out, q, cache, block_table, seq_of_token, positions, heads: int, dim: 
     common = (_p(out), out.stride(0), _p(q), _p(cache), _p(block_table), _p(seq_of_token),
               _p(positions), _p(gate), gate_ld, _p(slopes), n, heads, kv_heads, dim, vdim,
               page_size, block_table.shape[1], pages, int(window or 0), int(keep_first or 0))
+    if bf16_kernels:
+        if cache.dtype != torch.bfloat16:
+            raise KernelArgumentError(f"{what}: bf16_kernels read a bfloat16 cache")
+        _check(lib().prb_wattn_bf16(*common, int(bool(single)), float(scale), float(out_scale),
+                                    _p(sinks), gate_per, float(softcap or 0.0), _p(status),
+                                    _stream()), what)
+        return
     tail = (float(scale), float(out_scale), dtype_code(cache.dtype), dtype_code(out.dtype),
             _p(sinks), gate_per, float(softcap or 0.0), _p(status), _stream())
     if single:

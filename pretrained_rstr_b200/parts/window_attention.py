@@ -161,6 +161,9 @@ class WindowAttention(Mixer):
         self.rotary = RotaryAngles(self.freq, self.freq_lo) \
             if self.rot_dims and mode not in (True, "whole") else None
         gpu = torch.cuda.is_available()
+        # kernels for bfloat16 cache rows: (portions, single tokens)
+        self.bf16_ok = ops.wattn_bf16_supports(self.heads, self.kv_heads, self.dim, self.vdim) \
+            if gpu and runtime.dtype == torch.bfloat16 else (False, False)
         self.tile_rows = ops.wattn_tile_rows(self.heads, self.kv_heads, self.dim, self.vdim) if gpu else 0
         self.single_ok = gpu and ops.wattn_single_supports(self.heads, self.kv_heads, self.dim, self.vdim)
 
@@ -219,7 +222,8 @@ class WindowAttention(Mixer):
         o = ctx.scratch_zero("wattn_out", (cap, self.out.n_in), self.runtime.dtype)[:t]
         # a step of single tokens: a CTA per (token, key/value head) whose warps share out the
         # key blocks (rows of different requests share no keys); sizes that kernel does not
-        # take: the tiled kernel, a row a CTA
+        # take: the tiled kernel, a row a CTA.  Serving in bfloat16 has kernels of its own for
+        # both kinds of step
         single = ctx.max_q_len == 1 or ctx.layout.t_cap <= ctx.layout.b_cap
         ops.wattn(o, q, cache.k, group.block_table, ctx.seq_of_token, ctx.positions, self.heads,
                   self.dim, self.vdim, self.window, self.keep_first, self.scale,
@@ -227,7 +231,8 @@ class WindowAttention(Mixer):
                   out_scale=self.out_scale, status=ctx.status,
                   tile_rows=min(self.tile_rows, 1) if single else self.tile_rows,
                   single=single and self.single_ok, sinks=self.sinks,
-                  gate_per_value=self.value_gate, softcap=self.softcap)
+                  gate_per_value=self.value_gate, softcap=self.softcap,
+                  bf16_kernels=self.bf16_ok[1 if single else 0])
         self.out.forward(ctx, o, x, resid=x if accumulate else None)
 
 
