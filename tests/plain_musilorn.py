@@ -133,9 +133,15 @@ def capped_sink_attention(q, k, v, scale: float, cap: Optional[float], sink: boo
     return out
 
 
-def attention_mixer(W, p: str, mx: dict, h: torch.Tensor, positions, eps: float) -> torch.Tensor:
+def _exact(v: torch.Tensor) -> torch.Tensor:
+    return v
+
+
+def attention_mixer(W, p: str, mx: dict, h: torch.Tensor, positions, eps: float,
+                    r=_exact) -> torch.Tensor:
     """Queries and keys behind a short convolution; the convolved keys are the values; then a
-    norm per head with a shared weight, the rotation of interleaved pairs, the attention."""
+    norm per head with a shared weight, the rotation of interleaved pairs, the attention.  ``r``:
+    a rounding of what is cached and of what the output product reads."""
     T = h.shape[0]
     H, G, D = mx["heads"], mx["kv_heads"], mx["dim"]
     q = causal_convolution(h @ W[p + "q"].T, W[p + "q.conv"]).reshape(T, H, D)
@@ -148,8 +154,8 @@ def attention_mixer(W, p: str, mx: dict, h: torch.Tensor, positions, eps: float)
     if sc:
         freqs = banded_frequencies(freqs, sc["factor"], sc["low"], sc["high"], sc["original"])
     q, k = turn(q, positions, freqs, "interleaved"), turn(k, positions, freqs, "interleaved")
-    o = capped_sink_attention(q, k, v, mx["scale"], mx.get("softcap"))
-    return o.reshape(T, H * D) @ W[p + "o"].T
+    o = capped_sink_attention(q, r(k), r(v), mx["scale"], mx.get("softcap"))
+    return r(o.reshape(T, H * D)) @ W[p + "o"].T
 
 
 # ------------------------------------------------------------------------------ retention
@@ -165,7 +171,7 @@ def retention_outputs(q, k, v, decay: List[float]) -> torch.Tensor:
     return out
 
 
-def retention_mixer(W, p: str, mx: dict, h, positions, eps: float) -> torch.Tensor:
+def retention_mixer(W, p: str, mx: dict, h, positions, eps: float, r=_exact) -> torch.Tensor:
     T = h.shape[0]
     H, D, V = mx["heads"], mx["dim"], mx["vdim"]
     q, k = (h @ W[p + "q"].T).reshape(T, H, D), (h @ W[p + "k"].T).reshape(T, H, D)
@@ -174,7 +180,7 @@ def retention_mixer(W, p: str, mx: dict, h, positions, eps: float) -> torch.Tens
     q = turn(q, positions, freqs, "half")
     k = turn(k, positions, freqs, "half") * D ** -0.5
     o = unit_rms(retention_outputs(q, k, v, mx["decay"]), eps).reshape(T, H * V)
-    return (o * torch.nn.functional.silu(h @ W[p + "g"].T)) @ W[p + "o"].T
+    return r(o * torch.nn.functional.silu(h @ W[p + "g"].T)) @ W[p + "o"].T
 
 
 # ------------------------------------------------------------------------------- the rest
@@ -182,8 +188,8 @@ def tanh_gelu(z: torch.Tensor) -> torch.Tensor:
     return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z.pow(3))))
 
 
-def gated_unit(W, p: str, h) -> torch.Tensor:
-    return (tanh_gelu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+def gated_unit(W, p: str, h, r=_exact) -> torch.Tensor:
+    return r(tanh_gelu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
 def run_list(cfg: dict):
@@ -205,11 +211,11 @@ def _bf16(x: torch.Tensor) -> torch.Tensor:
 def forward(tokens: List[int], W: Dict[str, torch.Tensor], cfg: dict,
             taps: Optional[list] = None, rounded: bool = False) -> torch.Tensor:
     """Logits [T, vocab] of one sequence; ``taps`` collects the stream after every layer run.
-    ``rounded``: every product that reads the stream (a sublayer's norm of it, or the stream
-    itself where a pass begins) reads it rounded to bfloat16, what serving in bfloat16 does at
-    the least; the difference to the exact run says how far rounding alone moves a row."""
+    ``rounded``: what the matrix products read (norms of the stream, the stream where a pass
+    begins, mixers' results, activations) and what is cached is rounded to bfloat16, as serving in
+    bfloat16 does; the difference to the exact run says how far rounding alone moves a row."""
     eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
-    r = _bf16 if rounded else (lambda v: v)
+    r = _bf16 if rounded else _exact
     norm = lambda v, name: centred_norm(v, W[name], W[name + ".b"], eps)
     positions = torch.arange(len(tokens))
     x0 = W["embed"][tokens]
@@ -219,10 +225,10 @@ def forward(tokens: List[int], W: Dict[str, torch.Tensor], cfg: dict,
             x = r(torch.cat([x, x0], dim=-1)) @ W["loop.in"].T
         layer, p = cfg["layers"][i], f"l{i}."
         mixer = attention_mixer if layer["type"] == "attention" else retention_mixer
-        y = mixer(W, p + "mix.", layer["mixer"], r(norm(x, p + "norm1")), positions, eps)
+        y = mixer(W, p + "mix.", layer["mixer"], r(norm(x, p + "norm1")), positions, eps, r)
         x = x + m * norm(y, p + "norm1b")
         if layer.get("mlp"):
-            x = x + m * norm(gated_unit(W, p + "mlp.", r(norm(x, p + "norm2"))), p + "norm2b")
+            x = x + m * norm(gated_unit(W, p + "mlp.", r(norm(x, p + "norm2")), r), p + "norm2b")
         if taps is not None:
             taps.append(x.clone())
     logits = r(norm(x, "final.norm")) @ W["head"].T

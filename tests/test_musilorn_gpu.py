@@ -1,0 +1,770 @@
+"""Musilorn in the engine against the plain implementation (``plain_musilorn``): every mechanism
+alone at the kernels' interface, then whole models of several shapes under every way of
+cutting and batching the work, in 32-bit and in bfloat16, and greedy generation through the
+package's entry point."""
+import math
+import os
+import random
+import shutil
+
+import pytest
+import torch
+
+import plain_musilorn as P
+from helpers import Replayer, random_tokens
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda:0"
+
+
+def _i32(v):
+    return torch.tensor(v, dtype=torch.int32, device=DEV)
+
+
+def _steps(parts):
+    """positions, request of each token, row offsets and slots of a step made of
+    (slot, first position, tokens) parts, with one padding request behind them."""
+    pos, seq, qs, slots = [], [], [0], []
+    for b, (slot, p0, n) in enumerate(parts):
+        pos += list(range(p0, p0 + n))
+        seq += [b] * n
+        qs.append(qs[-1] + n)
+        slots.append(slot)
+    return _i32(pos), _i32(seq), _i32(qs + [qs[-1]]), _i32(slots + [-1])
+
+
+# ------------------------------------------------------------------ mechanisms, one by one
+@pytest.mark.parametrize("width,rows,dtype", [(72, 5, "float32"), (768, 3, "bfloat16"), (1600, 20, "bfloat16"),
+                                              (5000, 2, "float32"), (33, 1, "bfloat16")])
+def test_norm_sum_and_next_norm_kernel(width, rows, dtype):
+    """x + m norm(y) in place, with the next norm of the sum, a copy of it into a wider buffer, or
+    nothing behind it; layer norms with a bias, and root-mean-square ones."""
+    from pretrained_rstr_b200.csrc import ops
+    g = torch.Generator().manual_seed(width)
+    rn = lambda *s: torch.randn(*s, generator=g)
+    dt = getattr(torch, dtype)
+    tol = dict(atol=2e-5, rtol=2e-5) if dtype == "float32" else dict(atol=2e-2, rtol=1e-2)
+    for centred, centred2, eps in ((True, True, 1e-5), (False, True, 0.3), (True, False, 1e-2)):
+        x, y = rn(rows, width) * 3 + 1, rn(rows, width) * 0.2 + 5.0          # (a mean far from zero)
+        w1, b1, w2, b2 = rn(width), rn(width), rn(width), rn(width)
+        norm = lambda v, w, b, c: P.centred_norm(v.double(), w.double(), b.double(), eps) if c else \
+            P.unit_rms(v.double(), eps) * w.double()
+        want = x.double() + 0.7 * norm(y, w1, b1, centred)
+        dev = lambda t: t.to(DEV).contiguous()
+        bias = lambda b, c: dev(b) if c else None
+        for mode in ("norm", "copy", "none"):
+            xd = dev(x)
+            out = torch.full((rows, width + 8), 9.0, dtype=dt, device=DEV)
+            nxt = (dev(w2), bias(b2, centred2), eps, centred2) if mode == "norm" else None
+            ops.norm_pair(xd, dev(y), 0.7, dev(w1), bias(b1, centred), eps, centred,
+                          out=None if mode == "none" else out, next_norm=nxt)
+            assert torch.allclose(xd.cpu().double(), want, atol=2e-5, rtol=2e-5)
+            got = out.cpu().double()
+            assert bool((got[:, width:] == 9.0).all())
+            if mode == "norm":
+                assert torch.allclose(got[:, :width], norm(want, w2, b2, centred2), **tol)
+            elif mode == "copy":
+                assert torch.allclose(got[:, :width], want, **tol)
+
+
+def test_gated_gelu_cap_and_paired_embedding_kernels():
+    from pretrained_rstr_b200.csrc import ops
+    g = torch.Generator().manual_seed(1)
+    for n in (24, 30):                                   # four columns a thread, and one
+        inp = torch.randn(7, 2 * n + 8, generator=g) * 3
+        out = torch.zeros(7, n + 2 if n % 4 else n, device=DEV)
+        ops.gated_pair(out, inp.to(DEV), 0, n + 8, n, act="gelu_tanh")
+        want = P.tanh_gelu(inp[:, :n].double()) * inp[:, n + 8:].double()
+        assert torch.allclose(out[:, :n].cpu().double(), want, atol=1e-5, rtol=1e-5)
+    z = torch.randn(5, 96, generator=g) * 20
+    zd = z.to(DEV)
+    ops.tanh_cap(zd[:, :67], 4.5)
+    assert torch.allclose(zd[:, :67].cpu().double(), 4.5 * torch.tanh(z[:, :67].double() / 4.5), atol=1e-5)
+    assert torch.equal(zd[:, 67:].cpu(), z[:, 67:])
+    table = torch.randn(11, 40, generator=g).to(torch.bfloat16)
+    x = torch.empty(4, 40, device=DEV)
+    pair = torch.zeros(4, 88, dtype=torch.bfloat16, device=DEV)
+    ops.embed_scaled(x, _i32([3, 0, 10, 3]), table.to(DEV), 1.0, pair=pair)
+    rows = table[[3, 0, 10, 3]]
+    assert torch.equal(x.cpu(), rows.float())
+    assert torch.equal(pair[:, :40].cpu(), rows) and torch.equal(pair[:, 40:80].cpu(), rows)
+    assert not bool(pair[:, 80:].any())
+
+
+def test_rotary_angle_table():
+    """Far positions keep the angle's precision (a 32-bit product at 30,000 is off by 1e-3)."""
+    from pretrained_rstr_b200.csrc import ops
+    from pretrained_rstr_b200.parts.positions_rotary import split_frequencies
+    freqs = P.plain_frequencies(250.0, 10)
+    hi, lo = split_frequencies(freqs, DEV)
+    pos = [0, 1, 77, 4095, 30001]
+    out = torch.zeros(5, 5, 2, device=DEV)
+    ops.rotary_angles(out, _i32(pos), hi, lo)
+    angle = torch.tensor(pos, dtype=torch.float64)[:, None] * torch.tensor(freqs, dtype=torch.float64)
+    assert torch.allclose(out[..., 0].cpu().double(), torch.cos(angle), atol=2e-7)
+    assert torch.allclose(out[..., 1].cpu().double(), torch.sin(angle), atol=2e-7)
+
+
+class PrepareCase:
+    """What acts on queries and keys before they are attended to, behind a stand-in for the
+    projections' buffer: convolution, keys as values, norms per head, rotation."""
+
+    def __init__(self, heads, kv_heads, dim, taps, rot_dims, layout, seed):
+        self.heads, self.kv, self.dim, self.taps = heads, kv_heads, dim, taps
+        self.rot, self.layout = rot_dims, layout
+        g = torch.Generator().manual_seed(seed)
+        self.rn = lambda *s: torch.randn(*s, generator=g)
+        self.wq, self.wk = self.rn(heads * dim, taps), self.rn(kv_heads * dim, taps)
+        self.nq, self.nk = 1.0 + 0.3 * self.rn(dim), 1.0 + 0.3 * self.rn(dim)
+        self.freqs = P.plain_frequencies(300.0, rot_dims)
+        self.state = torch.full((3, taps - 1, (heads + kv_heads) * dim), 9.0, device=DEV)
+        self.page_size, pages = 16, 40
+        self.cache = torch.full((pages, kv_heads, 16, 2 * dim), 5.0, device=DEV)
+        self.eps = 1e-5
+
+    def plain(self, q, k):
+        T = q.shape[0]
+        q = P.causal_convolution(q.double(), self.wq.double()).reshape(T, self.heads, self.dim)
+        k = P.causal_convolution(k.double(), self.wk.double()).reshape(T, self.kv, self.dim)
+        v, pos = k, torch.arange(T)
+        q = P.turn(P.unit_rms(q, self.eps) * self.nq.double(), pos, self.freqs, self.layout)
+        k = P.turn(P.unit_rms(k, self.eps) * self.nk.double(), pos, self.freqs, self.layout)
+        return q, torch.cat([k, v], dim=-1)
+
+    def run(self, parts, table=True):
+        """parts: (slot, page of its first position, first position, q, k) per request."""
+        from pretrained_rstr_b200.csrc import ops
+        from pretrained_rstr_b200.parts.positions_rotary import split_frequencies
+        n = [p[3].shape[0] for p in parts]
+        proj = torch.cat([torch.cat([torch.zeros(m, 8), q, torch.zeros(m, 4), k], dim=1)
+                          for m, (_, _, _, q, k) in zip(n, parts)] + [torch.full((1, 12 + (self.heads + self.kv) * self.dim), 3.0)])
+        pos, seq, qs, slots = _steps([(p[0], p[2], m) for p, m in zip(parts, n)])
+        pad = lambda t, v: torch.cat([t, _i32([v])])                  # (a padding row behind them)
+        where = [page * self.page_size + p0 + i for (_, page, p0, _, _), m in zip(parts, n) for i in range(m)]
+        t = sum(n) + 1
+        q_out = torch.zeros(t, self.heads * self.dim, device=DEV)
+        hi, lo = split_frequencies(self.freqs or [0.0], DEV)
+        pos, seq = pad(pos, 0), pad(seq, -1)
+        angles = None
+        if table and self.rot:
+            angles = torch.zeros(t, self.rot // 2, 2, device=DEV)
+            ops.rotary_angles(angles, pos, hi, lo)
+        dev = lambda x: x.to(DEV).contiguous()
+        ops.wattn_prepare(q_out, self.cache, proj.to(DEV).contiguous(), 8, 12 + self.heads * self.dim, 0,
+                          dev(self.nq), dev(self.nk), _i32(where + [-1]), pos, hi, self.heads, self.kv,
+                          self.dim, self.dim, self.rot, self.eps, 0.0, 0, head_norm="before", freq_lo=lo,
+                          angles=angles, interleaved=self.layout == "interleaved", keys_are_values=True,
+                          conv=(dev(self.wq), dev(self.wk), self.state, seq, qs, slots,
+                                0 if max(n) == 1 else len(parts) + 1))
+        return q_out[:-1].cpu().double().reshape(t - 1, self.heads, self.dim)
+
+    def rows(self, page, p0, n):
+        flat = [page * self.page_size + p0 + i for i in range(n)]
+        return torch.stack([self.cache[s // 16, :, s % 16].cpu().double() for s in flat])
+
+
+@pytest.mark.parametrize("heads,kv,dim,taps,rot,layout", [
+    (4, 2, 16, 3, 16, "interleaved"), (3, 3, 40, 4, 12, "interleaved"), (2, 1, 64, 1, 64, "half"),
+    (6, 2, 10, 2, 0, "half"), (1, 1, 130, 6, 2, "interleaved")])
+def test_convolution_norm_and_rotation(heads, kv, dim, taps, rot, layout):
+    """A sequence whole, then in portions down to one token (the taps cross every cut) beside
+    another request; a slot's earlier inputs are not read at position 0 and are carried from
+    then on, by portions and by single tokens alike."""
+    c = PrepareCase(heads, kv, dim, taps, rot, layout, seed=dim + taps)
+    n = 90
+    q, k, q2, k2 = c.rn(n, heads * dim), c.rn(n, kv * dim), c.rn(31, heads * dim), c.rn(31, kv * dim)
+    (want_q, want_r), (want_q2, want_r2) = c.plain(q, k), c.plain(q2, k2)
+    tol = dict(atol=3e-5, rtol=3e-5)
+    assert torch.allclose(c.run([(1, 0, 0, q, k)]), want_q, **tol)
+    assert torch.allclose(c.rows(0, 0, n), want_r, **tol)
+    c.cache.fill_(5.0)
+    cuts = [1, 2, 1, 1, 5, 2, 1, 1, 1, 17, 2, 3, 1, 20, 1, 1]
+    at, i, other = 0, 0, 0
+    while at < n:
+        m = min(cuts[i % len(cuts)], n - at)
+        i += 1
+        parts, mo = [(2, 10, at, q[at:at + m], k[at:at + m])], 0
+        if other < 31 and i % 3:                          # another request rides along
+            mo = min(1 if m == 1 else 4, 31 - other)
+            parts.insert(0, (0, 20, other, q2[other:other + mo], k2[other:other + mo]))
+        got = c.run(parts, table=bool(i % 2))
+        assert torch.allclose(got[:mo], want_q2[other:other + mo], **tol)
+        assert torch.allclose(got[mo:], want_q[at:at + m], **tol)
+        other += mo
+        at += m
+    assert torch.allclose(c.rows(10, 0, n), want_r, **tol)
+    assert torch.allclose(c.rows(20, 0, other), want_r2[:other], **tol)
+
+
+class AttentionCase:
+    """Cache rows [k | v] of several requests in shuffled pages."""
+
+    def __init__(self, heads, kv_heads, dim, vdim, lengths, page_size, dtype, seed):
+        self.heads, self.kv, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        g = torch.Generator().manual_seed(seed)
+        self.rn = lambda *s: torch.randn(*s, generator=g)
+        most = -(-max(lengths) // page_size)
+        order = list(range(len(lengths) * most))
+        random.Random(seed).shuffle(order)
+        self.cache = torch.full((len(order), kv_heads, page_size, dim + vdim), 50.0)   # what others left
+        self.k = [self.rn(n, kv_heads, dim) for n in lengths]
+        self.v = [self.rn(n, kv_heads, vdim) for n in lengths]
+        self.q = [self.rn(n, heads, dim) for n in lengths]
+        self.table = [[order.pop() if i * page_size < n else -1 for i in range(most)] for n in lengths]
+        self.page_size, self.dtype = page_size, getattr(torch, dtype)
+
+    def stand_out(self, b, at, query, size):
+        """Key ``at`` of request b points where query ``query`` looks (for every head of its
+        group): one score far above the others."""
+        per = self.heads // self.kv
+        for g in range(self.kv):
+            d = self.q[b][query, g * per] / self.q[b][query, g * per].norm()
+            self.k[b][at, g] = d * size
+            for h in range(g * per, (g + 1) * per):
+                self.q[b][query, h] = d * math.sqrt(self.dim)
+
+    def finish(self):
+        for b, pages in enumerate(self.table):
+            for i in range(self.k[b].shape[0]):
+                row = torch.cat([self.k[b][i], self.v[b][i]], dim=-1)
+                self.cache[pages[i // self.page_size], :, i % self.page_size] = row
+        self.dev = self.cache.to(self.dtype).to(DEV)
+        # (the oracle sees the numbers the cache holds)
+        self.k = [k.to(self.dtype).double() for k in self.k]
+        self.v = [v.to(self.dtype).double() for v in self.v]
+
+    def run(self, rows, scale, cap, sink, **kw):
+        """rows: (request, position); a padding row lies behind them."""
+        from pretrained_rstr_b200.csrc import ops
+        q = torch.stack([self.q[b][i] for b, i in rows] + [self.q[0][0]]).reshape(len(rows) + 1, -1).to(DEV)
+        out = torch.full((len(rows) + 1, self.heads * self.vdim + 8), 3.0, dtype=self.dtype, device=DEV)
+        status = torch.zeros(4, dtype=torch.int32, device=DEV)
+        ops.wattn(out, q, self.dev, _i32(self.table), _i32([b for b, _ in rows] + [-1]),
+                  _i32([i for _, i in rows] + [0]), self.heads, self.dim, self.vdim, 0, 0, scale,
+                  sinks=torch.zeros(self.heads, device=DEV) if sink else None, softcap=cap or 0.0,
+                  status=status, **kw)
+        assert status.tolist() == [0, 0, 0, 0]
+        assert not bool(out[-1, :self.heads * self.vdim].any()) and bool((out[:, self.heads * self.vdim:] == 3.0).all())
+        return out[:-1, :self.heads * self.vdim].cpu().double().reshape(len(rows), self.heads, self.vdim)
+
+    def plain(self, rows, scale, cap, sink):
+        full = [P.capped_sink_attention(q.double(), k, v, scale, cap, sink)
+                for q, k, v in zip(self.q, self.k, self.v)]
+        return torch.stack([full[b][i] for b, i in rows])
+
+
+def _ways(heads, kv, dim, vdim, dtype):
+    """(keyword arguments of ``ops.wattn``, single tokens only?) of every kernel that takes the sizes."""
+    from pretrained_rstr_b200.csrc import ops
+    ways = [({}, False)]
+    tile = ops.wattn_tile_rows(heads, kv, dim, vdim)
+    ways += [({"tile_rows": n}, False) for n in {1, tile} if tile > 0]
+    if ops.wattn_single_supports(heads, kv, dim, vdim):
+        ways.append(({"single": True}, True))
+    if dtype == "bfloat16":
+        tiles, single = ops.wattn_bf16_supports(heads, kv, dim, vdim)
+        ways += [({"bf16_kernels": True}, False)] if tiles else []
+        ways += [({"bf16_kernels": True, "single": True}, True)] if single else []
+    return ways
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("heads,kv,dim,vdim,page", [
+    (4, 2, 16, 16, 16), (6, 6, 40, 40, 64), (12, 4, 64, 64, 64), (5, 1, 128, 96, 32), (8, 1, 72, 120, 16),
+    (10, 2, 96, 32, 64), (3, 1, 34, 34, 64), (12, 2, 128, 128, 64)])
+def test_capped_attention_with_a_unit_in_the_denominator(heads, kv, dim, vdim, page, dtype):
+    """Portions and single tokens of unequal requests, by every kernel: rows at page and block
+    borders, a key far away and one on a page's border whose scores stand out, first tokens
+    (where the added 1 counts most), with and without a cap and the added 1."""
+    lengths = [1, 66, 333, 140]
+    c = AttentionCase(heads, kv, dim, vdim, lengths, page, dtype, seed=dim + heads)
+    c.stand_out(2, 3, 332, 4.0)
+    c.stand_out(2, 64, 331, 4.0)
+    c.stand_out(3, 63, 128, 4.0)
+    c.finish()
+    scale = 1.7 / math.sqrt(dim)
+    portions = [(0, 0)] + [(1, i) for i in range(66)] + [(2, i) for i in range(300, 333)] + \
+        [(3, i) for i in range(62, 131)]
+    singles = [(0, 0), (1, 1), (1, 31), (1, 63), (1, 64), (2, 332), (2, 331), (3, 31), (3, 127), (3, 128), (3, 139)]
+    tol = dict(atol=2e-5, rtol=2e-5) if dtype == "float32" else dict(atol=4e-3, rtol=8e-3)
+    for cap, sink in ((2.5, True), (None, True), (30.0, False)):
+        for kw, only_single in _ways(heads, kv, dim, vdim, dtype):
+            for rows in ([singles] if only_single else [portions, singles]):
+                got, want = c.run(rows, scale, cap, sink, **kw), c.plain(rows, scale, cap, sink)
+                worst = float((got - want).abs().max())
+                assert torch.allclose(got, want, **tol), (kw, cap, sink, worst)
+    # the added 1 and the cap both show
+    assert float((c.plain([(1, 1)], scale, 2.5, True) - c.plain([(1, 1)], scale, 2.5, False)).abs().max()) > 0.05
+    assert float((c.plain([(2, 332)], scale, 2.5, True) - c.plain([(2, 332)], scale, None, True)).abs().max()) > 0.05
+
+
+def test_a_row_does_not_depend_on_its_batch_or_cut():
+    """A query's result from the tensor-core kernel is the same bits in a tile with others, alone,
+    and whatever else is in the step; likewise the single-token kernel beside other tokens."""
+    c = AttentionCase(6, 2, 64, 64, [200, 90], 64, "bfloat16", seed=3)
+    c.finish()
+    whole = c.run([(0, i) for i in range(200)], 0.125, 20.0, True, bf16_kernels=True)
+    part = c.run([(1, i) for i in range(7, 40)] + [(0, i) for i in range(101, 144)], 0.125, 20.0, True, bf16_kernels=True)
+    assert torch.equal(part[33:], whole[101:144])
+    alone = c.run([(0, 130)], 0.125, 20.0, True, bf16_kernels=True)
+    assert torch.equal(alone[0], whole[130])
+    many = c.run([(1, i) for i in range(90)] + [(0, 199)] + [(1, i) for i in range(90)], 0.125, 20.0, True,
+                 bf16_kernels=True, single=True)
+    one = c.run([(0, 199)], 0.125, 20.0, True, bf16_kernels=True, single=True)
+    assert torch.allclose(many[90], one[0], atol=4e-3) and torch.allclose(one[0], whole[199], atol=4e-3)
+
+
+class RetentionCase:
+    """Retention behind a stand-in for the projections' buffer, angles from the step's table."""
+
+    def __init__(self, heads, dim, vdim, rot, decay, seed):
+        self.heads, self.dim, self.vdim, self.rot, self.decay = heads, dim, vdim, rot, decay
+        g = torch.Generator().manual_seed(seed)
+        self.rn = lambda *s: torch.randn(*s, generator=g)
+        self.freqs = P.plain_frequencies(500.0, rot)
+        self.state = torch.full((3, heads, vdim, dim), 9.0, device=DEV)
+        self.eps = 1e-5
+
+    def rows(self, n):
+        h = self.heads
+        return [self.rn(n, h, self.dim), self.rn(n, h, self.dim), self.rn(n, h, self.vdim), self.rn(n, h, self.vdim)]
+
+    def plain(self, q, k, v, g):
+        pos = torch.arange(q.shape[0])
+        q, k = (P.turn(t.double(), pos, self.freqs, "half") for t in (q, k))
+        o = P.retention_outputs(q, k * self.dim ** -0.5, v.double(), self.decay)
+        return P.unit_rms(o, self.eps) * torch.nn.functional.silu(g.double())
+
+    def run(self, parts, mode):
+        """parts: (slot, first position, q, k, v, gate) per request; ``mode``: "step" (one launch),
+        "scan" (a CTA walks a request's portion) or "segments"."""
+        from pretrained_rstr_b200.csrc import ops
+        from pretrained_rstr_b200.parts.positions_rotary import split_frequencies
+        h, d, vd = self.heads, self.dim, self.vdim
+        proj = torch.cat([torch.cat([x.reshape(x.shape[0], -1) for x in p[2:]], dim=1) for p in parts])
+        proj = torch.nn.functional.pad(proj, (0, -proj.shape[1] % 4)).to(DEV).contiguous()
+        pos, seq, qs, slots = _steps([(p[0], p[1], p[2].shape[0]) for p in parts])
+        t = proj.shape[0]
+        hi, lo = split_frequencies(self.freqs or [0.0], DEV)
+        angles = None
+        if self.rot:
+            angles = torch.zeros(t, self.rot // 2, 2, device=DEV)
+            ops.rotary_angles(angles, pos, hi, lo)
+        decay = torch.tensor(self.decay, device=DEV)
+        cols = (0, h * d, 2 * h * d, 2 * h * d + h * vd)
+        out = torch.zeros(t, h * vd + 8, device=DEV)
+        if mode == "step":
+            ops.retention_step(out, proj, *cols, self.state, qs, slots, pos, decay, hi, len(parts) + 1, h, d, vd,
+                               self.rot, d ** -0.5, self.eps, angles=angles)
+        else:
+            segments = None
+            if mode == "segments":
+                n = ops.retention_max_segments(t, len(parts) + 1) + 1
+                segments = tuple(torch.full((n, h, vd, d), 3.0, device=DEV) for _ in range(2))
+            raw = torch.zeros(t, h * vd, device=DEV)
+            ops.retention_scan(raw, proj, *cols[:3], self.state, qs, slots, pos, decay, hi, len(parts) + 1, h, d,
+                               vd, self.rot, d ** -0.5, max(1, vd // 2), segments=segments, angles=angles)
+            ops.retention_finish(out, raw, proj, cols[3], seq, h, vd, self.eps)
+        return out.cpu().double()[:, :h * vd].reshape(t, h, vd)
+
+
+@pytest.mark.parametrize("mode", ["step", "scan", "segments"])
+@pytest.mark.parametrize("heads,dim,vdim,rot", [(2, 16, 24, 8), (3, 24, 8, 24), (1, 10, 17, 0), (2, 64, 16, 2)])
+def test_retention(heads, dim, vdim, rot, mode):
+    """A sequence whole, then in portions down to one token and longer than a segment, beside
+    another request; a slot's earlier state is not read at position 0; a token from 140 positions
+    back whose key and value stand out is still there."""
+    c = RetentionCase(heads, dim, vdim, rot, [0.999, 0.9, 0.98][:heads], seed=dim + vdim)
+    n = 150
+    a, b = c.rows(n), c.rows(31)
+    a[1][5] *= 20.0
+    want, want2 = c.plain(*a), c.plain(*b)
+    ok = P.retention_outputs(a[0].double(), a[1].double(), a[2].double(), c.decay).norm(dim=-1) > 0.3
+    tol = dict(atol=2e-4, rtol=2e-4)
+
+    def same(got, ref, keep=None):
+        if keep is not None:
+            got, ref = got[keep], ref[keep]
+        return torch.allclose(got, ref, **tol)
+
+    assert same(c.run([(1, 0, *a)], mode), want, ok)
+    cuts = [1, 2, 70, 1, 1, 5, 66, 2, 1, 1]
+    at, i, other = 0, 0, 0
+    while at < n:
+        m = min(cuts[i % len(cuts)], n - at)
+        i += 1
+        parts, mo = [(2, at, *(x[at:at + m] for x in a))], 0
+        if other < 31:
+            mo = min(3, 31 - other)
+            parts.insert(0, (0, other, *(x[other:other + mo] for x in b)))
+        got = c.run(parts, mode)
+        assert other == 0 or same(got[:mo], want2[other:other + mo])
+        assert same(got[mo:], want[at:at + m], ok[at:at + m])
+        other += mo
+        at += m
+
+
+# ------------------------------------------------------------------------ whole models
+def _att(heads, kv, dim, ff, conv, rot=None, base=10000.0, cap=20.0, scale=None, bands=None):
+    rot = {"base": base, "dims": dim if rot is None else rot}
+    if bands:
+        rot["scaling"] = dict(zip(("factor", "low", "high", "original"), bands))
+    return {"type": "attention", "mlp": None if ff is None else {"kind": "dense", "ff": ff},
+            "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "conv": conv, "softcap": cap,
+                      "scale": 1.4 / math.sqrt(dim) if scale is None else scale, "rot": rot}}
+
+
+def _ret(heads, dim, vdim, ff, decay, rot=None, base=10000.0):
+    return {"type": "retention", "mlp": None if ff is None else {"kind": "dense", "ff": ff},
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay,
+                      "rot": {"base": base, "dims": dim if rot is None else rot}}}
+
+
+def _model(vocab, width, layers, loop=None, mult=0.6, cap=9.0, eps=1e-5):
+    out = {"architecture": "Musilorn", "vocab": vocab, "width": width, "norm": {"eps": eps},
+           "residual_mult": mult, "logit_softcap": cap, "layers": layers}
+    if loop:
+        out["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return out
+
+
+SHAPE_A = _model(300, 72, [
+    _ret(3, 16, 24, 56, [0.9, 0.97, 0.995], rot=8),
+    _att(4, 2, 24, None, 2, rot=16, cap=4.0),
+    _att(2, 1, 16, 88, 5, cap=6.0, bands=(3.0, 1.0, 2.5, 96)),
+    _ret(2, 24, 8, None, [0.99, 0.8])], loop=(1, 3, 2))
+# a loop over everything from the first layer to the last, one tap, as many key/value heads as
+# heads, sizes no kernel has an instance for, a head without rotation, mult 1
+SHAPE_B = _model(515, 128, [
+    _att(3, 3, 40, 72, 1, rot=40, base=300.0, cap=50.0),
+    _att(6, 6, 10, None, 3, rot=0, cap=2.0),
+    _ret(1, 40, 136, 200, [0.985], rot=12, base=77.0)], loop=(0, 3, 3), mult=1.0, cap=30.0, eps=1e-6)
+# no loop, heads of 64 and 128, many query heads a key/value head
+SHAPE_C = _model(200, 256, [
+    _att(8, 2, 64, 320, 4, cap=15.0, bands=(8.0, 1.0, 4.0, 128)),
+    _ret(4, 64, 64, 192, [0.9, 0.99, 0.995, 0.999]),
+    _att(12, 2, 128, 160, 3, rot=64, cap=10.0, base=500000.0)], mult=0.4)
+# one pass of a loop that ends the model, a single layer behind the loop's start
+SHAPE_D = _model(97, 48, [_att(2, 2, 32, 40, 3), _ret(2, 8, 40, 40, [0.95, 0.9])], loop=(1, 2, 1))
+SHAPES = {"A": (SHAPE_A, 51), "B": (SHAPE_B, 52), "C": (SHAPE_C, 53), "D": (SHAPE_D, 54)}
+CASES = [(name, dtype) for name in SHAPES for dtype in ("float32", "bfloat16")]
+# Relative difference of a row of logits (see ``row_error``).  float32: summation order only.
+# bfloat16: normed streams, the mixers' results, activations and cache rows are rounded to 8
+# bits of mantissa, and a norm behind every branch brings its result (with its rounding) to
+# unit size.  The largest row and the middle one are both bounded.  A retention head whose sum
+# all but cancels before its unit norm moves far under any rounding of its inputs: the plain
+# implementation measures that itself, by rounding what its products read of the stream, and a
+# row may differ by 3 times what that rounding alone does to it; such rows stay few.
+TOL = {"float32": 2e-4, "bfloat16": 6e-2}
+TOL_MEDIAN = {"float32": 2e-5, "bfloat16": 2e-2}
+ROUNDING_FACTOR = 3.0
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    from pretrained_rstr_b200.config.registry import lookup
+    from pretrained_rstr_b200.weights import make_random_model
+    out = {}
+    for name, (raw, seed) in SHAPES.items():
+        cfg = lookup(raw).config_class.from_dict(raw)
+        for dtype in ("float32", "bfloat16"):
+            path = str(tmp_path_factory.mktemp(f"musilorn{name}_{dtype}"))
+            make_random_model(path, cfg, seed, torch.bfloat16 if dtype == "bfloat16" else torch.float32)
+            out[(name, dtype)] = path
+    return out
+
+
+class Oracle(dict):
+    """request -> logits [T, vocab]; ``moved[request][t]``: how far rounding what the products read
+    of the stream moves row t of the plain implementation itself (bfloat16 folders only)."""
+
+
+def _oracle(folder, prompts):
+    cfg, tensors = P.read_folder(folder)
+    out = Oracle()
+    out.moved = {}
+    for rid, ids in prompts.items():
+        out[rid] = P.forward(list(ids), tensors, cfg).to(torch.float32)
+        if "bfloat16" in folder:
+            rounded = P.forward(list(ids), tensors, cfg, rounded=True)
+            out.moved[rid] = [row_error(rounded[t], out[rid][t]) for t in range(len(ids))]
+    return out
+
+
+def row_error(row, ref) -> float:
+    """Root mean square of the difference (its mean taken off) over that of the reference row."""
+    d = row.double() - ref.double()
+    d = d - d.mean()
+    r = ref.double() - ref.double().mean()
+    return float(d.pow(2).mean().sqrt() / r.pow(2).mean().sqrt())
+
+
+def compare(rows, oracle, tol):
+    assert rows
+    errs, excused = [], 0
+    for (rid, pos), row in sorted(rows.items()):
+        err = row_error(row, oracle[rid][pos])
+        assert err == err, f"NaN at request {rid} position {pos}"
+        moved = getattr(oracle, "moved", {}).get(rid)
+        if err > tol and moved is not None and err <= ROUNDING_FACTOR * moved[pos]:
+            excused += 1
+            continue
+        assert err <= tol, (f"request {rid} position {pos} (page offset {pos % 64}): relative "
+                            f"difference {err:.3e} > {tol:.1e}")
+        errs.append(err)
+    errs.sort()
+    middle = errs[len(errs) // 2]
+    print(f"rows {len(errs)}: median {middle:.2e}, largest {errs[-1]:.2e}, excused {excused}")
+    assert excused <= max(1, len(rows) // 50), "too many ill-conditioned rows for the test to mean much"
+    bound = TOL_MEDIAN["float32" if tol == TOL["float32"] else "bfloat16"]
+    assert len(errs) < 8 or middle <= bound, f"the middle row differs by {middle:.3e} > {bound:.1e}"
+    return errs[-1]
+
+
+def _prompts(name, lengths, salt=0):
+    raw, seed = SHAPES[name]
+    return {f"r{i}": random_tokens(n, raw["vocab"], 1000 * seed + salt + i) for i, n in enumerate(lengths)}
+
+
+def test_layers_one_by_one(folders):
+    """The stream after every layer run (each pass of the loop counts) in 32-bit."""
+    from pretrained_rstr_b200.engine.batch import Entry
+    from pretrained_rstr_b200.engine.loading import load_model
+    for name in SHAPES:
+        folder = folders[(name, "float32")]
+        cfg, tensors = P.read_folder(folder)
+        ids = _prompts(name, [37])["r0"]
+        taps = []
+        P.forward(ids, tensors, cfg, taps=taps)
+        lm = load_model(folder, dtype="float32", page_size=64, max_batched_tokens=64, max_requests=2,
+                        max_tokens=128)
+        seen = []
+        lm.model.tap = lambda i, x: seen.append(x[:len(ids)].detach().cpu().double().clone())
+        lm.cache.open("a")
+        lm.runner.step([Entry("a", ids, [0])])
+        lm.runner.check_status()
+        assert len(seen) == len(taps) == len(P.run_list(cfg))
+        for i, (got, want) in enumerate(zip(seen, taps)):
+            assert float((got - want).abs().max()) < 2e-4 * float(want.abs().max()), f"{name}: layer run {i}"
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_whole_prompts_decode_and_portions(folders, name, dtype):
+    """Whole prompts in one step; the last tokens one by one; portions of several sizes, down to
+    two tokens, cut inside pages, convolutions and segments."""
+    folder = folders[(name, dtype)]
+    prompts = _prompts(name, [1, 2, 23, 64, 65, 150, 260])
+    oracle = _oracle(folder, prompts)
+    rp = Replayer(folder, dtype, max_tokens=512)
+    for rid, ids in prompts.items():
+        rp.step([(rid, ids, list(range(len(ids))))], end=[rid])
+    compare(rp.rows, oracle, TOL[dtype])
+    rp.rows.clear()
+    for rid, ids in prompts.items():
+        head = max(1, len(ids) - 40)
+        rp.step([(rid, ids[:head], [head - 1])], end=[rid] if head == len(ids) else [])
+        for i in range(head, len(ids)):
+            rp.step([(rid, ids[i:i + 1], [0])], end=[rid] if i == len(ids) - 1 else [])
+    compare(rp.rows, oracle, TOL[dtype])
+    rp.rows.clear()
+    sizes = [3, 2, 19, 2, 2, 40, 5, 64, 2, 66, 2, 130]
+    for r, (rid, ids) in enumerate(prompts.items()):
+        at, k = 0, r
+        while at < len(ids):
+            n = min(sizes[k % len(sizes)], len(ids) - at)
+            k += 1
+            rp.step([(rid, ids[at:at + n], list(range(n)))], end=[rid] if at + n >= len(ids) else [])
+            at += n
+    compare(rp.rows, oracle, TOL[dtype])
+
+
+def test_other_page_sizes(folders):
+    for name, dtype, page in (("A", "float32", 16), ("C", "bfloat16", 32), ("C", "bfloat16", 128)):
+        folder = folders[(name, dtype)]
+        prompts = _prompts(name, [70, 131], salt=30)
+        oracle = _oracle(folder, prompts)
+        rp = Replayer(folder, dtype, max_tokens=512, page_size=page)
+        for rid, ids in prompts.items():
+            rp.step([(rid, ids[:50], list(range(50)))])
+        for rid, ids in prompts.items():
+            rp.step([(rid, ids[50:60], list(range(10)))])
+            for i in range(60, len(ids)):
+                rp.step([(rid, ids[i:i + 1], [0])])
+        compare(rp.rows, oracle, TOL[dtype])
+
+
+@pytest.mark.parametrize("name,dtype", [("A", "float32"), ("A", "bfloat16"), ("B", "float32"), ("C", "bfloat16")])
+def test_long_decode(folders, name, dtype):
+    """Two tokens of prompt and 270 decoded one by one: several pages' borders are passed by single
+    tokens, the states are carried all the way."""
+    folder = folders[(name, dtype)]
+    prompts = _prompts(name, [272], salt=50)
+    oracle = _oracle(folder, prompts)
+    rp = Replayer(folder, dtype, max_tokens=320)
+    ids = prompts["r0"]
+    rp.step([("r0", ids[:2], [0, 1])])
+    for i in range(2, len(ids)):
+        rp.step([("r0", ids[i:i + 1], [0])])
+    compare(rp.rows, oracle, TOL[dtype])
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_mixed_batches_with_reuse(folders, name, dtype):
+    """Up to four live requests of unequal lengths, portions of some beside single tokens of
+    others, some left out of a step, in a pool so small that pages and state slots of finished
+    requests are used again: every row as if its request ran alone."""
+    folder = folders[(name, dtype)]
+    lengths = [130, 64, 200, 9, 33, 140, 1, 120, 2, 77]
+    prompts = _prompts(name, lengths, salt=90)
+    oracle = _oracle(folder, prompts)
+    biggest = sorted((-(-n // 64) * 64 for n in lengths), reverse=True)
+    rp = Replayer(folder, dtype, max_tokens=sum(biggest[:4]))
+    rng = random.Random(5)
+    waiting, live, slots_seen = list(prompts), {}, []
+    while waiting or live:
+        while waiting and len(live) < 4:
+            live[waiting.pop(0)] = 0
+        entries, end = [], []
+        for rid in list(live):
+            ids, at = prompts[rid], live[rid]
+            left = len(ids) - at
+            if rng.random() < 0.25 and len(live) > 1:
+                continue                                   # left out of this step
+            if left > 20 and at < len(ids) - 12:
+                n = min(left - 12, rng.choice([2, 3, 8, 21, 64, 70]))
+            else:
+                n = 1
+            entries.append((rid, ids[at:at + n], list(range(n))))
+            live[rid] = at + n
+            if live[rid] == len(ids):
+                end.append(rid)
+                del live[rid]
+        if entries:
+            rp.step(entries, end=end)
+            slots_seen += [rp.lm.cache.slot(r) for r in live if r in rp.pos]
+    cache = rp.lm.cache
+    assert cache.stats["allocated"] > cache.allocators[0].num_pages
+    assert cache.free_pages(0) == cache.allocators[0].num_pages
+    assert len(prompts) > 4 >= len(set(slots_seen))          # state slots were used again
+    compare(rp.rows, oracle, TOL[dtype])
+
+
+def test_steps_of_one_shape_with_and_without_portions(folders):
+    """Two steps of equal token and request counts, one of single tokens only and one with a
+    portion, taking turns until both are replayed from graphs: the convolution's saved inputs are
+    right behind either (a graph recorded for one must not stand in for the other)."""
+    folder = folders[("A", "float32")]
+    prompts = _prompts("A", [60, 60, 60], salt=70)
+    oracle = _oracle(folder, prompts)
+    rp = Replayer(folder, "float32", max_tokens=256)
+    at = {rid: 0 for rid in prompts}
+    ids = list(prompts)
+    for k in range(24):
+        if k % 2:
+            counts = {ids[0]: 1, ids[1]: 1, ids[2]: 1}
+        else:
+            counts = {ids[k % 3]: 3, ids[(k + 1) % 3]: 1, ids[(k + 2) % 3]: 1}
+        rp.step([(r, prompts[r][at[r]:at[r] + n], list(range(n))) for r, n in counts.items()])
+        for r, n in counts.items():
+            at[r] += n
+    assert len(rp.lm.runner._graphs) >= 2
+    compare(rp.rows, oracle, TOL["float32"])
+
+
+def test_marked_token_far_back_and_at_borders(folders, tmp_path):
+    """A model made so that a lost far key, a lost state or an unused first token shows: one token
+    id's table row is large, its key stands out wherever it sits.  It is put at the sequence's
+    start, on both sides of pages' and segments' borders and just before the end, in a prompt and
+    while decoding; the oracle without it is far from the oracle with it."""
+    from pretrained_rstr_b200.weights.safetensors_io import save_file
+    folder = folders[("A", "float32")]
+    cfg, tensors = P.read_folder(folder)
+    tensors = {k: v.clone() for k, v in tensors.items()}
+    marked = 7
+    tensors["embed"][marked] *= 8.0
+    for i in (1, 2):
+        tensors[f"l{i}.mix.k.norm"] *= 2.5
+    path = str(tmp_path / "marked")
+    os.makedirs(path)
+    shutil.copy(folder + "/config.json", path + "/config.json")
+    save_file({k: v.float() for k, v in tensors.items()}, path + "/model.safetensors")
+    cfg, tensors = P.read_folder(path)
+    n = 150
+    base = [t if t != marked else marked + 1 for t in random_tokens(n, cfg["vocab"], 400)]
+    prompts = {"none": base}
+    for spot in (0, 1, 2, 62, 63, 64, 65, 127, 128, n - 7, n - 2):
+        prompts[f"s{spot}"] = base[:spot] + [marked] + base[spot + 1:]
+    oracle = {rid: P.forward(ids, tensors, cfg).to(torch.float32) for rid, ids in prompts.items()}
+    for rid in prompts:
+        if rid != "none":
+            assert row_error(oracle[rid][n - 1], oracle["none"][n - 1]) > 10 * TOL["float32"], rid
+    rp = Replayer(path, "float32", max_tokens=4 * 192)
+    for rid, ids in prompts.items():                             # in a prompt
+        rp.step([(rid, ids, [n - 2, n - 1])], end=[rid])
+    compare(rp.rows, oracle, TOL["float32"])
+    rp.rows.clear()
+    for rid, ids in prompts.items():                             # decoding over the borders
+        rp.step([(rid, ids[:n - 90], [])])
+        for i in range(n - 90, n):
+            rp.step([(rid, ids[i:i + 1], [0])], end=[rid] if i == n - 1 else [])
+    compare(rp.rows, oracle, TOL["float32"])
+
+
+@pytest.mark.parametrize("name,dtype", [("A", "float32"), ("A", "bfloat16"), ("C", "bfloat16"), ("D", "float32")])
+def test_greedy_generation_entry_point(folders, name, dtype):
+    """``load_lm`` / ``generate_ids`` / ``generate_batch``: the scheduler's portions, batches
+    and the steps launched ahead of their token ids choose the plain implementation's tokens."""
+    from pretrained_rstr_b200 import generate_batch, generate_ids, load_lm
+    folder = folders[(name, dtype)]
+    cfg, tensors = P.read_folder(folder)
+    m = load_lm(folder, gpu=True, dtype=dtype, max_lanes=3, max_batched_tokens=128,
+                prefill_chunk=32, maxpos=256)
+    prompts = list(_prompts(name, [1, 9, 33, 70, 130], salt=200).values())
+    n_new = 10
+
+    def agree(prompt, got):
+        want = P.greedy(prompt, n_new, tensors, cfg)
+        for i, (a, b) in enumerate(zip(got, want)):
+            if a != b:
+                row = P.forward(list(prompt) + want[:i], tensors, cfg)[-1]
+                gap = abs(float(row[a] - row[b]))
+                assert dtype == "bfloat16" and gap < 0.1, \
+                    f"token {i} is {a}, plain says {b} (logit gap {gap:.3g})"
+                return
+        assert len(got) == len(want)
+
+    agree(prompts[1], generate_ids(m, prompts[1], n_new))
+    for p, got in zip(prompts, generate_batch(m, prompts, n_new)):
+        agree(p, got)
+    cache = m.engine.lm.cache
+    assert not cache.requests
+    cache.check()
+
+
+def test_replay_as_a_program(folders, tmp_path):
+    """``bin/trace_run`` on a Musilorn folder: the model class comes from config.json; logits of a
+    replayed trace match the plain ones."""
+    import json
+    import subprocess
+
+    import numpy as np
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    folder = folders[("A", "float32")]
+    cfg, tensors = P.read_folder(folder)
+    ids = random_tokens(40, cfg["vocab"], 77)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": ids[:30], "want": [0, 29]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": ids[30:32], "want": []},
+                                     {"id": "b", "tokens": ids[:3], "want": [2]}], "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": ids[32:], "want": [7]}], "end": ["a"]}]
+    out = tmp_path / "out"
+    proc = subprocess.run([os.path.join(root, "bin", "trace_run"), "--model", folder, "--dtype",
+                           "float32", "--out", str(out), "--max-tokens", "128"],
+                          input="\n".join(json.dumps(s) for s in steps) + "\n", text=True,
+                          capture_output=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2"]
+    want = P.forward(ids, tensors, cfg).to(torch.float32)
+    got = [torch.from_numpy(np.fromfile(out / f"{i}.f32", dtype="<f4").reshape(-1, cfg["vocab"]).copy())
+           for i in range(3)]
+    for row, ref in ((got[0][0], want[0]), (got[0][1], want[29]), (got[1][0], want[2]), (got[2][0], want[39])):
+        assert row_error(row, ref) < TOL["float32"]
