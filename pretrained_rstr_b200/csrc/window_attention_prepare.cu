@@ -71,12 +71,25 @@ struct HeadInput {
     __device__ __forceinline__ float get(int i) const {
         if (w == nullptr) return raw(i);
         float s = 0.0f;
+        if (back >= taps - 1 && bias == nullptr) {       // everything lies in this portion
+            for (int j = 0; j < taps; ++j) s = fmaf(w[i * taps + j], row[i - (long)(taps - 1 - j) * ld], s);
+            return s;
+        }
         for (int j = 0; j < taps; ++j) s = fmaf(w[i * taps + j], past(i, taps - 1 - j), s);
         return s;
     }
 };
 
-template <typename C>
+__device__ __forceinline__ void store_pair(float* p, float x, float y) {
+    *reinterpret_cast<float2*>(p) = make_float2(x, y);
+}
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float x, float y) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y);
+}
+
+// U: pairs (or coordinates that stay) a lane owns at most; their numbers are computed once and stay
+// in registers.  0: any size, computed again in every pass.
+template <typename C, int U>
 __global__ void __launch_bounds__(256) wattn_prepare_heads_kernel(PrepArgs a) {
     prb_grid_launch_dependents();
     const int lane = threadIdx.x & 31;
@@ -146,27 +159,56 @@ __global__ void __launch_bounds__(256) wattn_prepare_heads_kernel(PrepArgs a) {
     };
     auto first_of = [&](int u) { return a.interleaved ? 2 * u : u; };
     auto second_of = [&](int u) { return a.interleaved ? 2 * u + 1 : u + half; };
+    constexpr int NU = U > 0 ? U : 1;
+    float r0[NU], r1[NU];                                // (r1: a pair's second number)
+    if constexpr (U > 0) {
+#pragma unroll
+        for (int k = 0; k < U; ++k) {
+            const int u = lane + 32 * k;
+            r0[k] = u < units ? in.get(u < half ? first_of(u) : u - half + a.rot_dims) : 0.0f;
+            r1[k] = u < half ? in.get(second_of(u)) : 0.0f;
+        }
+    }
+    // unit u's numbers: from the registers, or computed
+    auto first_number = [&](int u, int k) {
+        if constexpr (U > 0) return r0[k];
+        else return in.get(u < half ? first_of(u) : u - half + a.rot_dims);
+    };
+    auto second_number = [&](int u, int k) {
+        if constexpr (U > 0) return r1[k];
+        else return in.get(second_of(u));
+    };
+    // every unit of the lane in turn (a loop the compiler can unroll when U is given)
+    auto each_unit = [&](auto f) {
+        if constexpr (U > 0) {
+#pragma unroll
+            for (int k = 0; k < U; ++k)
+                if (lane + 32 * k < units) f(lane + 32 * k, k);
+        } else {
+            for (int u = lane; u < units; u += 32) f(u, 0);
+        }
+    };
     float pre = 1.0f, post = 1.0f;
     if (!is_key && a.temp_every > 0)
         post = 1.0f + a.temp_coef * logf((float)((in.pos + 1) / a.temp_every) + 1.0f);
     if (a.norm_mode == 2 || a.norm_mode == 3) {
         float ss = 0.0f;
-        for (int u = lane; u < units; u += 32) {
-            if (u < half) {
-                const float x0 = in.get(first_of(u)), x1 = in.get(second_of(u));
-                if (a.norm_mode == 2) {
-                    ss = fmaf(x0, x0, fmaf(x1, x1, ss));
-                } else {
-                    float sn, cs;
-                    angle(u, cs, sn);
-                    const float r0 = x0 * cs - x1 * sn, r1 = x1 * cs + x0 * sn;
-                    ss = fmaf(r0, r0, fmaf(r1, r1, ss));
-                }
-            } else {
-                const float x = in.get(u - half + a.rot_dims);
-                ss = fmaf(x, x, ss);
+        each_unit([&](int u, int k) {
+            const float x0 = first_number(u, k);
+            if (u >= half) {
+                ss = fmaf(x0, x0, ss);
+                return;
             }
-        }
+            const float x1 = second_number(u, k);
+            if (a.norm_mode == 2) {
+                ss = fmaf(x0, x0, fmaf(x1, x1, ss));
+            } else {
+                float sn, cs;
+                angle(u, cs, sn);
+                const float y0 = x0 * cs - x1 * sn, y1 = x1 * cs + x0 * sn;
+                ss = fmaf(y0, y0, fmaf(y1, y1, ss));
+            }
+        });
         const float inv = 1.0f / sqrtf(prb_warp_sum(ss) / (float)dim + a.eps);
         if (a.norm_mode == 2) pre = inv;
         else post *= inv;
@@ -178,26 +220,46 @@ __global__ void __launch_bounds__(256) wattn_prepare_heads_kernel(PrepArgs a) {
         if (!is_key) qrow[i] = v;
         else if (crow) crow[i] = prb_from_float<C>(v);
     };
-    for (int u = lane; u < units; u += 32) {
-        if (u < half) {
-            const int i0 = first_of(u), i1 = second_of(u);
-            const float x0 = in.get(i0), x1 = in.get(i1);
-            float sn, cs;
-            angle(u, cs, sn);
-            const float y0 = x0 * pre * (nw ? nw[i0] : 1.0f), y1 = x1 * pre * (nw ? nw[i1] : 1.0f);
-            store(i0, (y0 * cs - y1 * sn) * post);
-            store(i1, (y1 * cs + y0 * sn) * post);
-            if (keys_are_values && crow) {
+    // pairs whose two numbers are neighbours go out in one piece
+    const bool together = a.interleaved && dim % 2 == 0 && a.vdim % 2 == 0;
+    auto store2 = [&](int i0, int i1, float y0, float y1, float x0, float x1) {
+        if (!is_key) {
+            if (together) {
+                *reinterpret_cast<float2*>(qrow + i0) = make_float2(y0, y1);
+            } else {
+                qrow[i0] = y0;
+                qrow[i1] = y1;
+            }
+            return;
+        }
+        if (crow == nullptr) return;
+        if (together) {
+            store_pair(crow + i0, y0, y1);
+            if (keys_are_values) store_pair(crow + dim + i0, x0, x1);
+        } else {
+            crow[i0] = prb_from_float<C>(y0);
+            crow[i1] = prb_from_float<C>(y1);
+            if (keys_are_values) {
                 crow[dim + i0] = prb_from_float<C>(x0);
                 crow[dim + i1] = prb_from_float<C>(x1);
             }
+        }
+    };
+    each_unit([&](int u, int k) {
+        const float x0 = first_number(u, k);
+        if (u < half) {
+            const int i0 = first_of(u), i1 = second_of(u);
+            const float x1 = second_number(u, k);
+            float sn, cs;
+            angle(u, cs, sn);
+            const float y0 = x0 * pre * (nw ? nw[i0] : 1.0f), y1 = x1 * pre * (nw ? nw[i1] : 1.0f);
+            store2(i0, i1, (y0 * cs - y1 * sn) * post, (y1 * cs + y0 * sn) * post, x0, x1);
         } else {
             const int i = u - half + a.rot_dims;
-            const float x = in.get(i);
-            store(i, x * pre * (nw ? nw[i] : 1.0f) * post);
-            if (keys_are_values && crow) crow[dim + i] = prb_from_float<C>(x);
+            store(i, x0 * pre * (nw ? nw[i] : 1.0f) * post);
+            if (keys_are_values && crow) crow[dim + i] = prb_from_float<C>(x0);
         }
-    }
+    });
     if (is_key && a.v_col >= 0 && crow) {
         const float* vrow = a.proj + (size_t)t * a.ld + a.v_col + hd * a.vdim;
         for (int j = lane; j < a.vdim; j += 32)
@@ -300,9 +362,20 @@ PRB_API int prb_wattn_prepare_heads(float* q_out, void* cache, const float* proj
     // few units: two warps a CTA, so that they spread over the SMs
     const int warps = units <= 4L * prb_sm_count() ? 2 : 8;
     const unsigned blocks = (unsigned)((units + warps - 1) / warps);
-    if (cache_dtype == PRB_F32) wattn_prepare_heads_kernel<float><<<blocks, warps * 32, 0, stream>>>(a);
-    else if (cache_dtype == PRB_BF16) wattn_prepare_heads_kernel<__nv_bfloat16><<<blocks, warps * 32, 0, stream>>>(a);
+    const int lane_units = (dim - rot_dims / 2 + 31) / 32;
+#define PREP1(CT, UN) wattn_prepare_heads_kernel<CT, UN><<<blocks, warps * 32, 0, stream>>>(a)
+#define PREP(CT)                                                                                 \
+    do {                                                                                         \
+        if (lane_units == 1) PREP1(CT, 1);                                                       \
+        else if (lane_units == 2) PREP1(CT, 2);                                                  \
+        else if (lane_units <= 4) PREP1(CT, 4);                                                  \
+        else PREP1(CT, 0);                                                                       \
+    } while (0)
+    if (cache_dtype == PRB_F32) PREP(float);
+    else if (cache_dtype == PRB_BF16) PREP(__nv_bfloat16);
     else return PRB_E_DTYPE;
+#undef PREP
+#undef PREP1
     PRB_LAUNCH_CHECK();
     if (conv_q != nullptr && taps > 1 && n_requests > 0) {
         const int channels = (heads + kv_heads) * dim;

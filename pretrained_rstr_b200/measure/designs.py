@@ -78,9 +78,9 @@ def cache_bytes_per_token(m) -> int:
 
 
 def _mixers(m):
-    """Every mixer of the model's layer runs (the two of a pair side by side apart)."""
-    for block in m.loaded.model.blocks:
-        mixer = getattr(block, "mixer", None)
+    """The mixer of every layer run of the model, in order (the two of a pair side by side apart)."""
+    for entry in m.loaded.model.order:
+        mixer = getattr(m.loaded.model.blocks[entry.layer], "mixer", None)
         if mixer is not None:
             yield from getattr(mixer, "children", [mixer])
 
@@ -90,10 +90,20 @@ def request_bytes(m, context: int) -> int:
     holds ``context`` tokens: mixers that say so themselves (``step_bytes(context)``: a window's
     keys, a layer that reads another's cache, a state) are asked; the others count every cache
     row of the context."""
-    asked = [mx.step_bytes(context) for mx in _mixers(m) if hasattr(mx, "step_bytes")]
-    if asked:
-        return sum(asked)
-    return context * cache_bytes_per_token(m)
+    total = 0
+    for mixer in _mixers(m):
+        if hasattr(mixer, "step_bytes"):
+            total += mixer.step_bytes(context)
+            continue
+        spec = mixer.kv_spec()
+        if spec is not None:
+            total += context * spec.kv_heads * spec.head_dim * 2 * (2 if spec.values else 1)
+        for st in mixer.state_specs():
+            n = 1
+            for d in st.shape:
+                n *= d
+            total += 2 * 4 * n
+    return total
 
 
 def measure_size(name: str, batches: Sequence[int] = (1, 8, 64), context: int = 1000,

@@ -177,9 +177,11 @@ class WindowAttention(Mixer):
                           torch.float32)]
 
     def step_bytes(self, context: int) -> int:
-        """Cache bytes a single token at ``context`` tokens reads: the rows it sees."""
+        """Bytes a single token at ``context`` tokens reads: the rows it sees, its saved inputs."""
         seen = min(context, self.window + self.keep_first) if self.window else context
-        return seen * self.kv_heads * (self.dim + self.vdim) * self.runtime.dtype.itemsize
+        rows = seen * self.kv_heads * (self.dim + self.vdim) * self.runtime.dtype.itemsize
+        inputs = max(self.taps - 1, 0) * (self.heads + self.kv_heads) * self.dim
+        return rows + 2 * 4 * inputs                 # (a convolution's saved inputs: read, written back)
 
     def fuse_input_rows(self, name: str, weight) -> str:
         return self.input.add(name, weight)
