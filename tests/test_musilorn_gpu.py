@@ -440,8 +440,8 @@ SHAPE_B = _model(515, 128, [
     _att(6, 6, 10, None, 3, rot=0, cap=2.0),
     _ret(1, 40, 136, 200, [0.985], rot=12, base=77.0)], loop=(0, 3, 3), mult=1.0, cap=30.0, eps=1e-6)
 # no loop, heads of 64 and 128, many query heads a key/value head
-SHAPE_C = _model(200, 256, [
-    _att(8, 2, 64, 320, 4, cap=15.0, bands=(8.0, 1.0, 4.0, 128)),
+SHAPE_C = _model(200, 192, [
+    _att(10, 2, 64, 288, 4, cap=12.0, bands=(6.0, 1.0, 4.0, 128)),
     _ret(4, 64, 64, 192, [0.9, 0.99, 0.995, 0.999]),
     _att(12, 2, 128, 160, 3, rot=64, cap=10.0, base=500000.0)], mult=0.4)
 # one pass of a loop that ends the model, a single layer behind the loop's start
