@@ -1,0 +1,240 @@
+// Activations between the two products of a feed-forward, a launch each:
+//
+// expert_act: a router that scores by the softmax over all experts and chooses by score plus a
+//   correction per expert, and the gated activation of the chosen experts with their weights (the
+//   scores without the correction, optionally shares of their sum, times a constant).  The last
+//   `identity` of the router's experts give back the feed-forward's input: their weight times the
+//   input joins the stream here.  An optional shared expert runs for every token, optionally times
+//   sigmoid of one more column.
+// act_columns: act(in) of a range of columns.
+// Inputs are columns of one 32-bit product; results in the products' type.  32-bit arithmetic.
+#include "common.cuh"
+
+namespace {
+__device__ __forceinline__ float ea_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float ea_gate(float g, int act) {     // 0: silu, 1: gelu (tanh form)
+    return act == 1 ? prb_activate(g, PRB_ACT_GELU_TANH) : g * ea_sigmoid(g);
+}
+
+struct ExpertArgs {
+    void* out; long out_ld;
+    const float* in; long in_ld;
+    int gate_col, up_col, router_col, shared_gate_col, shared_up_col, shared_weight_col;
+    int n_rows, experts, identity, top, group, shared, renorm, act;
+    float factor;
+    const float* correction;         // [experts + identity], or null
+    // identity experts: x += weight * h, with h given or (h == null) x / rms(x) * norm_w
+    float* x; long x_ld; int width;
+    const void* h; long h_ld;
+    const float* norm_w;
+    float eps;
+};
+
+template <typename O>
+__device__ __forceinline__ void store4(O* o, const float (&v)[4]) {
+    if constexpr (sizeof(O) == 4) {
+        *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(o) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo),
+                                                  *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+
+// CTAs (row, slice of the row's columns); every CTA of a row chooses for itself.
+template <typename O>
+__global__ void __launch_bounds__(256) expert_act_kernel(ExpertArgs a) {
+    extern __shared__ float sh[];                    // [all] scores, [all] choice, [all] weights
+    __shared__ float scratch[32];
+    __shared__ float own_s[2];                       // the identity experts' weight, the shared expert's
+    const int all = a.experts + a.identity;
+    float* sc = sh;
+    float* pick = sh + all;
+    float* wt = sh + 2 * all;
+    prb_grid_launch_dependents();
+    const int t = blockIdx.x;
+    const float* row = a.in + (size_t)t * a.in_ld;
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        float top_z = -INFINITY;
+        for (int e = lane; e < all; e += 32) top_z = fmaxf(top_z, row[a.router_col + e]);
+        top_z = prb_warp_max(top_z);
+        float sum = 0.0f;
+        for (int e = lane; e < all; e += 32) {
+            const float p = expf(row[a.router_col + e] - top_z);
+            sc[e] = p;
+            sum += p;
+        }
+        sum = prb_warp_sum(sum);
+        for (int e = lane; e < all; e += 32) {
+            const float s = sc[e] / sum;
+            sc[e] = s;
+            pick[e] = s + (a.correction ? a.correction[e] : 0.0f);
+            wt[e] = 0.0f;
+        }
+        __syncwarp();
+        float chosen = 0.0f;
+        for (int k = 0; k < a.top; ++k) {            // the largest left; ties: the lower index
+            float best = -INFINITY;
+            int arg = all;
+            for (int e = lane; e < all; e += 32) {
+                const float v = pick[e];
+                if (v > best) { best = v; arg = e; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float v = __shfl_xor_sync(0xffffffffu, best, o);
+                const int w = __shfl_xor_sync(0xffffffffu, arg, o);
+                if (w < all && (arg >= all || v > best || (v == best && w < arg))) { best = v; arg = w; }
+            }
+            if (arg >= all) break;                   // (a row of NaNs: padding, or a fault upstream)
+            if (lane == 0) {
+                wt[arg] = sc[arg];
+                pick[arg] = -INFINITY;
+            }
+            chosen += sc[arg];
+            __syncwarp();
+        }
+        const float mult = a.factor / (a.renorm ? chosen : 1.0f);
+        float own = 0.0f;
+        for (int e = lane; e < all; e += 32) {
+            const float w = wt[e] * mult;
+            wt[e] = w;
+            if (e >= a.experts) own += w;
+        }
+        own = prb_warp_sum(own);
+        if (lane == 0) {
+            own_s[0] = own;
+            own_s[1] = a.shared_weight_col >= 0 ? ea_sigmoid(row[a.shared_weight_col]) : 1.0f;
+        }
+    }
+    __syncthreads();
+    // columns: the experts' (experts * group), then the shared expert's
+    const int n_exp = a.experts * a.group, n_all = n_exp + a.shared;
+    const int per = ((n_all + (int)gridDim.y - 1) / (int)gridDim.y + 3) / 4 * 4;
+    const int lo = blockIdx.y * per, hi = min(n_all, lo + per);
+    O* o = (O*)a.out + (size_t)t * a.out_ld;
+    const bool vec = a.group % 4 == 0 && (a.gate_col | a.up_col | a.in_ld | a.out_ld) % 4 == 0 &&
+                     (a.shared == 0 || (a.shared_gate_col | a.shared_up_col | a.shared) % 4 == 0) &&
+                     ((uintptr_t)a.in) % 16 == 0 && ((uintptr_t)a.out) % (4 * sizeof(O)) == 0;
+    if (vec) {
+        for (int i = lo + threadIdx.x * 4; i < hi; i += blockDim.x * 4) {
+            const bool routed = i < n_exp;
+            const float w = routed ? wt[i / a.group] : own_s[1];
+            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if (w != 0.0f) {                         // (columns of experts not chosen are not read)
+                const int gc = routed ? a.gate_col + i : a.shared_gate_col + i - n_exp;
+                const int uc = routed ? a.up_col + i : a.shared_up_col + i - n_exp;
+                const float4 g = *reinterpret_cast<const float4*>(row + gc);
+                const float4 u = *reinterpret_cast<const float4*>(row + uc);
+                v[0] = w * ea_gate(g.x, a.act) * u.x;
+                v[1] = w * ea_gate(g.y, a.act) * u.y;
+                v[2] = w * ea_gate(g.z, a.act) * u.z;
+                v[3] = w * ea_gate(g.w, a.act) * u.w;
+            }
+            store4(o + i, v);
+        }
+    } else {
+        for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) {
+            const bool routed = i < n_exp;
+            const float w = routed ? wt[i / a.group] : own_s[1];
+            float v = 0.0f;
+            if (w != 0.0f)
+                v = routed ? w * ea_gate(row[a.gate_col + i], a.act) * row[a.up_col + i]
+                           : w * ea_gate(row[a.shared_gate_col + i - n_exp], a.act) *
+                                 row[a.shared_up_col + i - n_exp];
+            o[i] = prb_from_float<O>(v);
+        }
+    }
+    if (a.identity > 0 && blockIdx.y == 0 && own_s[0] != 0.0f) {
+        const float w = own_s[0];
+        float* x = a.x + (size_t)t * a.x_ld;
+        if (a.h != nullptr) {
+            const O* h = (const O*)a.h + (size_t)t * a.h_ld;
+            for (int i = threadIdx.x; i < a.width; i += blockDim.x)
+                x[i] = fmaf(w, prb_to_float<O>(h[i]), x[i]);
+        } else {
+            float ss = 0.0f;
+            for (int i = threadIdx.x; i < a.width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+            ss = prb_block_sum(ss, scratch);
+            const float inv = w / sqrtf(ss / (float)a.width + a.eps);
+            for (int i = threadIdx.x; i < a.width; i += blockDim.x)
+                x[i] = fmaf(x[i] * inv, a.norm_w ? a.norm_w[i] : 1.0f, x[i]);
+        }
+    }
+}
+
+__device__ __forceinline__ float column_act(float v, int act) {
+    switch (act) {
+        case 0: { const float r = fmaxf(v, 0.0f); return r * r; }
+        case 1: return fmaxf(v, 0.0f);
+        case 2: return prb_activate(v, PRB_ACT_GELU_TANH);
+        default: return v * ea_sigmoid(v);
+    }
+}
+
+template <typename O, bool VEC>
+__global__ void act_columns_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ in, long in_ld,
+                                   int n, int n_rows, int act) {
+    prb_grid_launch_dependents();
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if constexpr (VEC) {
+        const int n4 = n / 4;
+        if (idx >= (size_t)n_rows * n4) return;
+        const int t = (int)(idx / n4), i = (int)(idx - (size_t)t * n4) * 4;
+        const float4 u = *reinterpret_cast<const float4*>(in + (size_t)t * in_ld + i);
+        const float v[4] = {column_act(u.x, act), column_act(u.y, act), column_act(u.z, act), column_act(u.w, act)};
+        store4(out + (size_t)t * out_ld + i, v);
+    } else {
+        if (idx >= (size_t)n_rows * n) return;
+        const int t = (int)(idx / n), i = (int)(idx - (size_t)t * n);
+        out[(size_t)t * out_ld + i] = prb_from_float<O>(column_act(in[(size_t)t * in_ld + i], act));
+    }
+}
+}  // namespace
+
+PRB_API int prb_expert_act(void* out, long out_ld, const float* in, long in_ld, int gate_col, int up_col,
+                           int router_col, int shared_gate_col, int shared_up_col, int shared_weight_col,
+                           int n_rows, int experts, int identity, int top, int group, int shared, int renorm,
+                           int act, float factor, const float* correction, float* x, long x_ld, int width,
+                           const void* h, long h_ld, const float* norm_w, float eps, int dtype,
+                           cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    const int all = experts + identity;
+    if (experts < 0 || identity < 0 || all <= 0 || all > 2048 || top <= 0 || top > all || group <= 0 ||
+        shared < 0 || act < 0 || act > 1)
+        return PRB_E_SIZE;
+    if (identity > 0 && (x == nullptr || width <= 0)) return PRB_E_ARG;
+    const ExpertArgs a{out, out_ld, in, in_ld, gate_col, up_col, router_col, shared_gate_col, shared_up_col,
+                       shared_weight_col, n_rows, experts, identity, top, group, shared, renorm, act, factor,
+                       correction, x, x_ld, width, h, h_ld, norm_w, eps};
+    // slices of 2,048 columns, fewer while the rows alone fill the GPU
+    int slices = (experts * group + shared + 2047) / 2048;
+    if (slices < 1) slices = 1;
+    if (slices > 64) slices = 64;
+    while (slices > 1 && (long)n_rows * slices > 8L * prb_sm_count()) slices = (slices + 1) / 2;
+    const dim3 grid(n_rows, slices);
+    const size_t smem = (size_t)3 * all * sizeof(float);
+    if (dtype == PRB_F32) expert_act_kernel<float><<<grid, 256, smem, stream>>>(a);
+    else if (dtype == PRB_BF16) expert_act_kernel<__nv_bfloat16><<<grid, 256, smem, stream>>>(a);
+    else return PRB_E_DTYPE;
+    PRB_LAUNCH_CHECK();
+    return 0;
+}
+
+// act 0: relu(.)^2, 1: relu, 2: gelu (tanh form), 3: silu; `in` points at the first column.
+PRB_API int prb_act_columns(void* out, long out_ld, const float* in, long in_ld, int n, int n_rows, int act,
+                            int out_dtype, cudaStream_t stream) {
+    if (n <= 0 || n_rows <= 0) return 0;
+    if (act < 0 || act > 3) return PRB_E_ARG;
+    if (out_dtype != PRB_F32 && out_dtype != PRB_BF16) return PRB_E_DTYPE;
+    const size_t esz = out_dtype == PRB_F32 ? 4 : 2, total = (size_t)n * n_rows;
+    const bool vec = (n | in_ld | out_ld) % 4 == 0 && ((uintptr_t)in) % 16 == 0 && ((uintptr_t)out) % (4 * esz) == 0;
+    const unsigned blocks = (unsigned)(((vec ? total / 4 : total) + 255) / 256);
+#define ACTC(OT, V) act_columns_kernel<OT, V><<<blocks, 256, 0, stream>>>((OT*)out, out_ld, in, in_ld, n, n_rows, act)
+    if (out_dtype == PRB_F32) { if (vec) ACTC(float, true); else ACTC(float, false); }
+    else { if (vec) ACTC(__nv_bfloat16, true); else ACTC(__nv_bfloat16, false); }
+#undef ACTC
+    PRB_LAUNCH_CHECK();
+    return 0;
+}

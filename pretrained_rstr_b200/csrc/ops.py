@@ -141,7 +141,7 @@ def _declare(h: ctypes.CDLL) -> None:
     h.prb_norm_pair.restype = c_int
     h.prb_tanh_cap.argtypes = [P, L, I, I, F, P]
     h.prb_tanh_cap.restype = c_int
-    h.prb_rotary_angles.argtypes = [P, P, P, P, I, I, P]
+    h.prb_rotary_angles.argtypes = [P, P, P, P, I, I, F, P]
     h.prb_rotary_angles.restype = c_int
     h.prb_wattn_prepare_heads.argtypes = [P, P, P, L, I, I, I] + [P] * 7 + \
         [I, P, I, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, I, I, I, I, P, P]
@@ -237,6 +237,34 @@ def _declare(h: ctypes.CDLL) -> None:
     for name in ("prb_lru_max_taps", "prb_lru_conv", "prb_lru_gates", "prb_lru_scan",
                  "prb_mmem_supports", "prb_mmem_step", "prb_mmem_segment",
                  "prb_mmem_max_segments", "prb_mmem_scan_supports", "prb_mmem_scan"):
+        getattr(h, name).restype = c_int
+    h.prb_dscan_segment.argtypes = []
+    h.prb_dscan_max_segments.argtypes = [I, I]
+    h.prb_dscan_supports.argtypes = [I, I]
+    h.prb_dscan_segments.argtypes = [P, L, P, L, I, P, L, I, P, L, P, L, I, P, P, F, P, P, P, P, I, I, I,
+                                     I, I, I, P, P, P, I, P, L, P, L, P, F, F, I, P, P]
+    h.prb_gla_finish.argtypes = [P, L, P, L, P, L, P, P, I, I, I, F, F, I, P]
+    h.prb_gla_decay.argtypes = [P, L, P, L, P, P, I, I, I, F, P]
+    h.prb_gla_step_supports.argtypes = [I, I]
+    h.prb_gla_step.argtypes = [P, L, P, L, I, I, I, I, I, P, P, F, F, P, F, F, P, P, P, P, I, I, I, I, I,
+                               I, I, I, P, P]
+    ssm = [P, L, I, I, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, L, P, I, F, F, P, L, P]
+    h.prb_ssm_max_taps.argtypes = []
+    h.prb_ssm_chunk_supports.argtypes = [I, I]
+    h.prb_ssm_step_supports.argtypes = [I, I]
+    h.prb_ssm_prepare.argtypes = ssm + [P, L, I, P, P, I, P]
+    h.prb_ssm_chunks.argtypes = ssm + [P, L, P, P, P, P, P, P, I, P]
+    h.prb_ssm_finish.argtypes = ssm + [I, I, P]
+    h.prb_ssm_step.argtypes = ssm + [P, I, P]
+    h.prb_embed_norm.argtypes = [P, P, P, P, I, I, I, F, I, P, P]
+    h.prb_expert_act.argtypes = [P, L, P, L, I, I, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P, L, I, P, L,
+                                 P, F, I, P]
+    h.prb_act_columns.argtypes = [P, L, P, L, I, I, I, I, P]
+    for name in ("prb_dscan_segment", "prb_dscan_max_segments", "prb_dscan_supports",
+                 "prb_dscan_segments", "prb_gla_finish", "prb_gla_decay", "prb_gla_step_supports",
+                 "prb_gla_step", "prb_ssm_max_taps", "prb_ssm_chunk_supports",
+                 "prb_ssm_step_supports", "prb_ssm_prepare", "prb_ssm_chunks", "prb_ssm_finish",
+                 "prb_ssm_step", "prb_embed_norm", "prb_expert_act", "prb_act_columns"):
         getattr(h, name).restype = c_int
     for name in ("prb_tmix_lanes", "prb_tmix_shift", "prb_tmix_scan", "prb_tmix_finish",
                  "prb_tmix_step_supports", "prb_tmix_segment", "prb_tmix_max_segments",
@@ -1072,9 +1100,9 @@ def tanh_cap(z, cap: float) -> None:
     _check(lib().prb_tanh_cap(_p(z), z.stride(0), z.shape[0], z.shape[1], float(cap), _stream()), what)
 
 
-def rotary_angles(out, positions, freq, freq_lo) -> None:
-    """out[t, i] = (cos, sin) of positions[t] * (freq[i] + freq_lo[i]), the product in 64-bit; out
-    float32 [T, n, 2]."""
+def rotary_angles(out, positions, freq, freq_lo, magnitude: float = 1.0) -> None:
+    """out[t, i] = magnitude * (cos, sin) of positions[t] * (freq[i] + freq_lo[i]), the product in
+    64-bit; out float32 [T, n, 2]."""
     what = "rotary_angles"
     _need(out, torch.float32, "out", what)
     _need(positions, torch.int32, "positions", what)
@@ -1083,7 +1111,7 @@ def rotary_angles(out, positions, freq, freq_lo) -> None:
     if out.dim() != 3 or out.shape[2] != 2 or positions.numel() < n or freq.numel() < half:
         raise KernelArgumentError(f"{what}: shapes do not fit")
     _check(lib().prb_rotary_angles(_p(out), _p(positions), _p(freq), _p(_freq_lo(freq_lo, 2 * half, what)),
-                                   n, half, _stream()), what)
+                                   n, half, float(magnitude), _stream()), what)
 
 
 def _angles(angles, rows: int, rot_dims: int, what: str):
@@ -1340,6 +1368,20 @@ def embed_scaled(out, tokens, table, scale: float, keep=None, status=None, pair=
                                   table.shape[0], float(scale), dtype_code(table.dtype), _p(pair),
                                   0 if pair is None else pair.stride(0), _p(status), _stream()),
            what)
+
+
+def embed_norm(out, tokens, table, weight, eps: float, status=None) -> None:
+    """out[t] = r / sqrt(mean(r^2) + eps) * weight with r = table[tokens[t]] (float32 [T, width])."""
+    what = "embed_norm"
+    _need(out, torch.float32, "out", what)
+    _need(tokens, torch.int32, "tokens", what)
+    _need(table, None, "table", what)
+    _need(weight, torch.float32, "weight", what)
+    n, width = out.shape
+    if table.shape[1] != width or tokens.numel() < n or weight.numel() != width:
+        raise KernelArgumentError(f"{what}: table, weight or token count does not fit the output")
+    _check(lib().prb_embed_norm(_p(out), _p(tokens), _p(table), _p(weight), n, width, table.shape[0],
+                                float(eps), dtype_code(table.dtype), _p(status), _stream()), what)
 
 
 SCORE_CODES = {"sigmoid": 0, "identity": 1, "softmax": 2}
@@ -2206,3 +2248,324 @@ def mmem_scan(out, raw, gates, proj, cols, i_bias, f_bias, norm_w, state_s, stat
     _check(code, what)
     if code == 0 and n > 0:
         add_launches(4 if segments is not None else 2)
+
+
+# ------------------------------------------------ activations between a feed-forward's products
+def _columns_of(inp, what: str) -> None:
+    if not inp.is_cuda or inp.dtype != torch.float32 or inp.stride(1) != 1:
+        raise KernelArgumentError(f"{what}: inp must be float32 on CUDA with unit inner stride")
+
+
+def act_columns(out, inp, act: str = "relu_squared") -> None:
+    """out[t, i] = act(inp[t, i]) for the columns of ``inp`` (float32; a column slice is fine); out in
+    the activation type with at least as many columns."""
+    what = "act_columns"
+    _columns_of(inp, what)
+    n_rows, n = inp.shape
+    if not out.is_cuda or out.stride(1) != 1 or out.shape[0] < n_rows or out.shape[1] < n:
+        raise KernelArgumentError(f"{what}: out has the wrong shape")
+    _check(lib().prb_act_columns(_p(out), out.stride(0), _p(inp), inp.stride(0), n, n_rows,
+                                 ROUTED_ACT_CODES[act], dtype_code(out.dtype), _stream()), what)
+
+
+def expert_act(out, inp, gate_col: int, up_col: int, router_col: int, experts: int, top: int, group: int,
+               identity: int = 0, correction=None, renormalize: bool = False, factor: float = 1.0,
+               act: str = "sigmoid", shared=None, stream=None) -> None:
+    """A router over ``experts + identity`` logits (columns ``router_col`` .. of ``inp``) and the
+    chosen experts' gated activations in one launch.  s = softmax over all logits; the ``top``
+    largest s + ``correction`` (float32, or None) are chosen with the weights s (``renormalize``:
+    divided by their sum) times ``factor``; out[t, e * group + i] = weight_e * f(gate) * up, zero
+    for experts not chosen.  ``shared`` = (gate column, up column, size, weight column or -1): an
+    expert every token runs, behind the others' columns, times sigmoid(the weight column).  The last
+    ``identity`` experts give back the feed-forward's input: ``stream`` = (x float32 [T, width], h)
+    receives x += weight * h, with h a tensor in out's type or (norm weight or None, eps): h = x /
+    sqrt(mean(x^2) + eps) * weight, of x as it is when the kernel begins."""
+    what = "expert_act"
+    _columns_of(inp, what)
+    n = experts * group
+    sg, su, size, sw = shared if shared is not None else (0, 0, 0, -1)
+    if not out.is_cuda or out.stride(1) != 1 or out.shape[0] < inp.shape[0] or \
+            out.shape[1] < n + size or max(gate_col, up_col) + n > inp.shape[1] or \
+            router_col + experts + identity > inp.shape[1] or max(sg, su) + size > inp.shape[1] or \
+            sw >= inp.shape[1]:
+        raise KernelArgumentError(f"{what}: columns outside the tensors")
+    if correction is not None:
+        _need(correction, torch.float32, "correction", what)
+        if correction.numel() != experts + identity:
+            raise KernelArgumentError(f"{what}: one correction per expert")
+    x = h = weight = None
+    eps = 0.0
+    if identity > 0:
+        if stream is None:
+            raise KernelArgumentError(f"{what}: identity experts join a stream")
+        x, h = stream
+        _need(x, torch.float32, "x", what)
+        if x.shape[0] < inp.shape[0]:
+            raise KernelArgumentError(f"{what}: fewer rows in the stream than in inp")
+        if isinstance(h, tuple):
+            (weight, eps), h = h, None
+            if weight is not None:
+                _need(weight, torch.float32, "norm weight", what)
+                if weight.numel() != x.shape[1]:
+                    raise KernelArgumentError(f"{what}: the norm's weight does not fit the stream")
+        elif h.dtype != out.dtype or h.stride(1) != 1 or h.shape[0] < inp.shape[0] or \
+                h.shape[1] != x.shape[1]:
+            raise KernelArgumentError(f"{what}: h does not fit the stream")
+    _check(lib().prb_expert_act(
+        _p(out), out.stride(0), _p(inp), inp.stride(0), int(gate_col), int(up_col), int(router_col),
+        int(sg), int(su), int(sw), inp.shape[0], int(experts), int(identity), int(top), int(group),
+        int(size), 1 if renormalize else 0, GATED_ACT_CODES[act], float(factor), _p(correction), _p(x),
+        0 if x is None else x.stride(0), 0 if x is None else x.shape[1], _p(h),
+        0 if h is None else h.stride(0), _p(weight), float(eps), dtype_code(out.dtype), _stream()), what)
+
+
+# ------------------------------------------------ matrix states with decays
+def dscan_segment() -> int:
+    """Tokens of a segment of :func:`decayed_scan`."""
+    return int(lib().prb_dscan_segment())
+
+
+def dscan_max_segments(t_cap: int, b_cap: int) -> int:
+    """Segments a step of at most ``t_cap`` tokens in ``b_cap`` requests can have."""
+    return int(lib().prb_dscan_max_segments(int(t_cap), int(b_cap)))
+
+
+def dscan_supports(dim: int, vdim: int):
+    """(whether :func:`decayed_scan` takes heads of these sizes, whether with ``finish``)."""
+    bits = int(lib().prb_dscan_supports(int(dim), int(vdim)))
+    return bool(bits & 1), bool(bits & 2)
+
+
+def decayed_scan(raw, q, k, v, decay, state, q_start, state_slot, positions, n_requests: int, heads: int,
+                 dim: int, vdim: int, segments, share=(1, 1), k_scale=None, direct=None,
+                 q_scale: float = 1.0, finish=None, status=None) -> None:
+    """Per head S_t = diag(a_t) S_(t-1) + s_t k_t v_t^T and o_t = q_scale * S_t^T q_t + direct * v_t over
+    the step's tokens, request by request, in segments that run side by side.  q, k and v are float32
+    [T, ...] column slices (head h reads ``dim`` numbers of q from (h // share[0]) * dim, of k from
+    (h // share[1]) * dim and ``vdim`` of v from h * vdim); ``decay`` holds a - 1: [T, heads * dim] or
+    [T, heads]; ``k_scale`` s [T, heads] and ``direct`` [heads] may be None.  ``state`` [slots, heads,
+    vdim, dim] is read (zero at position 0) and written back.  ``segments`` = (own, start, decay):
+    workspaces [n, heads, vdim, dim] twice and [n, heads, dim or 1].  ``raw`` float32 [T, heads * vdim]
+    receives o; or ``finish`` = (out, gate, norm weight [vdim], eps, out_scale): out = o /
+    sqrt(mean(o^2) + eps) * weight * silu(gate) * out_scale instead."""
+    what = "decayed_scan"
+    for name, t in (("q", q), ("k", k), ("v", v), ("decay", decay)):
+        _columns_of(t, f"{what} ({name})")
+    for name, t in (("q_start", q_start), ("state_slot", state_slot), ("positions", positions)):
+        _need(t, torch.int32, name, what)
+    _need(state, torch.float32, "state", what)
+    n = q.shape[0]
+    per_key = decay.shape[1] != heads or dim == 1
+    own, start, dec = segments
+    for name, t in (("own", own), ("start", start), ("decay workspace", dec)):
+        _need(t, torch.float32, name, what)
+    if tuple(state.shape[1:]) != (heads, vdim, dim) or heads % share[0] or heads % share[1] or \
+            q.shape[1] < heads // share[0] * dim or k.shape[1] < heads // share[1] * dim or \
+            v.shape[1] < heads * vdim or min(k.shape[0], v.shape[0], decay.shape[0]) < n or \
+            (per_key and decay.shape[1] < heads * dim) or q_start.numel() < n_requests + 1 or \
+            state_slot.numel() < n_requests or positions.numel() < n or \
+            min(own.numel(), start.numel()) < own.shape[0] * heads * vdim * dim or \
+            dec.numel() < own.shape[0] * heads * (dim if per_key else 1):
+        raise KernelArgumentError(f"{what}: shapes do not fit")
+    for name, t, size in (("k_scale", k_scale, n * heads), ("direct", direct, heads)):
+        if t is not None:
+            _need(t, torch.float32, name, what)
+            if t.numel() < size:
+                raise KernelArgumentError(f"{what}: {name} is too short")
+    out = gate = norm_w = None
+    eps = 0.0
+    out_scale = 1.0
+    if finish is not None:
+        out, gate, norm_w, eps, out_scale = finish
+        _columns_of(gate, f"{what} (gate)")
+        _need(norm_w, torch.float32, "norm weight", what)
+        if out.stride(1) != 1 or out.shape[0] < n or out.shape[1] < heads * vdim or \
+                gate.shape[0] < n or gate.shape[1] < heads * vdim or norm_w.numel() != vdim:
+            raise KernelArgumentError(f"{what}: the finish's shapes do not fit")
+    else:
+        _need(raw, torch.float32, "raw", what)
+        if raw.shape[0] < n or raw.shape[1] < heads * vdim:
+            raise KernelArgumentError(f"{what}: raw has the wrong shape")
+    _check(lib().prb_dscan_segments(
+        _p(raw) if finish is None else None, 0 if finish is not None else raw.stride(0), _p(q), q.stride(0),
+        int(share[0]), _p(k), k.stride(0), int(share[1]), _p(v), v.stride(0), _p(decay), decay.stride(0),
+        1 if per_key else 0, _p(k_scale), _p(direct), float(q_scale), _p(state), _p(q_start),
+        _p(state_slot), _p(positions), n, int(n_requests), int(heads), int(dim), int(vdim),
+        state.shape[0], _p(own), _p(start), _p(dec), own.shape[0], _p(out),
+        0 if out is None else out.stride(0), _p(gate), 0 if gate is None else gate.stride(0), _p(norm_w),
+        float(eps), float(out_scale), F32 if out is None else dtype_code(out.dtype), _p(status),
+        _stream()), what)
+    add_launches(2)
+
+
+def gla_finish(out, raw, gate, norm_w, seq_of_token, heads: int, vdim: int, eps: float,
+               out_scale: float = 1.0) -> None:
+    """The finish of :func:`decayed_scan` on its raw sums."""
+    what = "gla_finish"
+    _need(raw, torch.float32, "raw", what)
+    _columns_of(gate, f"{what} (gate)")
+    _need(norm_w, torch.float32, "norm weight", what)
+    _need(seq_of_token, torch.int32, "seq_of_token", what)
+    n = raw.shape[0]
+    if raw.shape[1] < heads * vdim or gate.shape[0] < n or gate.shape[1] < heads * vdim or \
+            out.stride(1) != 1 or out.shape[0] < n or out.shape[1] < heads * vdim or \
+            norm_w.numel() != vdim or seq_of_token.numel() < n:
+        raise KernelArgumentError(f"{what}: shapes do not fit")
+    _check(lib().prb_gla_finish(_p(out), out.stride(0), _p(raw), raw.stride(0), _p(gate), gate.stride(0),
+                                _p(norm_w), _p(seq_of_token), n, int(heads), int(vdim), float(eps),
+                                float(out_scale), dtype_code(out.dtype), _stream()), what)
+
+
+def gla_decay(decay, low_rank, w2t, bias, tau: float) -> None:
+    """decay[t, c] = sigmoid(z)^(1 / tau) - 1 with z = low_rank[t] . w2t[:, c] + bias[c]; ``w2t``
+    float32 [rank, channels]."""
+    what = "gla_decay"
+    _need(decay, torch.float32, "decay", what)
+    _columns_of(low_rank, what)
+    _need(w2t, torch.float32, "w2t", what)
+    _need(bias, torch.float32, "bias", what)
+    rank, channels = w2t.shape
+    n = low_rank.shape[0]
+    if decay.shape[0] < n or decay.shape[1] < channels or low_rank.shape[1] != rank or bias.numel() != channels:
+        raise KernelArgumentError(f"{what}: shapes do not fit")
+    _check(lib().prb_gla_decay(_p(decay), decay.stride(0), _p(low_rank), low_rank.stride(0), _p(w2t),
+                               _p(bias), n, channels, rank, 1.0 / float(tau), _stream()), what)
+
+
+def gla_step_supports(dim: int, vdim: int) -> bool:
+    """Whether :func:`gla_step` takes heads of these sizes."""
+    return bool(lib().prb_gla_step_supports(int(dim), int(vdim)))
+
+
+def gla_step(out, proj, cols, w2t, bias, tau: float, q_scale: float, norm_w, state, q_start, state_slot,
+             positions, n_requests: int, heads: int, dim: int, vdim: int, eps: float,
+             out_scale: float = 1.0, status=None) -> None:
+    """Decays (:func:`gla_decay`), recurrence and finish (:func:`decayed_scan`) of a step in which every
+    request brings one token, in one launch.  ``cols``: the first columns of q, k, v, the low-rank
+    projection and the gate in ``proj`` (float32)."""
+    what = "gla_step"
+    _columns_of(proj, what)
+    for name, t in (("w2t", w2t), ("bias", bias), ("norm weight", norm_w), ("state", state)):
+        _need(t, torch.float32, name, what)
+    for name, t in (("q_start", q_start), ("state_slot", state_slot), ("positions", positions)):
+        _need(t, torch.int32, name, what)
+    q, k, v, lr, g = (int(c) for c in cols)
+    n, width = proj.shape
+    rank = w2t.shape[0]
+    if tuple(state.shape[1:]) != (heads, vdim, dim) or tuple(w2t.shape) != (rank, heads * dim) or \
+            bias.numel() != heads * dim or norm_w.numel() != vdim or max(q, k) + heads * dim > width or \
+            max(v, g) + heads * vdim > width or lr + rank > width or out.stride(1) != 1 or \
+            out.shape[0] < n or out.shape[1] < heads * vdim or q_start.numel() < n_requests + 1 or \
+            state_slot.numel() < n_requests or positions.numel() < n:
+        raise KernelArgumentError(f"{what}: shapes do not fit")
+    _check(lib().prb_gla_step(_p(out), out.stride(0), _p(proj), proj.stride(0), q, k, v, lr, g, _p(w2t),
+                              _p(bias), 1.0 / float(tau), float(q_scale), _p(norm_w), float(eps),
+                              float(out_scale), _p(state), _p(q_start), _p(state_slot), _p(positions), n,
+                              int(n_requests), int(heads), int(dim), int(vdim), rank, state.shape[0],
+                              dtype_code(out.dtype), _p(status), _stream()), what)
+
+
+# ------------------------------------------------ the state-space mixer
+def ssm_max_taps() -> int:
+    return int(lib().prb_ssm_max_taps())
+
+
+def ssm_chunk_supports(vdim: int, dim: int) -> bool:
+    """Whether the tensor-core kernels (:meth:`StateSpace.chunks`) take heads of these sizes."""
+    return bool(lib().prb_ssm_chunk_supports(int(vdim), int(dim)))
+
+
+def ssm_step_supports(vdim: int, dim: int) -> bool:
+    return bool(lib().prb_ssm_step_supports(int(vdim), int(dim)))
+
+
+class StateSpace:
+    """What the state-space kernels of one step have in common: the projection and its first columns
+    (``cols``: z, the convolved channels [x | B | C], dt), the layer's 32-bit weights (``conv_w`` [taps,
+    channels], ``conv_b`` [channels], ``dt_bias``, ``neg_a`` = -exp(A_log) and ``direct`` [heads],
+    ``norm_w`` [heads * vdim]), the request states, the step's description, ``raw`` float32 [T, heads *
+    vdim] and ``out`` in the activation type."""
+
+    def __init__(self, proj, cols, conv_w, conv_b, dt_bias, neg_a, direct, norm_w, conv_state, state,
+                 seq_of_token, q_start, state_slot, positions, n_requests: int, heads: int, vdim: int,
+                 dim: int, groups: int, parts: int, eps: float, out_scale: float, raw, out, status=None):
+        what = "state_space"
+        _columns_of(proj, what)
+        taps, channels = conv_w.shape
+        inner = heads * vdim
+        n = proj.shape[0]
+        for name, t, size in (("conv_w", conv_w, taps * channels), ("conv_b", conv_b, channels),
+                              ("dt_bias", dt_bias, heads), ("neg_a", neg_a, heads),
+                              ("direct", direct, heads), ("norm weight", norm_w, inner)):
+            _need(t, torch.float32, name, what)
+            if t.numel() != size:
+                raise KernelArgumentError(f"{what}: {name} must hold {size} numbers")
+        for name, t, size in (("seq_of_token", seq_of_token, n), ("q_start", q_start, n_requests + 1),
+                              ("state_slot", state_slot, n_requests), ("positions", positions, n)):
+            _need(t, torch.int32, name, what)
+            if t.numel() < size:
+                raise KernelArgumentError(f"{what}: {name} is too short")
+        _need(state, torch.float32, "state", what)
+        _need(raw, torch.float32, "raw", what)
+        z, x, dt = (int(c) for c in cols)
+        if heads % groups or inner % parts or channels != inner + 2 * groups * dim or \
+                tuple(state.shape[1:]) != (heads, vdim, dim) or max(z + inner, x + channels, dt + heads) > \
+                proj.shape[1] or raw.shape[0] < n or raw.shape[1] < inner or out.stride(1) != 1 or \
+                out.shape[0] < n or out.shape[1] < inner:
+            raise KernelArgumentError(f"{what}: shapes do not fit")
+        if taps > 1:
+            _need(conv_state, torch.float32, "saved inputs", what)
+            if tuple(conv_state.shape) != (state.shape[0], taps - 1, channels):
+                raise KernelArgumentError(f"{what}: the saved inputs have the wrong shape")
+        else:
+            conv_state = None
+        self.n, self.heads, self.channels, self.out_dtype = n, heads, channels, dtype_code(out.dtype)
+        self.vdim, self.dim, self.n_requests = vdim, dim, n_requests
+        self._args = (_p(proj), proj.stride(0), z, x, dt, _p(conv_w), _p(conv_b), _p(dt_bias), _p(neg_a),
+                      _p(direct), _p(conv_state), _p(state), _p(seq_of_token), _p(q_start), _p(state_slot),
+                      _p(positions), n, int(n_requests), int(heads), int(vdim), int(dim), int(groups), taps,
+                      state.shape[0], _p(raw), raw.stride(0), _p(norm_w), int(parts), float(eps),
+                      float(out_scale), _p(out), out.stride(0), _p(status))
+
+    def prepare(self, xbc, dt, decay, as_log: bool) -> None:
+        """Convolution and silu into ``xbc`` [T, >= channels]; step sizes and log decays (``as_log``)
+        or decays minus one, float32 [T, heads]."""
+        what = "ssm_prepare"
+        for name, t in (("dt", dt), ("decay", decay)):
+            _need(t, torch.float32, name, what)
+            if t.numel() < self.n * self.heads:
+                raise KernelArgumentError(f"{what}: {name} is too short")
+        if not xbc.is_cuda or xbc.stride(1) != 1 or xbc.shape[0] < self.n or xbc.shape[1] < self.channels:
+            raise KernelArgumentError(f"{what}: xbc has the wrong shape")
+        _check(lib().prb_ssm_prepare(*self._args, _p(xbc), xbc.stride(0), dtype_code(xbc.dtype), _p(dt),
+                                     _p(decay), 1 if as_log else 0, _stream()), what)
+
+    def chunks(self, xbc, dt, log_decay, own, start_hi, start_lo, seg_decay) -> None:
+        """The recurrence in segments on tensor cores: ``raw`` = (S^T C + D x) silu(z).  Workspaces: own
+        float32 and start_hi, start_lo bfloat16 [segments, heads, vdim, dim], seg_decay [segments, heads]."""
+        what = "ssm_chunks"
+        for name, t, dt_ in (("own", own, torch.float32), ("start_hi", start_hi, torch.bfloat16),
+                             ("start_lo", start_lo, torch.bfloat16), ("seg_decay", seg_decay, torch.float32),
+                             ("dt", dt, torch.float32), ("log_decay", log_decay, torch.float32)):
+            _need(t, dt_, name, what)
+        n = own.shape[0]
+        size = n * self.heads * self.vdim * self.dim
+        if xbc.dtype != torch.bfloat16 or min(own.numel(), start_hi.numel(), start_lo.numel()) < size or \
+                seg_decay.numel() < n * self.heads:
+            raise KernelArgumentError(f"{what}: workspaces of the wrong shape or type")
+        _check(lib().prb_ssm_chunks(*self._args, _p(xbc), xbc.stride(0), _p(dt), _p(log_decay), _p(own),
+                                    _p(start_hi), _p(start_lo), _p(seg_decay), n, _stream()), what)
+        add_launches(2)
+
+    def finish(self, gated: bool) -> None:
+        """``out`` = the norm in parts of ``raw`` (times silu(z) first unless ``gated``), times its
+        weight; the saved inputs are brought up to date."""
+        _check(lib().prb_ssm_finish(*self._args, 0 if gated else 1, self.out_dtype, _stream()), "ssm_finish")
+
+    def step(self, arrived) -> None:
+        """A step in which every request brings one token, in one launch; ``arrived``: int32 zeros, one
+        per request, left zero."""
+        _need(arrived, torch.int32, "arrived", "ssm_step")
+        if arrived.numel() < self.n_requests:
+            raise KernelArgumentError("ssm_step: one counter per request")
+        _check(lib().prb_ssm_step(*self._args, _p(arrived), self.out_dtype, _stream()), "ssm_step")

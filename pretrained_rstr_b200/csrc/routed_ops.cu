@@ -1,7 +1,7 @@
 // Small kernels of designs that scale their embedding, re-inject it, and route tokens to
 // experts by independent scores:
 //   * token embedding times a constant, optionally kept a second time (a stream that is
-//     joined by its own beginning again later);
+//     joined by its own beginning again later), or normed;
 //   * a router by scores: z in 32-bit, s = sigmoid(z) (or z itself), the `top` largest, their
 //     scores as weights, optionally divided by their sum;
 //   * the activation of routed experts whose weight multiplies the expert's INPUT:
@@ -44,6 +44,34 @@ __global__ void embed_scaled_kernel(float* __restrict__ out, float* __restrict__
         if (k) k[i] = v;
         if (pr) pr[i] = pr[width + i] = prb_from_float<W>(v);
     }
+}
+
+// ------------------------------------------------------------------ normed embedding
+// The token's row brought to unit root-mean-square times a weight per coordinate; a CTA a token.
+template <typename W>
+__global__ void embed_norm_kernel(float* __restrict__ out, const int* __restrict__ tokens,
+                                  const W* __restrict__ table, const float* __restrict__ weight,
+                                  int n_tokens, int width, int vocab, float eps, int* status) {
+    __shared__ float scratch[32];
+    prb_grid_launch_dependents();
+    const int t = blockIdx.x;
+    const int tok = tokens[t];
+    float* o = out + (size_t)t * width;
+    if (tok < 0 || tok >= vocab) {
+        if (threadIdx.x == 0) prb_set_status(status, PRB_S_TOKEN_RANGE, t, tok, vocab);
+        for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = 0.0f;
+        return;
+    }
+    const W* e = table + (size_t)tok * width;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = prb_to_float<W>(e[i]);
+        ss = fmaf(v, v, ss);
+    }
+    ss = prb_block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x)
+        o[i] = prb_to_float<W>(e[i]) * inv * weight[i];
 }
 
 // ------------------------------------------------------------------ router by scores
@@ -273,6 +301,24 @@ PRB_API int prb_embed_scaled(float* out, float* keep, const int* tokens, const v
         embed_scaled_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
             out, keep, tokens, (const __nv_bfloat16*)table, n_tokens, width, vocab, scale,
             (__nv_bfloat16*)pair, pair_ld, status);
+    else
+        return PRB_E_DTYPE;
+    PRB_LAUNCH_CHECK();
+    return 0;
+}
+
+PRB_API int prb_embed_norm(float* out, const int* tokens, const void* table, const float* weight,
+                           int n_tokens, int width, int vocab, float eps, int table_dtype, int* status,
+                           cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (width <= 0 || vocab <= 0 || weight == nullptr) return PRB_E_SIZE;
+    const int threads = width >= 256 ? 256 : ((width + 31) / 32) * 32;
+    if (table_dtype == PRB_F32)
+        embed_norm_kernel<float><<<n_tokens, threads, 0, stream>>>(out, tokens, (const float*)table, weight,
+                                                                   n_tokens, width, vocab, eps, status);
+    else if (table_dtype == PRB_BF16)
+        embed_norm_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
+            out, tokens, (const __nv_bfloat16*)table, weight, n_tokens, width, vocab, eps, status);
     else
         return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();

@@ -18,7 +18,8 @@
 // every pass, and read before they write); in a step with portions they are read by a portion's
 // first tokens while they would be written from its last, so wattn_conv_state does it afterwards.
 //
-// rotary_angles: cosine and sine of every token's angles once per step, for all layers and heads.
+// rotary_angles: cosine and sine of every token's angles, times one magnitude, once per step, for
+//   all layers and heads.
 // All arithmetic is 32-bit, the angles' products 64-bit.
 #include "common.cuh"
 
@@ -307,24 +308,24 @@ __global__ void wattn_conv_state_kernel(PrepArgs a) {
 
 __global__ void rotary_angles_kernel(float2* __restrict__ out, const int* __restrict__ positions,
                                      const float* __restrict__ freq, const float* __restrict__ freq_lo,
-                                     int n_tokens, int half) {
+                                     int n_tokens, int half, float magnitude) {
     prb_grid_launch_dependents();
     const long e = (long)blockIdx.x * blockDim.x + threadIdx.x;
     if (e >= (long)n_tokens * half) return;
     const int t = (int)(e / half), i = (int)(e - (long)t * half);
     float sn, cs;
     prb_sincos_angle((float)positions[t], freq[i], &sn, &cs, freq_lo ? freq_lo[i] : 0.0f);
-    out[e] = make_float2(cs, sn);
+    out[e] = make_float2(cs * magnitude, sn * magnitude);
 }
 }  // namespace
 
 PRB_API int prb_rotary_angles(void* out, const int* positions, const float* freq, const float* freq_lo,
-                              int n_tokens, int half, cudaStream_t stream) {
+                              int n_tokens, int half, float magnitude, cudaStream_t stream) {
     if (n_tokens <= 0 || half <= 0) return 0;
     if (((uintptr_t)out) % 8 != 0) return PRB_E_ALIGN;
     const long total = (long)n_tokens * half;
     rotary_angles_kernel<<<(unsigned)((total + 127) / 128), 128, 0, stream>>>(
-        (float2*)out, positions, freq, freq_lo, n_tokens, half);
+        (float2*)out, positions, freq, freq_lo, n_tokens, half, magnitude);
     PRB_LAUNCH_CHECK();
     return 0;
 }

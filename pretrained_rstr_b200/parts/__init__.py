@@ -1,6 +1,7 @@
-from . import (attention, block, differential_attention, embedding, feed_forward, head,  # noqa: F401  (register)
-               latent_attention, linear_recurrence, matrix_memory, norms, positions, retention,
-               side_by_side, stream_join, time_mix, window_attention)
+from . import (attention, block, differential_attention, embedding, feed_forward,  # noqa: F401  (register)
+               gated_linear_attention, head, latent_attention, linear_recurrence, matrix_memory,
+               norms, positions, retention, side_by_side, state_space, stream_join, time_mix,
+               window_attention)
 from .interfaces import (Block, Embedding, FeedForward, Head, KVSpec, LayerCache, Mixer, Norm,
                          PositionEncoding, StateSpec)
 from .linear import Linear

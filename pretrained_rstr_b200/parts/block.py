@@ -138,20 +138,53 @@ class ParallelBlock(Block):
     32-bit.  The mixer's norm runs first; the feed-forward then reads the untouched stream
     (its norm may ride in its first matrix product, see :class:`LazyNorm`) and adds its
     result, and the mixer, which works from its normed copy, adds its own after that.  A
-    layer without a feed-forward has the mixer's norm alone."""
+    layer without a feed-forward has the mixer's norm alone.
+
+    With ONE norm (``norms`` = {"shared"}) both branches read its result: x <- x + (mixer(h) +
+    feed_forward(h)), h = norm(x).  Branches that offer their products (``products``: the fused first
+    product and the product that ends them) then share both: one product reads h for all of the
+    layer's projections, and one brings all of its results to the stream; the norm may ride in the
+    first (the stream stays as it was until the last)."""
     graph_safe = True
 
     def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Dict[str, Norm],
                  width: int, runtime):
         self.has_ff = not getattr(feed_forward, "is_none", False)
+        self.shared = set(norms) == {"shared"}
         wanted = {"mixer", "feed_forward"} if self.has_ff else {"mixer"}
-        if set(norms) != wanted:
-            raise ValueError(f"parallel wants the norms {sorted(wanted)}, got {sorted(norms)}")
+        if not self.shared and set(norms) != wanted:
+            raise ValueError(f"parallel wants the norms {sorted(wanted)} or ['shared'], got {sorted(norms)}")
         self.mixer, self.feed_forward = mixer, feed_forward
         self.norms = dict(norms)
         self.width, self.runtime = width, runtime
+        self.result = None                  # the branches' common last product, if they have one
+        if self.shared and self.has_ff:
+            mine = getattr(mixer, "products", lambda: None)()
+            theirs = getattr(feed_forward, "products", lambda: None)()
+            if mine is not None and theirs is not None:
+                mine[0].absorb(theirs[0])
+                mine[1].absorb(theirs[1])
+                self.result = mine[1]
+                self.result.closer = self
+
+    def _forward_shared(self, ctx, x, cache: LayerCache) -> None:
+        h = ctx.scratch("block_normed", (ctx.token_capacity, self.width), self.runtime.dtype)[:x.shape[0]]
+        norm = self.norms["shared"]
+        if self.result is not None or not self.has_ff:
+            h_in = PreNormBlock._normed(ctx, self.mixer, norm, x, h)
+            self.mixer.forward(ctx, h_in, x, cache)
+            if self.has_ff:
+                self.feed_forward.forward(ctx, h_in, x)
+                self.result.close(ctx, x)
+            return
+        norm.forward(ctx, x, h)
+        self.mixer.forward(ctx, h, x, cache)
+        self.feed_forward.forward(ctx, h, x)
 
     def forward(self, ctx, x, cache: LayerCache) -> None:
+        if self.shared:
+            self._forward_shared(ctx, x, cache)
+            return
         t = x.shape[0]
         cap = ctx.token_capacity
         h1 = ctx.scratch("block_normed", (cap, self.width), self.runtime.dtype)[:t]

@@ -46,6 +46,25 @@ class ScaledTokenEmbedding(Embedding):
                          pair=pair)
 
 
+class NormedTokenEmbedding(Embedding):
+    """x[t] = r / sqrt(mean(r^2) + eps) * (offset + weight) with r = table[token[t]]."""
+    graph_safe = True
+
+    def __init__(self, table: torch.Tensor, weight: torch.Tensor, vocab: int, width: int, eps: float,
+                 offset: float, runtime):
+        if tuple(table.shape) != (vocab, width) or weight.numel() != width:
+            raise ValueError(f"normed_token_embedding: table is {list(table.shape)} with {weight.numel()} "
+                             f"weights, expected [{vocab}, {width}]")
+        self.table = table.to(runtime.dtype).contiguous()
+        self.weight = (weight.to(torch.float32) + float(offset)).contiguous()
+        self.vocab, self.width, self.eps = vocab, width, float(eps)
+
+    def forward(self, ctx, position, x) -> None:
+        if position.table() is not None:
+            raise ValueError("normed_token_embedding adds no position table")
+        ops.embed_norm(x, ctx.tokens, self.table, self.weight, self.eps, ctx.status)
+
+
 class TokenPairEmbedding(Embedding):
     """x[t] = table[token] * scale + pairs[row]: a second table indexed by a hash of (previous token,
     token), row = (prev * mul_prev + token * mul_cur) mod buckets; a sequence's first token
@@ -88,6 +107,10 @@ register_part("embedding", "token_embedding",
 register_part("embedding", "scaled_token_embedding",
               lambda p, store, rt: ScaledTokenEmbedding(
                   store.get(p["weights"], rt.dtype), p["vocab"], p["width"], p["scale"], rt))
+register_part("embedding", "normed_token_embedding",
+              lambda p, store, rt: NormedTokenEmbedding(
+                  store.get(p["weights"], rt.dtype), store.get(p["norm"]), p["vocab"], p["width"],
+                  p["eps"], p.get("offset", 0.0), rt))
 register_part("embedding", "token_pair_embedding",
               lambda p, store, rt: TokenPairEmbedding(
                   store.get(p["table"], rt.dtype), store.get(p["pairs"], rt.dtype), p["vocab"],

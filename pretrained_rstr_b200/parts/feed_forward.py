@@ -7,7 +7,7 @@ import torch
 
 from ..csrc import ops
 from .interfaces import FeedForward
-from .linear import Linear, padded_linear
+from .linear import LazyNorm, Linear, ResultProduct, padded_linear
 from .registry import register_part
 
 
@@ -49,6 +49,34 @@ class NoFeedForward(FeedForward):
     def forward(self, ctx, h, x, accumulate: bool = True) -> None:
         if not accumulate:
             x.zero_()
+
+
+class ActMLP(FeedForward):
+    """down(act(up(h))) without biases.  Unlike :class:`DenseMLP`, whose activation is its first
+    product's epilogue, the first product is a fused one with a 32-bit result, so that it (and the
+    last) can be shared with a mixer that reads the same input (:meth:`products`)."""
+    graph_safe = True
+    can_overwrite = True
+    accepts_lazy_norm = True      # the first matrix product may compute the norm itself
+
+    def __init__(self, up, down, width: int, inner: int, activation: str, runtime):
+        from .latent_attention import FusedInput
+        if tuple(up.shape) != (inner, width) or tuple(down.shape) != (width, inner):
+            raise ValueError("act_mlp: matrices have the wrong shape")
+        if activation not in ops.ROUTED_ACT_CODES:
+            raise ValueError(f"act_mlp: unknown activation {activation!r}")
+        self.input = FusedInput(width, runtime, "mlp_in")
+        self.input.add("up", up)
+        self.down = ResultProduct(down, runtime, "mlp_act")
+        self.activation = activation
+
+    def products(self):
+        return self.input, self.down
+
+    def forward(self, ctx, h, x, accumulate: bool = True) -> None:
+        proj = self.input.run(ctx, h)
+        ops.act_columns(self.down.buffer(ctx, x.shape[0]), self.input.view(proj, "up"), self.activation)
+        self.down.run(ctx, x, accumulate)
 
 
 class GatedMLP(FeedForward):
@@ -103,6 +131,11 @@ class GatedMoE(FeedForward):
     softmax over the chosen logits alone; "softmax", the chosen experts' shares of the softmax
     over ALL experts (``renormalize``: divided by their sum), times ``router_scale``.
 
+    With "softmax" scores: ``identity`` more experts of the router have no matrices, their output is
+    the input itself; ``correction`` (a weight, one number per expert) joins the scores for the choice
+    alone; ``shared_gate`` (weight ``shared.sg``, one row) multiplies the shared expert by its sigmoid.
+    Any of the three has scores, choice, activations and identity experts in one launch.
+
     All experts' gate and up rows, the shared expert's, the router's and whatever an
     arrangement fuses in are ONE matrix product; the activations of experts a token did not
     choose are multiplied by zero and those it chose by their weight, and one product with all
@@ -124,7 +157,16 @@ class GatedMoE(FeedForward):
         self.router_scale = float(p.get("router_scale", 1.0))
         if self.score not in ("softmax_chosen", "softmax"):
             raise ValueError(f"gated_moe: unknown score {self.score!r}")
-        if not 1 <= self.top <= n:
+        self.identity = int(p.get("identity") or 0)
+        self.correction = None
+        #: scores, choice and activations in one launch
+        self.one_launch = bool(self.identity or p.get("correction") or p.get("shared_gate"))
+        if self.one_launch and (self.score != "softmax" or self.limit or self.shared_limit or
+                                self.act_alpha != 1.0 or self.up_shift):
+            raise ValueError("gated_moe: identity experts, corrections and a gated shared expert go with "
+                             "softmax scores and plain SiLU gates")
+        n_all = n + self.identity
+        if not 1 <= self.top <= n_all:
             raise ValueError(f"gated_moe: top {self.top} of {n} experts")
         self.runtime = runtime
         pre = p["prefix"]
@@ -139,16 +181,24 @@ class GatedMoE(FeedForward):
         self.input.add("gate", torch.cat([need(f"e{e}.gate", (inner, width)) for e in range(n)]))
         self.input.add("up", torch.cat([need(f"e{e}.up", (inner, width)) for e in range(n)]))
         downs = [need(f"e{e}.down", (width, inner)) for e in range(n)]
+        self.shared_gated = bool(self.shared_inner and p.get("shared_gate"))
         if self.shared_inner:
             self.input.add("shared_gate", need("shared.gate", (self.shared_inner, width)))
             self.input.add("shared_up", need("shared.up", (self.shared_inner, width)))
             downs.append(need("shared.down", (width, self.shared_inner)))
-        self.input.add("router", need("router", (n, width)))
+            if self.shared_gated:
+                self.input.add("shared_weight", need("shared.sg", (1, width)))
+        self.input.add("router", need("router", (n_all, width)))
+        if p.get("correction"):
+            self.correction = need("correction", (n_all,)).to(torch.float32).contiguous()
         self.router_bias = need("router.b", (n,)).to(torch.float32).contiguous() \
             if p.get("router_bias", True) else None
         if self.score == "softmax" and self.router_bias is not None:
             raise ValueError("gated_moe: the softmax over all experts takes no router bias")
-        self.down = padded_linear(torch.cat(downs, dim=1), runtime)
+        self.down = ResultProduct(torch.cat(downs, dim=1), runtime, "moe_act")
+
+    def products(self):
+        return self.input, self.down
 
     def fuse_input_rows(self, name: str, weight) -> str:
         return self.input.add(name, weight)
@@ -156,7 +206,32 @@ class GatedMoE(FeedForward):
     def fused_rows(self, name: str):
         return self.input.view(self._proj, name)
 
+    def _forward_one_launch(self, ctx, h, x, accumulate: bool) -> None:
+        proj = self._proj = self.input.run(ctx, h)
+        at = lambda name: self.input.cols[name][0]
+        shared = None
+        if self.shared_inner:
+            shared = (at("shared_gate"), at("shared_up"), self.shared_inner,
+                      at("shared_weight") if self.shared_gated else -1)
+        stream = None
+        if self.identity:
+            # the input itself: as a tensor, or worked out from a stream that is still what the norm read
+            lazy = accumulate and isinstance(h, LazyNorm) and not h.done and h.fusable and \
+                h.rows is None and h.x is x and not getattr(h.norm, "centred", True)
+            stream = (x, (h.norm.gamma, h.norm.eps) if lazy else
+                      h.tensor() if isinstance(h, LazyNorm) else h)
+            if not accumulate:
+                x.zero_()
+        ops.expert_act(self.down.buffer(ctx, x.shape[0]), proj, at("gate"), at("up"), at("router"),
+                       self.experts, self.top, self.inner, identity=self.identity,
+                       correction=self.correction, renormalize=self.renormalize,
+                       factor=self.router_scale, shared=shared, stream=stream)
+        self.down.run(ctx, x, accumulate or bool(self.identity))
+
     def forward(self, ctx, h, x, accumulate: bool = True) -> None:
+        if self.one_launch:
+            self._forward_one_launch(ctx, h, x, accumulate)
+            return
         t = x.shape[0]
         cap = ctx.token_capacity
         proj = self._proj = self.input.run(ctx, h)
@@ -172,7 +247,7 @@ class GatedMoE(FeedForward):
             ops.route(scale, chosen, chosen_w, self.input.view(proj, "router"), None,
                       self.router_bias, self.top)
         n_act = self.experts * self.inner
-        a = ctx.scratch_zero("moe_act", (cap, self.down.n_in), self.runtime.dtype)[:t]
+        a = self.down.buffer(ctx, t)
         ops.gated_pair(a, proj, cols["gate"][0], cols["up"][0], n_act, limit=self.limit,
                        act_alpha=self.act_alpha, up_shift=self.up_shift, scale=scale,
                        group=self.inner)
@@ -180,7 +255,7 @@ class GatedMoE(FeedForward):
             ops.gated_pair(a, proj, cols["shared_gate"][0], cols["shared_up"][0],
                            self.shared_inner, out_col=n_act, limit=self.shared_limit,
                            act_alpha=self.act_alpha, up_shift=self.up_shift)
-        self.down.forward(ctx, a, x, resid=x if accumulate else None)
+        self.down.run(ctx, x, accumulate)
 
 
 class RoutedExperts(FeedForward):
@@ -254,6 +329,9 @@ def _gated_mlp(p, store, rt) -> GatedMLP:
 
 
 register_part("feed_forward", "dense_mlp", _dense_mlp)
+register_part("feed_forward", "act_mlp",
+              lambda p, store, rt: ActMLP(store.get(p["weights"]["up"]), store.get(p["weights"]["down"]),
+                                          p["width"], p["inner"], p["activation"], rt))
 register_part("feed_forward", "gated_mlp", _gated_mlp)
 register_part("feed_forward", "gated_moe", lambda p, store, rt: GatedMoE(p, store, rt))
 register_part("feed_forward", "routed_experts", lambda p, store, rt: RoutedExperts(p, store, rt))

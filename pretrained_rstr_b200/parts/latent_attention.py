@@ -57,15 +57,38 @@ def _pad8(n: int) -> int:
 class FusedInput:
     """One matrix product for several consumers of the same input: segments of rows, each
     starting at a multiple of 8 columns of the float32 result.  Segments are added while the
-    model is built; the matrix is put together at the first use."""
+    model is built; the matrix is put together at the first use.
+
+    Two parts that read the same input can have one product: ``a.absorb(b)`` moves b's segments
+    into a; b.run then hands out the result of a's product, which has to run before it."""
 
     def __init__(self, width: int, runtime, key: str):
         self.width, self.runtime, self.key = width, runtime, key
         self._parts: List[Tuple[str, torch.Tensor]] = []
         self.cols: Dict[str, Tuple[int, int]] = {}          # name -> (first column, columns)
         self._linear: Optional[Linear] = None
+        self.host: Optional["FusedInput"] = None            # whose product this one's rows ride in
+        self._guests: List[Tuple[str, "FusedInput"]] = []   # (prefix of its segments' names, guest)
+        self._result: Optional[torch.Tensor] = None         # of the step that runs
+
+    def absorb(self, other: "FusedInput") -> None:
+        """Take over ``other``'s segments (and what is added to it from now on)."""
+        if other is self or other.host is not None or self.host is not None or \
+                other._linear is not None or self._linear is not None:
+            raise RuntimeError("fused products can be joined once, before they are built")
+        if other.width != self.width:
+            raise ValueError(f"fused products over {self.width} and {other.width} inputs")
+        prefix = f"{other.key}.{len(self._guests)}."
+        other.host = self
+        self._guests.append((prefix, other))
+        for name, w in other._parts:
+            self.add(prefix + name, w)
+        other._parts = []
 
     def add(self, name: str, weight: torch.Tensor) -> str:
+        if self.host is not None:
+            self.host.add(next(p for p, g in self.host._guests if g is self) + name, weight)
+            return name
         if self._linear is not None:
             raise RuntimeError("the fused product is built already")
         if weight.dim() != 2 or weight.shape[1] != self.width:
@@ -86,13 +109,19 @@ class FusedInput:
                 at += w.shape[0] + pad
             self._linear = Linear(torch.cat(rows, dim=0), None, self.runtime)
             self._parts = []
+            for prefix, guest in self._guests:
+                guest.cols.update({name[len(prefix):]: at for name, at in self.cols.items()
+                                   if name.startswith(prefix)})
         return self._linear
 
     def run(self, ctx, h) -> torch.Tensor:
+        if self.host is not None:
+            return self.host._result
         lin = self.linear()
         t = h.shape[0]
         out = ctx.scratch(self.key, (ctx.token_capacity, lin.n_out), torch.float32)[:t]
         lin.forward(ctx, h, out)
+        self._result = out
         return out
 
     def view(self, out: torch.Tensor, name: str) -> torch.Tensor:

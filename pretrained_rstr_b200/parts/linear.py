@@ -106,6 +106,77 @@ def padded_linear(weight: torch.Tensor, runtime) -> Linear:
     return Linear(weight, None, runtime)
 
 
+class ResultProduct:
+    """The matrix product a part ends with: x (+)= r . W^T + b, from a buffer of its own that the
+    part fills (:meth:`buffer`, then :meth:`run`).
+
+    Results that join the same stream can share one product: ``a.absorb(b)`` puts b's matrix beside
+    a's (a row of the common buffer is [r_a | r_b]; biases add up), ``b.run`` then does nothing, and
+    whoever joined them sets ``a.closer`` and calls :meth:`close` when all have filled their
+    columns.  Segments start at multiples of 8 columns; the columns between stay zero."""
+
+    def __init__(self, weight: torch.Tensor, runtime, key: str, bias: Optional[torch.Tensor] = None):
+        self.runtime, self.key = runtime, key
+        self.n_out = int(weight.shape[0])
+        self.parts = [(weight, bias)]
+        self.host: Optional["ResultProduct"] = None
+        self.column = 0                        # first column in the common buffer
+        self.columns = -(-int(weight.shape[1]) // 8) * 8
+        self.total = self.columns              # (of all that share the product)
+        self.closer = None                     # who runs the common product, or None: run() does
+        self._linear: Optional[Linear] = None
+
+    def absorb(self, other: "ResultProduct") -> None:
+        if other is self or self.host is not None or other.host is not None or \
+                self._linear is not None or other._linear is not None:
+            raise RuntimeError("result products can be joined once, before they are built")
+        if other.n_out != self.n_out:
+            raise ValueError(f"result products of {self.n_out} and {other.n_out} outputs")
+        for guest in [other] + getattr(other, "guests", []):
+            guest.host = self
+            guest.column += self.total
+        self.guests = getattr(self, "guests", []) + [other] + getattr(other, "guests", [])
+        self.parts += other.parts
+        self.key = f"{self.key}+{other.key}"
+        self.total += other.total
+        other.parts = []
+
+    def linear(self) -> Linear:
+        if self._linear is None:
+            pieces, bias = [], None
+            for w, b in self.parts:
+                pieces.append(w.to(self.runtime.dtype))
+                pad = -w.shape[1] % 8
+                if pad:
+                    pieces.append(torch.zeros((w.shape[0], pad), dtype=self.runtime.dtype, device=w.device))
+                if b is not None:
+                    bias = b.to(torch.float32) if bias is None else bias + b.to(torch.float32)
+            # (the buffer's layout is part of its name: columns that stay zero lie elsewhere in another)
+            self.key += "/" + ",".join(str(int(w.shape[1])) for w, _b in self.parts)
+            self._linear = Linear(torch.cat(pieces, dim=1) if len(pieces) > 1 else pieces[0], bias,
+                                  self.runtime)
+            self.parts = []
+        return self._linear
+
+    def buffer(self, ctx, t: int) -> torch.Tensor:
+        """[t, columns] in the activation type: the part writes its real columns."""
+        host = self.host or self
+        host.linear()
+        rows = ctx.scratch_zero(host.key, (ctx.token_capacity, host.total), self.runtime.dtype)[:t]
+        return rows if host.total == self.columns else rows[:, self.column:self.column + self.columns]
+
+    def run(self, ctx, x: torch.Tensor, accumulate: bool = True) -> None:
+        if self.host is None and self.closer is None:
+            self.close(ctx, x, accumulate)
+
+    def close(self, ctx, x: torch.Tensor, accumulate: bool = True) -> None:
+        if self.host is not None:
+            return
+        lin = self.linear()
+        rows = ctx.scratch_zero(self.key, (ctx.token_capacity, self.total), self.runtime.dtype)[:x.shape[0]]
+        lin.forward(ctx, rows, x, resid=x if accumulate else None)
+
+
 class LazyNorm:
     """A norm of ``x`` (of its rows ``rows``, if given: an int32 tensor of row indices) that
     runs when its result is first needed.  A consumer that can compute the norm itself
@@ -121,6 +192,10 @@ class LazyNorm:
         self.fusable = all(hasattr(norm, f) for f in ("gamma", "beta", "eps")) and \
             getattr(norm, "kind", "") in ("layer_norm", "rms_norm") and norm.gamma is not None
         self.shape = out.shape
+
+    @property
+    def done(self) -> bool:
+        return self._done
 
     def tensor(self) -> torch.Tensor:
         if not self._done:

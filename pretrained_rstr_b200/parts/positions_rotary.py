@@ -85,12 +85,13 @@ def banded_frequencies(base: float, dims: int, factor: float, low: float, high: 
 
 
 class RotaryAngles:
-    """Cosines and sines of every token's angles, computed once per step and shared by all layers,
-    heads and passes whose frequencies are the same."""
+    """Cosines and sines of every token's angles, times one ``magnitude``, computed once per step and
+    shared by all layers, heads and passes whose frequencies and magnitude are the same."""
 
-    def __init__(self, freq, freq_lo):
-        self.freq, self.freq_lo = freq, freq_lo
-        mark = hashlib.sha256(freq.cpu().numpy().tobytes() + freq_lo.cpu().numpy().tobytes())
+    def __init__(self, freq, freq_lo, magnitude: float = 1.0):
+        self.freq, self.freq_lo, self.magnitude = freq, freq_lo, float(magnitude)
+        mark = hashlib.sha256(freq.cpu().numpy().tobytes() + freq_lo.cpu().numpy().tobytes() +
+                              repr(self.magnitude).encode())
         self.key = f"rotary_angles_{mark.hexdigest()[:16]}"
 
     def table(self, ctx, rows: int):
@@ -99,6 +100,6 @@ class RotaryAngles:
         out = done.get(self.key)
         if out is None:
             out = ctx.scratch(self.key, (ctx.token_capacity, self.freq.numel(), 2), torch.float32)[:rows]
-            ops.rotary_angles(out, ctx.positions, self.freq, self.freq_lo)
+            ops.rotary_angles(out, ctx.positions, self.freq, self.freq_lo, self.magnitude)
             done[self.key] = out
         return out

@@ -8,7 +8,9 @@ its projections in one fused product and offers room in it (``fuse_input_rows``)
 child can take its own from a host (``takes_input_host``), the second child's projections ride
 in the first child's product: one product a layer reads the stream for both (``input_host`` is
 offered to every second child; one that keeps a product of its own over another input ignores
-it).  ``share_product`` False keeps the products apart."""
+it).  ``share_product`` False keeps the products apart.  Children that end in a
+:class:`~pretrained_rstr_b200.parts.linear.ResultProduct` (``products``) share that too: one product
+brings both results to the stream."""
 from __future__ import annotations
 
 from .interfaces import LayerCache, Mixer
@@ -36,6 +38,21 @@ class SideBySide(Mixer):
         for c in self.children:
             if not getattr(c, "can_overwrite", False):
                 raise ValueError(f"side_by_side: {type(c).__name__} cannot start a sum")
+        first, second = self.children
+        self.result = None                 # the children's common last product, if they have one
+        if hasattr(first, "products") and hasattr(second, "products") and p.get("share_product", True):
+            self.result = first.products()[1]
+            self.result.absorb(second.products()[1])
+            self.result.closer = self
+        # (the second child then never reads the input itself)
+        self.accepts_lazy_norm = getattr(first, "accepts_lazy_norm", False) and \
+            getattr(second, "host", None) is not None
+
+    def products(self):
+        """(input product, result product) both children ride in, or None."""
+        if self.result is None or getattr(self.children[1], "host", None) is None:
+            return None
+        return self.children[0].products()[0], self.result
 
     @property
     def graph_safe(self) -> bool:
@@ -57,6 +74,8 @@ class SideBySide(Mixer):
         first, second = self.children
         first.forward(ctx, h, x, cache, accumulate=accumulate)
         second.forward(ctx, h, x, cache, accumulate=True)
+        if self.result is not None and self.result.closer is self:
+            self.result.close(ctx, x, accumulate)
 
 
 register_part("mixer", "side_by_side", lambda p, store, rt: SideBySide(p, store, rt))

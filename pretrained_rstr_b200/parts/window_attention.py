@@ -9,7 +9,9 @@ values ``vdim``.  Every option is a parameter, and a design names the ones it ha
 ``rot_dims`` / ``rot_base``  rotary positions on each head's first coordinates; ``rot_layout`` "half"
                       or "interleaved" (pairs (2i, 2i + 1)); ``rot_factor``: every frequency is
                       divided by it (linear scaling); ``rot_bands`` {factor, low, high, original}:
-                      frequencies scaled by their wavelength (see ``banded_frequencies``)
+                      frequencies scaled by their wavelength (see ``banded_frequencies``);
+                      ``rot_yarn`` {factor, original, fast, slow}: YaRN's frequencies, with its
+                      magnitude on cosines and sines (see ``yarn_frequencies``)
 ``conv``              a causal convolution over time on every channel of q and k, ``conv`` taps
                       long, without a bias (weights ``q_conv`` / ``k_conv``, [channels, taps]), before
                       norm and rotation.  The last taps - 1 projected values of a request are
@@ -21,7 +23,8 @@ values ``vdim``.  Every option is a parameter, and a design names the ones it ha
                       ``q_norm`` / ``k_norm``); "head": per head, before the rotation, with
                       weights of ``dim`` numbers that all heads share; "head_after": per head,
                       after the rotation, without weights
-``bias``              q, k and v have biases (weights ``q_bias`` / ``k_bias`` / ``v_bias``)
+``bias``              q, k and v have biases (weights ``q_bias`` / ``k_bias`` / ``v_bias``);
+                      ``out_bias``: so has the output projection (weight ``out_bias``)
 ``sink``              a learned number per head (weight ``sink``) whose exponential joins the
                       softmax's denominator once: it has no key and no value and is not scaled;
                       ``sink_score``: the same with one constant for all heads (0: the
@@ -52,9 +55,9 @@ import torch
 from ..csrc import ops
 from .interfaces import KVSpec, LayerCache, Mixer, StateSpec
 from .latent_attention import FusedInput
-from .linear import padded_linear
+from .linear import ResultProduct
 from .positions_rotary import (RotaryAngles, banded_frequencies, rotary_frequencies,
-                               split_frequencies)
+                               split_frequencies, yarn_frequencies)
 from .registry import register_part
 
 
@@ -142,7 +145,11 @@ class WindowAttention(Mixer):
         if self.taps:
             self.conv_w = tuple(need(n, (h * self.dim, self.taps)).to(torch.float32).contiguous()
                                 for n, h in (("q_conv", self.heads), ("k_conv", self.kv_heads)))
-        self.out = padded_linear(need("out", (self.width, self.heads * self.vdim)), runtime)
+        out_bias = None
+        if p.get("out_bias"):              # (the mixer's constant acts on the bias too)
+            out_bias = need("out_bias", (self.width,)).to(torch.float32) * self.out_scale
+        self.out = ResultProduct(need("out", (self.width, self.heads * self.vdim)), runtime, "wattn_out",
+                                 out_bias)
         self.slopes = None
         if p.get("slope_bits") is not None:
             bits = float(p["slope_bits"])
@@ -150,7 +157,14 @@ class WindowAttention(Mixer):
                                         for h in range(self.heads)],
                                        dtype=torch.float64).to(torch.float32).to(dev)
         base, bands = float(p.get("rot_base", 10000.0)), p.get("rot_bands")
-        if bands and self.rot_dims:
+        yarn, magnitude = p.get("rot_yarn"), 1.0
+        if yarn and mode in (True, "whole"):
+            raise ValueError("window_attention: a norm over whole projections goes with no stretched angles")
+        if yarn and self.rot_dims:
+            (self.freq, self.freq_lo), magnitude = yarn_frequencies(
+                base, self.rot_dims, float(yarn["factor"]), float(yarn["original"]), float(yarn["fast"]),
+                float(yarn["slow"]), dev, with_lo=True)
+        elif bands and self.rot_dims:
             self.freq, self.freq_lo = split_frequencies(
                 banded_frequencies(base, self.rot_dims, float(bands["factor"]), float(bands["low"]),
                                    float(bands["high"]), float(bands["original"])), dev)
@@ -158,7 +172,7 @@ class WindowAttention(Mixer):
             self.freq, self.freq_lo = rotary_frequencies(
                 base, self.rot_dims, dev, divide_by=float(p.get("rot_factor") or 1.0), with_lo=True)
         # (a norm over whole projections is another kernel, which computes its own angles)
-        self.rotary = RotaryAngles(self.freq, self.freq_lo) \
+        self.rotary = RotaryAngles(self.freq, self.freq_lo, magnitude) \
             if self.rot_dims and mode not in (True, "whole") else None
         gpu = torch.cuda.is_available()
         # kernels for bfloat16 cache rows: (portions, single tokens)
@@ -182,6 +196,10 @@ class WindowAttention(Mixer):
         rows = seen * self.kv_heads * (self.dim + self.vdim) * self.runtime.dtype.itemsize
         inputs = max(self.taps - 1, 0) * (self.heads + self.kv_heads) * self.dim
         return rows + 2 * 4 * inputs                 # (a convolution's saved inputs: read, written back)
+
+    def products(self):
+        """(the fused first product, the product that ends the mixer)."""
+        return self.input, self.out
 
     def fuse_input_rows(self, name: str, weight) -> str:
         return self.input.add(name, weight)
@@ -221,7 +239,7 @@ class WindowAttention(Mixer):
                           angles=self.rotary.table(ctx, t) if self.rotary else None,
                           interleaved=self.interleaved, keys_are_values=self.keys_are_values,
                           conv=conv)
-        o = ctx.scratch_zero("wattn_out", (cap, self.out.n_in), self.runtime.dtype)[:t]
+        o = self.out.buffer(ctx, t)
         # a step of single tokens: a CTA per (token, key/value head) whose warps share out the
         # key blocks (rows of different requests share no keys); sizes that kernel does not
         # take: the tiled kernel, a row a CTA.  Serving in bfloat16 has kernels of its own for
@@ -235,7 +253,7 @@ class WindowAttention(Mixer):
                   single=single and self.single_ok, sinks=self.sinks,
                   gate_per_value=self.value_gate, softcap=self.softcap,
                   bf16_kernels=self.bf16_ok[1 if single else 0])
-        self.out.forward(ctx, o, x, resid=x if accumulate else None)
+        self.out.run(ctx, x, accumulate)
 
 
 register_part("mixer", "window_attention", lambda p, store, rt: WindowAttention(p, store, rt))
