@@ -21,7 +21,9 @@
 namespace {
 using namespace dscan;
 constexpr int DS_TB = 16;            // tokens staged at a time
-constexpr int DS_THREADS = 512;
+constexpr int ds_threads(int kpl) { return kpl == 4 ? 512 : 256; }
+constexpr int DS_CC = 8;             // value columns a thread of the segmented passes holds
+constexpr int GS_CC = 4;             // and one of the single-token kernel
 
 struct Finish {
     void* out;                       // null: raw sums
@@ -63,9 +65,10 @@ __device__ __forceinline__ void finish_row(const Finish& f, const float* src, in
         o[j] = prb_from_float<O>(src[j] * inv * f.norm_w[j] * silu(gp[j]));
 }
 
-// MODE 1: a segment's own sums from zero; 2: a segment from its start with outputs.
+// MODE 1: a segment's own sums from zero; 2: a segment from its start with outputs.  Scales of the
+// keys and the direct path go with decays per head.
 template <int KPL, bool PER_KEY, int MODE, typename O>
-__global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
+__global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
     extern __shared__ __align__(16) float sm[];
     prb_grid_launch_dependents();
     const int hd = blockIdx.x, cg = blockIdx.z;
@@ -86,23 +89,24 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
     const int cw = PER_KEY ? dp : 4;
     const int stage = DS_TB * (2 * dp + cw + cols + 4);
     float* o_s = sm + 2 * stage;                     // [DS_TB][vdim], with the finish inside
-    const int ln = threadIdx.x % L, cl = threadIdx.x / L;
-    const int c0 = cg * cols + cl * DS_CC;           // this thread's first value column
-    const bool mine = cl * DS_CC < cols;
+    const int ln = threadIdx.x % L, cl = min((int)threadIdx.x / L * DS_CC, cols - DS_CC);
+    const int c0 = cg * cols + cl;                   // this thread's first value column
+    const bool mine = (int)threadIdx.x / L * DS_CC < cols;       // (threads beyond work along, and store nothing)
     const size_t per_head = (size_t)vdim * dim, per_state = (size_t)a.heads * per_head;
     float S[DS_CC][KPL], Pd[KPL];
-    load_state<KPL>(S, MODE == 2 && mine ? a.seg_start + (size_t)blockIdx.y * per_state + hd * per_head : nullptr,
-                    ln, c0, dim, vdim);
+    load_state<DS_CC, KPL>(S, MODE == 2 ? a.seg_start + (size_t)blockIdx.y * per_state + hd * per_head : nullptr,
+                           ln, c0, dim, vdim);
 #pragma unroll
     for (int i = 0; i < KPL; ++i) Pd[i] = 0.0f;
     const float* qb = a.q + (size_t)(hd / a.q_share) * dim;
     const float* kb = a.k + (size_t)(hd / a.k_share) * dim;
-    const float* vb = a.v + (size_t)hd * vdim;
+    const float* vb = a.v + (size_t)hd * vdim + cg * cols;
     const float* cb = PER_KEY ? a.c + (size_t)hd * dim : a.c + hd;
-    const bool vec = dim % 4 == 0 && vdim % 4 == 0 && cols % 4 == 0 &&
+    const int vcols = min(cols, vdim - cg * cols);   // columns of this CTA that exist
+    const bool vec = dim % 4 == 0 && vdim % 4 == 0 &&
                      (a.q_ld | a.k_ld | a.v_ld) % 4 == 0 && (!PER_KEY || a.c_ld % 4 == 0) &&
                      ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (PER_KEY ? (uintptr_t)a.c : 0)) % 16 == 0;
-    const float dd = a.direct ? a.direct[hd] : 0.0f;
+    const float dd = !PER_KEY && a.direct ? a.direct[hd] : 0.0f;
     if (dp > dim) {                                  // keys beyond the head: zero in both stages
         for (int e = threadIdx.x; e < 2 * DS_TB * (dp - dim); e += blockDim.x) {
             const int row = e / (dp - dim), i = dim + e % (dp - dim);
@@ -110,6 +114,12 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
             base[0] = 0.0f;
             base[DS_TB * dp] = 0.0f;
             if (PER_KEY) base[2 * DS_TB * dp] = 0.0f;
+        }
+    }
+    if (cols > vcols) {                              // and values beyond it
+        for (int e = threadIdx.x; e < 2 * DS_TB * (cols - vcols); e += blockDim.x) {
+            const int row = e / (cols - vcols), i = vcols + e % (cols - vcols);
+            sm[(row / DS_TB) * stage + DS_TB * (2 * dp + cw) + (row % DS_TB) * cols + i] = 0.0f;
         }
     }
     auto fetch = [&](int tb, int into) {
@@ -120,7 +130,7 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
         float* d_s = v_s + DS_TB * cols;
         const int nb = min(DS_TB, t1 - tb);
         if (vec) {
-            const int d4 = dim / 4, v4 = cols / 4;
+            const int d4 = dim / 4, v4 = vcols / 4;
             for (int e = threadIdx.x; e < nb * d4; e += blockDim.x) {
                 const int tok = e / d4, i = (e - tok * d4) * 4;
                 const size_t t = tb + tok;
@@ -130,8 +140,7 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
             }
             for (int e = threadIdx.x; e < nb * v4; e += blockDim.x) {
                 const int tok = e / v4, i = (e - tok * v4) * 4;
-                if (cg * cols + i < vdim)
-                    copy16(v_s + tok * cols + i, vb + (size_t)(tb + tok) * a.v_ld + cg * cols + i);
+                copy16(v_s + tok * cols + i, vb + (size_t)(tb + tok) * a.v_ld + i);
             }
         } else {
             for (int e = threadIdx.x; e < nb * dim; e += blockDim.x) {
@@ -141,18 +150,25 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
                 k_s[tok * dp + i] = kb[t * a.k_ld + i];
                 if (PER_KEY) c_s[tok * dp + i] = cb[t * a.c_ld + i];
             }
-            for (int e = threadIdx.x; e < nb * cols; e += blockDim.x) {
-                const int tok = e / cols, i = e - tok * cols;
-                if (cg * cols + i < vdim)
-                    v_s[tok * cols + i] = vb[(size_t)(tb + tok) * a.v_ld + cg * cols + i];
+            for (int e = threadIdx.x; e < nb * vcols; e += blockDim.x) {
+                const int tok = e / vcols, i = e - tok * vcols;
+                v_s[tok * cols + i] = vb[(size_t)(tb + tok) * a.v_ld + i];
             }
         }
-        for (int tok = threadIdx.x; tok < nb; tok += blockDim.x) {
-            d_s[tok * 4] = a.ks ? a.ks[(size_t)(tb + tok) * a.heads + hd] : 1.0f;
-            if (!PER_KEY) c_s[tok * 4] = cb[(size_t)(tb + tok) * a.c_ld];
+        if (!PER_KEY) {
+            for (int tok = threadIdx.x; tok < nb; tok += blockDim.x) {
+                d_s[tok * 4] = a.ks ? a.ks[(size_t)(tb + tok) * a.heads + hd] : 1.0f;
+                c_s[tok * 4] = cb[(size_t)(tb + tok) * a.c_ld];
+            }
         }
         copy_commit();
     };
+    const bool holder = mine && (ln & (L / DS_CC - 1)) == 0;
+    const int held = held_column<DS_CC>(ln, L);
+    const bool writes = holder && c0 + held < vdim;
+    // where a token's sum of this lane goes: the finish's rows, or raw sums
+    float* o_to = a.fin.out ? o_s + c0 + held : a.raw + (size_t)hd * vdim + c0 + held;
+    const size_t o_ld = a.fin.out ? vdim : a.raw_ld;
     fetch(t0, 0);
     int turn = 0;
     for (int tb = t0; tb < t1; tb += DS_TB, turn ^= 1) {
@@ -163,38 +179,40 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
         const float* q_s = sm + turn * stage;
         const float* k_s = q_s + DS_TB * dp;
         const float* c_s = k_s + DS_TB * dp;
-        const float* v_s = c_s + DS_TB * cw;
-        const float* d_s = v_s + DS_TB * cols;
+        const float* v_s = c_s + DS_TB * cw + cl;
+        const float* d_s = v_s - cl + DS_TB * cols;
         const int nb = min(DS_TB, t1 - tb);
+        float* o_at = o_to + (a.fin.out ? 0 : (size_t)tb * o_ld);
 #pragma unroll 2
         for (int tok = 0; tok < nb; ++tok) {
-            float v[DS_CC], part[DS_CC], raw[DS_CC];
-            const float ks = d_s[tok * 4];
+            float v[DS_CC], part[DS_CC];
 #pragma unroll
-            for (int j = 0; j < DS_CC; ++j) {
-                raw[j] = mine && cl * DS_CC + j < cols && c0 + j < vdim ? v_s[tok * cols + cl * DS_CC + j] : 0.0f;
-                v[j] = raw[j] * ks;
+            for (int j = 0; j < DS_CC; j += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(v_s + tok * cols + j);
+                v[j] = x.x; v[j + 1] = x.y; v[j + 2] = x.z; v[j + 3] = x.w;
+            }
+            if (!PER_KEY) {
+                const float ks = d_s[tok * 4];
+#pragma unroll
+                for (int j = 0; j < DS_CC; ++j) v[j] *= ks;
             }
             const float* c_at = PER_KEY ? c_s + tok * dp + ln * KPL : c_s + tok * 4;
-            advance<KPL, PER_KEY, MODE == 2>(S, k_s + tok * dp + ln * KPL, c_at, q_s + tok * dp + ln * KPL, v, part);
-            if (MODE == 1 && cl == 0) {              // 1 + p <- (1 + p)(1 + c)
+            advance<DS_CC, KPL, PER_KEY, MODE == 2>(S, k_s + tok * dp + ln * KPL, c_at, q_s + tok * dp + ln * KPL,
+                                                    v, part);
+            if (MODE == 1) {                         // 1 + p <- (1 + p)(1 + c)
+                if (PER_KEY) {
+                    if (cl == 0) {
 #pragma unroll
-                for (int i = 0; i < KPL; ++i) {
-                    const float c = PER_KEY ? c_at[i] : c_at[0];
-                    Pd[i] = fmaf(Pd[i], c, Pd[i] + c);
+                        for (int i = 0; i < KPL; ++i) Pd[i] = fmaf(Pd[i], c_at[i], Pd[i] + c_at[i]);
+                    }
+                } else {
+                    Pd[0] = fmaf(Pd[0], c_at[0], Pd[0] + c_at[0]);
                 }
             }
             if (MODE == 2) {
-                const float sum = close_columns(part, ln, L);
-                if (mine && (ln & ((L >> 2) - 1)) == 0) {
-                    const int j = held_column(ln, L);
-                    if (c0 + j < vdim && cl * DS_CC + j < cols) {
-                        const float x = j == 0 ? raw[0] : j == 1 ? raw[1] : j == 2 ? raw[2] : raw[3];
-                        const float o = fmaf(dd, x, sum * a.q_scale);
-                        if (a.fin.out) o_s[tok * vdim + c0 + j] = o;
-                        else a.raw[(size_t)(tb + tok) * a.raw_ld + (size_t)hd * vdim + c0 + j] = o;
-                    }
-                }
+                float sum = close_columns<DS_CC>(part, ln, L) * a.q_scale;
+                if (!PER_KEY) sum = fmaf(dd, v_s[tok * cols + held], sum);
+                if (writes) o_at[tok * o_ld] = sum;
             }
         }
         __syncthreads();
@@ -204,11 +222,12 @@ __global__ void __launch_bounds__(DS_THREADS) dscan_seg_kernel(SegArgs a) {
         }
     }
     if (mine) {
-        if (MODE == 1) store_state<KPL>(S, a.seg_own + (size_t)blockIdx.y * per_state + hd * per_head, ln, c0, dim, vdim);
+        if (MODE == 1)
+            store_state<DS_CC, KPL>(S, a.seg_own + (size_t)blockIdx.y * per_state + hd * per_head, ln, c0, dim, vdim);
         if (MODE == 2 && last)
-            store_state<KPL>(S, a.state + (size_t)slot * per_state + hd * per_head, ln, c0, dim, vdim);
+            store_state<DS_CC, KPL>(S, a.state + (size_t)slot * per_state + hd * per_head, ln, c0, dim, vdim);
     }
-    if (MODE == 1 && cl == 0 && cg == 0) {
+    if (MODE == 1 && mine && cl == 0 && cg == 0) {
         if (PER_KEY) {
 #pragma unroll
             for (int i = 0; i < KPL; ++i)
@@ -334,8 +353,8 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     float* q_s = sm;                                 // [dp]
     float* k_s = q_s + dp;
     float* c_s = k_s + dp;
-    float* v_s = c_s + dp;                           // [vdim rounded to DS_CC]
-    float* o_s = v_s + (vdim + DS_CC - 1) / DS_CC * DS_CC;
+    float* v_s = c_s + dp;                           // [vdim rounded to GS_CC]
+    float* o_s = v_s + (vdim + GS_CC - 1) / GS_CC * GS_CC;
     prb_grid_launch_dependents();
     const int hd = blockIdx.x, b = blockIdx.y;
     // (the step's description and the state of the step before lie behind launches that have
@@ -344,11 +363,11 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     const int slot = a.state_slot[b];
     const bool run = t1 > t && t >= 0 && t1 <= a.n_tokens && slot >= 0 && slot < a.n_slots;
     const int ln = threadIdx.x % L, cl = threadIdx.x / L;
-    const int c0 = cl * DS_CC;
+    const int c0 = cl * GS_CC;
     float* sp = a.state + ((size_t)(run ? slot : 0) * a.heads + hd) * vdim * dim;
     const bool carried = run && a.positions[t] > 0;
-    float S[DS_CC][KPL];
-    load_state<KPL>(S, carried && c0 < vdim ? sp : nullptr, ln, c0, dim, vdim);
+    float S[GS_CC][KPL];
+    load_state<GS_CC, KPL>(S, carried && c0 < vdim ? sp : nullptr, ln, c0, dim, vdim);
     float w2[GS_RANK];
     const int ch = hd * dim + (int)threadIdx.x, channels = a.heads * dim;
     const bool decays = (int)threadIdx.x < dim;
@@ -367,7 +386,7 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
         k_s[i] = i < dim ? row[a.k_col + hd * dim + i] : 0.0f;
         if (i >= dim) c_s[i] = 0.0f;
     }
-    for (int i = threadIdx.x; i < (vdim + DS_CC - 1) / DS_CC * DS_CC; i += blockDim.x)
+    for (int i = threadIdx.x; i < (vdim + GS_CC - 1) / GS_CC * GS_CC; i += blockDim.x)
         v_s[i] = i < vdim ? row[a.v_col + hd * vdim + i] : 0.0f;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
         float z = 0.0f;
@@ -385,23 +404,23 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
         c_s[i] = decay_minus_one(z, a.inv_tau);
     }
     __syncthreads();
-    float v[DS_CC], part[DS_CC];
+    float v[GS_CC], part[GS_CC];
 #pragma unroll
-    for (int j = 0; j < DS_CC; ++j) v[j] = c0 < vdim ? v_s[c0 + j] : 0.0f;
-    advance<KPL, true, true>(S, k_s + ln * KPL, c_s + ln * KPL, q_s + ln * KPL, v, part);
-    const float sum = close_columns(part, ln, L);
+    for (int j = 0; j < GS_CC; ++j) v[j] = c0 < vdim ? v_s[c0 + j] : 0.0f;
+    advance<GS_CC, KPL, true, true>(S, k_s + ln * KPL, c_s + ln * KPL, q_s + ln * KPL, v, part);
+    const float sum = close_columns<GS_CC>(part, ln, L);
     if ((ln & ((L >> 2) - 1)) == 0) {
-        const int j = held_column(ln, L);
+        const int j = held_column<GS_CC>(ln, L);
         if (c0 + j < vdim) o_s[c0 + j] = sum * a.q_scale;
     }
-    if (c0 < vdim) store_state<KPL>(S, sp, ln, c0, dim, vdim);
+    if (c0 < vdim) store_state<GS_CC, KPL>(S, sp, ln, c0, dim, vdim);
     __syncthreads();
     if (threadIdx.x < 32) finish_row<O>(a.fin, o_s, t, hd, vdim, threadIdx.x);
 }
 
 int seg_cols(int dim, int vdim) {
     const int lanes = lanes_of(dim);
-    int cols = DS_THREADS / lanes * DS_CC;
+    int cols = ds_threads(keys_per_lane(dim)) / lanes * DS_CC;
     if (cols > vdim) cols = (vdim + DS_CC - 1) / DS_CC * DS_CC;
     return cols;
 }
@@ -437,6 +456,7 @@ PRB_API int prb_dscan_segments(float* raw, long raw_ld, const float* q, long q_l
     if (!ok || heads <= 0 || q_share <= 0 || k_share <= 0 || n_requests > 65535) return PRB_E_SIZE;
     if (out != nullptr && (ok != 3 || gate == nullptr || norm_w == nullptr)) return PRB_E_ARG;
     if (out == nullptr && raw == nullptr) return PRB_E_ARG;
+    if (per_key && (ks != nullptr || direct != nullptr)) return PRB_E_ARG;
     const int need = prb_dscan_max_segments(n_tokens, n_requests);
     if (segments < need || need > 65535) return PRB_E_SIZE;
     if (out_dtype != PRB_F32 && out_dtype != PRB_BF16) return PRB_E_DTYPE;
@@ -508,7 +528,7 @@ PRB_API int prb_gla_decay(float* c_out, long c_ld, const float* lr, long lr_ld, 
     if (n_tokens <= 0) return 0;
     const size_t smem = (size_t)GD_TOKENS * rank * sizeof(float);
     if (channels <= 0 || rank <= 0 || smem > 40 * 1024) return PRB_E_SIZE;
-    const dim3 grid((n_tokens + GD_TOKENS - 1) / GD_TOKENS, (channels + 1023) / 1024);
+    const dim3 grid((n_tokens + GD_TOKENS - 1) / GD_TOKENS, (channels + 255) / 256);
     gla_decay_kernel<<<grid, 256, smem, stream>>>(c_out, c_ld, lr, lr_ld, w2t, bias, n_tokens, channels,
                                                   rank, inv_tau);
     PRB_LAUNCH_CHECK();
@@ -517,7 +537,7 @@ PRB_API int prb_gla_decay(float* c_out, long c_ld, const float* lr, long lr_ld, 
 
 PRB_API int prb_gla_step_supports(int dim, int vdim) {
     const int lanes = lanes_of(dim);
-    return lanes > 0 && vdim > 0 && (vdim + DS_CC - 1) / DS_CC * lanes <= (keys_per_lane(dim) == 4 ? 1024 : 512) ? 1 : 0;
+    return lanes > 0 && vdim > 0 && (vdim + GS_CC - 1) / GS_CC * lanes <= (keys_per_lane(dim) == 4 ? 1024 : 512) ? 1 : 0;
 }
 
 // Every request brings one token.
@@ -530,8 +550,8 @@ PRB_API int prb_gla_step(void* out, long out_ld, const float* proj, long ld, int
     if (n_tokens <= 0 || n_requests <= 0) return 0;
     if (heads <= 0 || rank <= 0 || n_requests > 65535 || !prb_gla_step_supports(dim, vdim)) return PRB_E_SIZE;
     const int lanes = lanes_of(dim), kpl = keys_per_lane(dim);
-    const int vp = (vdim + DS_CC - 1) / DS_CC * DS_CC;
-    const int threads = (vp / DS_CC * lanes + 31) / 32 * 32;
+    const int vp = (vdim + GS_CC - 1) / GS_CC * GS_CC;
+    const int threads = (vp / GS_CC * lanes + 31) / 32 * 32;
     const size_t smem = (size_t)(3 * lanes * kpl + 2 * vp) * sizeof(float);
     GlaStepArgs a{proj, ld, q_col, k_col, v_col, lr_col, w2t, bias, inv_tau, q_scale, state, q_start,
                   state_slot, positions, n_tokens, n_requests, heads, dim, vdim, rank, lanes, n_slots,

@@ -4,33 +4,31 @@
 //
 //     S_t = diag(a_t) S_(t-1) + k_t v_t^T              o_t = S_t^T q_t
 //
-// The state lies as [vdim][dim].  A thread holds KPL neighbouring keys of DS_CC value columns in
-// registers; the `dim` keys of a column are spread over L neighbouring lanes (a power of two
-// from 4 to 32).  A decay travels as c = a - 1 and a step is S + (k v + c S), so that a decay
+// The state lies as [vdim][dim].  A thread holds KPL neighbouring keys of CC value columns (4 or 8)
+// in registers; the `dim` keys of a column are spread over L neighbouring lanes (a power of two
+// from 8 to 32).  A decay travels as c = a - 1 and a step is S + (k v + c S), so that a decay
 // close to one keeps its precision.  The order of every sum depends on the sizes only.
 #pragma once
 #include "common.cuh"
 
 namespace dscan {
-constexpr int DS_CC = 4;             // value columns a thread holds
-
 inline int keys_per_lane(int dim) { return dim <= 128 ? 4 : dim <= 256 ? 8 : 16; }
 // Lanes a column is spread over (0: beyond the kernels).
 inline int lanes_of(int dim) {
     if (dim <= 0 || dim > 512) return 0;
     const int kpl = keys_per_lane(dim);
-    int lanes = 4;
+    int lanes = 8;
     while (lanes * kpl < dim) lanes *= 2;
     return lanes;
 }
 
-// The numbers of a thread's columns c0 .. c0 + DS_CC - 1 from or to rows of `dim` numbers.
-template <int KPL>
-__device__ __forceinline__ void load_state(float (&S)[DS_CC][KPL], const float* from, int ln, int c0,
+// The numbers of a thread's columns c0 .. c0 + CC - 1 from or to rows of `dim` numbers.
+template <int CC, int KPL>
+__device__ __forceinline__ void load_state(float (&S)[CC][KPL], const float* from, int ln, int c0,
                                            int dim, int vdim) {
     const bool vec = dim % 4 == 0;
 #pragma unroll
-    for (int c = 0; c < DS_CC; ++c) {
+    for (int c = 0; c < CC; ++c) {
         const bool live = from != nullptr && c0 + c < vdim;
         const float* row = from + (size_t)(c0 + c) * dim;
         if (vec) {
@@ -50,12 +48,12 @@ __device__ __forceinline__ void load_state(float (&S)[DS_CC][KPL], const float* 
         }
     }
 }
-template <int KPL>
-__device__ __forceinline__ void store_state(const float (&S)[DS_CC][KPL], float* to, int ln, int c0,
+template <int CC, int KPL>
+__device__ __forceinline__ void store_state(const float (&S)[CC][KPL], float* to, int ln, int c0,
                                             int dim, int vdim) {
     const bool vec = dim % 4 == 0;
 #pragma unroll
-    for (int c = 0; c < DS_CC; ++c) {
+    for (int c = 0; c < CC; ++c) {
         if (c0 + c >= vdim) continue;
         float* row = to + (size_t)(c0 + c) * dim;
         if (vec) {
@@ -76,22 +74,21 @@ __device__ __forceinline__ void store_state(const float (&S)[DS_CC][KPL], float*
     }
 }
 
-// One token: k, c, q point at the lane's KPL numbers (c at one number when !PER_KEY), v at the
-// thread's DS_CC values (already times the key's scale).  part[c] = the lane's share of q . S.
-template <int KPL, bool PER_KEY, bool OUT>
-__device__ __forceinline__ void advance(float (&S)[DS_CC][KPL], const float* k, const float* c,
-                                        const float* q, const float (&v)[DS_CC],
-                                        float (&part)[DS_CC]) {
+// One token: k, c, q point at the lane's KPL numbers (c at one number when !PER_KEY), v holds the
+// thread's values (already times the key's scale).  part[c] = the lane's share of q . S.
+template <int CC, int KPL, bool PER_KEY, bool OUT>
+__device__ __forceinline__ void advance(float (&S)[CC][KPL], const float* k, const float* c, const float* q,
+                                        const float (&v)[CC], float (&part)[CC]) {
     const float c1 = PER_KEY ? 0.0f : c[0];
 #pragma unroll
-    for (int j = 0; j < DS_CC; ++j) part[j] = 0.0f;
+    for (int j = 0; j < CC; ++j) part[j] = 0.0f;
 #pragma unroll
     for (int g = 0; g < KPL / 4; ++g) {
         const float4 k4 = reinterpret_cast<const float4*>(k)[g];
         const float4 c4 = PER_KEY ? reinterpret_cast<const float4*>(c)[g] : make_float4(c1, c1, c1, c1);
         const float4 q4 = OUT ? reinterpret_cast<const float4*>(q)[g] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-        for (int j = 0; j < DS_CC; ++j) {
+        for (int j = 0; j < CC; ++j) {
             float* s = &S[j][4 * g];
             s[0] += fmaf(c4.x, s[0], k4.x * v[j]);
             s[1] += fmaf(c4.y, s[1], k4.y * v[j]);
@@ -107,24 +104,33 @@ __device__ __forceinline__ void advance(float (&S)[DS_CC][KPL], const float* k, 
     }
 }
 
-// Sums of the lanes' four shares: afterwards lane ln holds column held_column(ln, L), and the
-// lanes with (ln & (L / 4 - 1)) == 0 cover all four.
-__device__ __forceinline__ float close_columns(const float (&p)[DS_CC], int ln, int L) {
+// Sums of the lanes' CC shares: halves of the columns change sides until a lane holds one, which the
+// lanes left over close.  Afterwards lane ln holds column held_column(ln, L), and the lanes with
+// (ln & (L / CC - 1)) == 0 cover them all.
+template <int CC>
+__device__ __forceinline__ float close_columns(const float (&p)[CC], int ln, int L) {
+    float a[CC];
+#pragma unroll
+    for (int j = 0; j < CC; ++j) a[j] = p[j];
     int h = L >> 1;
-    bool up = (ln & h) != 0;
-    float a0 = up ? p[2] : p[0], a1 = up ? p[3] : p[1];
-    const float b0 = up ? p[0] : p[2], b1 = up ? p[1] : p[3];
-    a0 += __shfl_xor_sync(0xffffffffu, b0, h);
-    a1 += __shfl_xor_sync(0xffffffffu, b1, h);
-    h >>= 1;
-    up = (ln & h) != 0;
-    float a = up ? a1 : a0;
-    a += __shfl_xor_sync(0xffffffffu, up ? a0 : a1, h);
-    for (h >>= 1; h > 0; h >>= 1) a += __shfl_xor_sync(0xffffffffu, a, h);
-    return a;
+#pragma unroll
+    for (int n = CC / 2; n > 0; n >>= 1, h >>= 1) {
+        const bool up = (ln & h) != 0;
+#pragma unroll
+        for (int j = 0; j < n; ++j) {
+            const float keep = up ? a[n + j] : a[j], send = up ? a[j] : a[n + j];
+            a[j] = keep + __shfl_xor_sync(0xffffffffu, send, h);
+        }
+    }
+    for (; h > 0; h >>= 1) a[0] += __shfl_xor_sync(0xffffffffu, a[0], h);
+    return a[0];
 }
+template <int CC>
 __device__ __forceinline__ int held_column(int ln, int L) {
-    return ((ln & (L >> 1)) ? 2 : 0) + ((ln & (L >> 2)) ? 1 : 0);
+    int j = 0;
+#pragma unroll
+    for (int n = CC / 2, h = L >> 1; n > 0; n >>= 1, h >>= 1) j += (ln & h) ? n : 0;
+    return j;
 }
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }

@@ -41,126 +41,149 @@ __device__ __forceinline__ void store4(O* o, const float (&v)[4]) {
     }
 }
 
-// CTAs (row, slice of the row's columns); every CTA of a row chooses for itself.
-template <typename O>
-__global__ void __launch_bounds__(256) expert_act_kernel(ExpertArgs a) {
-    extern __shared__ float sh[];                    // [all] scores, [all] choice, [all] weights
-    __shared__ float scratch[32];
-    __shared__ float own_s[2];                       // the identity experts' weight, the shared expert's
-    const int all = a.experts + a.identity;
-    float* sc = sh;
-    float* pick = sh + all;
-    float* wt = sh + 2 * all;
-    prb_grid_launch_dependents();
-    const int t = blockIdx.x;
-    const float* row = a.in + (size_t)t * a.in_ld;
-    if (threadIdx.x < 32) {
-        const int lane = threadIdx.x;
-        float top_z = -INFINITY;
-        for (int e = lane; e < all; e += 32) top_z = fmaxf(top_z, row[a.router_col + e]);
-        top_z = prb_warp_max(top_z);
-        float sum = 0.0f;
+// Scores, choice and weights of one row, by a warp: wt[e] of every expert, own[0] the identity experts'
+// weight together, own[1] the shared expert's.
+__device__ __forceinline__ void choose(const ExpertArgs& a, const float* row, float* sc, float* pick, float* wt,
+                                       float* own) {
+    const int lane = threadIdx.x & 31, all = a.experts + a.identity;
+    float top_z = -INFINITY;
+    for (int e = lane; e < all; e += 32) {
+        const float z = row[a.router_col + e];
+        sc[e] = z;
+        top_z = fmaxf(top_z, z);
+    }
+    top_z = prb_warp_max(top_z);
+    float sum = 0.0f;
+    for (int e = lane; e < all; e += 32) {
+        const float p = expf(sc[e] - top_z);
+        sc[e] = p;
+        sum += p;
+    }
+    sum = prb_warp_sum(sum);
+    for (int e = lane; e < all; e += 32) {
+        const float s = sc[e] / sum;
+        sc[e] = s;
+        pick[e] = s + (a.correction ? a.correction[e] : 0.0f);
+        wt[e] = 0.0f;
+    }
+    __syncwarp();
+    float chosen = 0.0f;
+    for (int k = 0; k < a.top; ++k) {                // the largest left; ties: the lower index
+        float best = -INFINITY;
+        int arg = all;
         for (int e = lane; e < all; e += 32) {
-            const float p = expf(row[a.router_col + e] - top_z);
-            sc[e] = p;
-            sum += p;
+            const float v = pick[e];
+            if (v > best) { best = v; arg = e; }
         }
-        sum = prb_warp_sum(sum);
-        for (int e = lane; e < all; e += 32) {
-            const float s = sc[e] / sum;
-            sc[e] = s;
-            pick[e] = s + (a.correction ? a.correction[e] : 0.0f);
-            wt[e] = 0.0f;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v = __shfl_xor_sync(0xffffffffu, best, o);
+            const int w = __shfl_xor_sync(0xffffffffu, arg, o);
+            if (w < all && (arg >= all || v > best || (v == best && w < arg))) { best = v; arg = w; }
+        }
+        if (arg >= all) break;                       // (a row of NaNs: padding, or a fault upstream)
+        chosen += sc[arg];
+        if (lane == 0) {
+            wt[arg] = sc[arg];
+            pick[arg] = -INFINITY;
         }
         __syncwarp();
-        float chosen = 0.0f;
-        for (int k = 0; k < a.top; ++k) {            // the largest left; ties: the lower index
-            float best = -INFINITY;
-            int arg = all;
-            for (int e = lane; e < all; e += 32) {
-                const float v = pick[e];
-                if (v > best) { best = v; arg = e; }
-            }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float v = __shfl_xor_sync(0xffffffffu, best, o);
-                const int w = __shfl_xor_sync(0xffffffffu, arg, o);
-                if (w < all && (arg >= all || v > best || (v == best && w < arg))) { best = v; arg = w; }
-            }
-            if (arg >= all) break;                   // (a row of NaNs: padding, or a fault upstream)
-            if (lane == 0) {
-                wt[arg] = sc[arg];
-                pick[arg] = -INFINITY;
-            }
-            chosen += sc[arg];
-            __syncwarp();
-        }
-        const float mult = a.factor / (a.renorm ? chosen : 1.0f);
-        float own = 0.0f;
-        for (int e = lane; e < all; e += 32) {
-            const float w = wt[e] * mult;
-            wt[e] = w;
-            if (e >= a.experts) own += w;
-        }
-        own = prb_warp_sum(own);
-        if (lane == 0) {
-            own_s[0] = own;
-            own_s[1] = a.shared_weight_col >= 0 ? ea_sigmoid(row[a.shared_weight_col]) : 1.0f;
-        }
     }
-    __syncthreads();
-    // columns: the experts' (experts * group), then the shared expert's
+    const float mult = a.factor / (a.renorm ? chosen : 1.0f);
+    float mine = 0.0f;
+    for (int e = lane; e < all; e += 32) {
+        const float w = wt[e] * mult;
+        wt[e] = w;
+        if (e >= a.experts) mine += w;
+    }
+    mine = prb_warp_sum(mine);
+    if (lane == 0) {
+        own[0] = mine;
+        own[1] = a.shared_weight_col >= 0 ? ea_sigmoid(row[a.shared_weight_col]) : 1.0f;
+    }
+}
+
+// x += weight * input of one row, by the CTA.
+template <typename O>
+__device__ __forceinline__ void add_input(const ExpertArgs& a, int t, float w, float* scratch) {
+    float* x = a.x + (size_t)t * a.x_ld;
+    if (a.h != nullptr) {
+        const O* h = (const O*)a.h + (size_t)t * a.h_ld;
+        for (int i = threadIdx.x; i < a.width; i += blockDim.x) x[i] = fmaf(w, prb_to_float<O>(h[i]), x[i]);
+        return;
+    }
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < a.width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+    ss = prb_block_sum(ss, scratch);
+    const float inv = w / sqrtf(ss / (float)a.width + a.eps);
+    for (int i = threadIdx.x; i < a.width; i += blockDim.x)
+        x[i] = fmaf(x[i] * inv, a.norm_w ? a.norm_w[i] : 1.0f, x[i]);
+}
+
+// CTAs (ROWS rows, slice of their columns); every CTA of a row chooses for itself, a warp a row.
+// Columns: the experts' (experts * group), then the shared expert's.
+constexpr int EA_ROWS = 8;
+template <typename O, int ROWS>
+__global__ void __launch_bounds__(256) expert_act_kernel(ExpertArgs a) {
+    extern __shared__ float sh[];                    // per row: [all] scores, [all] choice, [all] weights
+    __shared__ float scratch[32];
+    __shared__ float own_s[ROWS][2];
+    const int all = a.experts + a.identity;
+    prb_grid_launch_dependents();
+    const int t0 = blockIdx.x * ROWS, nt = min(ROWS, a.n_rows - t0);
     const int n_exp = a.experts * a.group, n_all = n_exp + a.shared;
     const int per = ((n_all + (int)gridDim.y - 1) / (int)gridDim.y + 3) / 4 * 4;
     const int lo = blockIdx.y * per, hi = min(n_all, lo + per);
-    O* o = (O*)a.out + (size_t)t * a.out_ld;
     const bool vec = a.group % 4 == 0 && (a.gate_col | a.up_col | a.in_ld | a.out_ld) % 4 == 0 &&
                      (a.shared == 0 || (a.shared_gate_col | a.shared_up_col | a.shared) % 4 == 0) &&
                      ((uintptr_t)a.in) % 16 == 0 && ((uintptr_t)a.out) % (4 * sizeof(O)) == 0;
-    if (vec) {
-        for (int i = lo + threadIdx.x * 4; i < hi; i += blockDim.x * 4) {
-            const bool routed = i < n_exp;
-            const float w = routed ? wt[i / a.group] : own_s[1];
-            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            if (w != 0.0f) {                         // (columns of experts not chosen are not read)
-                const int gc = routed ? a.gate_col + i : a.shared_gate_col + i - n_exp;
-                const int uc = routed ? a.up_col + i : a.shared_up_col + i - n_exp;
-                const float4 g = *reinterpret_cast<const float4*>(row + gc);
-                const float4 u = *reinterpret_cast<const float4*>(row + uc);
-                v[0] = w * ea_gate(g.x, a.act) * u.x;
-                v[1] = w * ea_gate(g.y, a.act) * u.y;
-                v[2] = w * ea_gate(g.z, a.act) * u.z;
-                v[3] = w * ea_gate(g.w, a.act) * u.w;
-            }
-            store4(o + i, v);
-        }
-    } else {
-        for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) {
-            const bool routed = i < n_exp;
-            const float w = routed ? wt[i / a.group] : own_s[1];
-            float v = 0.0f;
-            if (w != 0.0f)
-                v = routed ? w * ea_gate(row[a.gate_col + i], a.act) * row[a.up_col + i]
-                           : w * ea_gate(row[a.shared_gate_col + i - n_exp], a.act) *
-                                 row[a.shared_up_col + i - n_exp];
-            o[i] = prb_from_float<O>(v);
-        }
+    auto gate_at = [&](int i) { return i < n_exp ? a.gate_col + i : a.shared_gate_col + i - n_exp; };
+    auto up_at = [&](int i) { return i < n_exp ? a.up_col + i : a.shared_up_col + i - n_exp; };
+    prb_grid_wait();
+    // a single row's first columns are asked for before anyone knows which experts it chooses
+    float4 g0 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), u0 = g0;
+    const int first = lo + (int)threadIdx.x * 4;
+    if (ROWS == 1 && vec && first < hi) {
+        const float* row = a.in + (size_t)t0 * a.in_ld;
+        g0 = *reinterpret_cast<const float4*>(row + gate_at(first));
+        u0 = *reinterpret_cast<const float4*>(row + up_at(first));
     }
-    if (a.identity > 0 && blockIdx.y == 0 && own_s[0] != 0.0f) {
-        const float w = own_s[0];
-        float* x = a.x + (size_t)t * a.x_ld;
-        if (a.h != nullptr) {
-            const O* h = (const O*)a.h + (size_t)t * a.h_ld;
-            for (int i = threadIdx.x; i < a.width; i += blockDim.x)
-                x[i] = fmaf(w, prb_to_float<O>(h[i]), x[i]);
+    const int warp = threadIdx.x >> 5;
+    if (warp < nt) {
+        float* mine = sh + (size_t)warp * 3 * all;
+        choose(a, a.in + (size_t)(t0 + warp) * a.in_ld, mine, mine + all, mine + 2 * all, own_s[warp]);
+    }
+    __syncthreads();
+    for (int r = 0; r < nt; ++r) {
+        const float* row = a.in + (size_t)(t0 + r) * a.in_ld;
+        const float* wt = sh + (size_t)r * 3 * all + 2 * all;
+        O* o = (O*)a.out + (size_t)(t0 + r) * a.out_ld;
+        const float shared_w = own_s[r][1];
+        if (vec) {
+            for (int i = first; i < hi; i += blockDim.x * 4) {
+                const float w = i < n_exp ? wt[i / a.group] : shared_w;
+                float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                if (w != 0.0f) {                     // (columns of experts not chosen are not read)
+                    float4 g = g0, u = u0;
+                    if (ROWS > 1 || i != first) {
+                        g = *reinterpret_cast<const float4*>(row + gate_at(i));
+                        u = *reinterpret_cast<const float4*>(row + up_at(i));
+                    }
+                    v[0] = w * ea_gate(g.x, a.act) * u.x;
+                    v[1] = w * ea_gate(g.y, a.act) * u.y;
+                    v[2] = w * ea_gate(g.z, a.act) * u.z;
+                    v[3] = w * ea_gate(g.w, a.act) * u.w;
+                }
+                store4(o + i, v);
+            }
         } else {
-            float ss = 0.0f;
-            for (int i = threadIdx.x; i < a.width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
-            ss = prb_block_sum(ss, scratch);
-            const float inv = w / sqrtf(ss / (float)a.width + a.eps);
-            for (int i = threadIdx.x; i < a.width; i += blockDim.x)
-                x[i] = fmaf(x[i] * inv, a.norm_w ? a.norm_w[i] : 1.0f, x[i]);
+            for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) {
+                const float w = i < n_exp ? wt[i / a.group] : shared_w;
+                o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(row[gate_at(i)], a.act) * row[up_at(i)] : 0.0f);
+            }
         }
+        if (a.identity > 0 && blockIdx.y == 0 && own_s[r][0] != 0.0f)
+            add_input<O>(a, t0 + r, own_s[r][0], scratch);
     }
 }
 
@@ -177,6 +200,7 @@ template <typename O, bool VEC>
 __global__ void act_columns_kernel(O* __restrict__ out, long out_ld, const float* __restrict__ in, long in_ld,
                                    int n, int n_rows, int act) {
     prb_grid_launch_dependents();
+    prb_grid_wait();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if constexpr (VEC) {
         const int n4 = n / 4;
@@ -208,18 +232,35 @@ PRB_API int prb_expert_act(void* out, long out_ld, const float* in, long in_ld, 
     const ExpertArgs a{out, out_ld, in, in_ld, gate_col, up_col, router_col, shared_gate_col, shared_up_col,
                        shared_weight_col, n_rows, experts, identity, top, group, shared, renorm, act, factor,
                        correction, x, x_ld, width, h, h_ld, norm_w, eps};
-    // slices of 2,048 columns, fewer while the rows alone fill the GPU
-    int slices = (experts * group + shared + 2047) / 2048;
-    if (slices < 1) slices = 1;
-    if (slices > 64) slices = 64;
-    while (slices > 1 && (long)n_rows * slices > 8L * prb_sm_count()) slices = (slices + 1) / 2;
-    const dim3 grid(n_rows, slices);
-    const size_t smem = (size_t)3 * all * sizeof(float);
-    if (dtype == PRB_F32) expert_act_kernel<float><<<grid, 256, smem, stream>>>(a);
-    else if (dtype == PRB_BF16) expert_act_kernel<__nv_bfloat16><<<grid, 256, smem, stream>>>(a);
-    else return PRB_E_DTYPE;
-    PRB_LAUNCH_CHECK();
-    return 0;
+    const int columns = experts * group + shared;
+    cudaError_t e;
+    if (n_rows <= 64) {
+        // a row a CTA and slice, four columns a thread where that leaves no more than 64 slices
+        const int slices = columns < 1024 ? 1 : (columns + 1023) / 1024 > 64 ? 64 : (columns + 1023) / 1024;
+        const dim3 grid(n_rows, slices);
+        const size_t smem = (size_t)3 * all * sizeof(float);
+        if (dtype == PRB_F32) e = prb_launch_dependent(expert_act_kernel<float, 1>, grid, dim3(256), smem, stream, a);
+        else if (dtype == PRB_BF16)
+            e = prb_launch_dependent(expert_act_kernel<__nv_bfloat16, 1>, grid, dim3(256), smem, stream, a);
+        else return PRB_E_DTYPE;
+    } else {
+        const int groups = (n_rows + EA_ROWS - 1) / EA_ROWS;
+        int slices = (columns + 1023) / 1024;
+        if (slices < 1) slices = 1;
+        while (slices > 1 && (long)groups * slices > 8L * prb_sm_count()) slices = (slices + 1) / 2;
+        const dim3 grid(groups, slices);
+        const size_t smem = (size_t)3 * EA_ROWS * all * sizeof(float);
+        if (smem > 40 * 1024) {
+            cudaFuncSetAttribute(expert_act_kernel<float, EA_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            cudaFuncSetAttribute(expert_act_kernel<__nv_bfloat16, EA_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        }
+        if (dtype == PRB_F32)
+            e = prb_launch_maybe_early(false, expert_act_kernel<float, EA_ROWS>, grid, dim3(256), smem, stream, a);
+        else if (dtype == PRB_BF16)
+            e = prb_launch_maybe_early(false, expert_act_kernel<__nv_bfloat16, EA_ROWS>, grid, dim3(256), smem, stream, a);
+        else return PRB_E_DTYPE;
+    }
+    return e == cudaSuccess ? 0 : (int)e;
 }
 
 // act 0: relu(.)^2, 1: relu, 2: gelu (tanh form), 3: silu; `in` points at the first column.
@@ -231,10 +272,12 @@ PRB_API int prb_act_columns(void* out, long out_ld, const float* in, long in_ld,
     const size_t esz = out_dtype == PRB_F32 ? 4 : 2, total = (size_t)n * n_rows;
     const bool vec = (n | in_ld | out_ld) % 4 == 0 && ((uintptr_t)in) % 16 == 0 && ((uintptr_t)out) % (4 * esz) == 0;
     const unsigned blocks = (unsigned)(((vec ? total / 4 : total) + 255) / 256);
-#define ACTC(OT, V) act_columns_kernel<OT, V><<<blocks, 256, 0, stream>>>((OT*)out, out_ld, in, in_ld, n, n_rows, act)
-    if (out_dtype == PRB_F32) { if (vec) ACTC(float, true); else ACTC(float, false); }
-    else { if (vec) ACTC(__nv_bfloat16, true); else ACTC(__nv_bfloat16, false); }
+    cudaError_t e;
+#define ACTC(OT, V)                                                                                          \
+    e = prb_launch_maybe_early(n_rows <= 64, act_columns_kernel<OT, V>, dim3(blocks), dim3(256), 0, stream,   \
+                               (OT*)out, out_ld, in, in_ld, n, n_rows, act)
+    if (out_dtype == PRB_F32) { if (vec) { ACTC(float, true); } else { ACTC(float, false); } }
+    else { if (vec) { ACTC(__nv_bfloat16, true); } else { ACTC(__nv_bfloat16, false); } }
 #undef ACTC
-    PRB_LAUNCH_CHECK();
-    return 0;
+    return e == cudaSuccess ? 0 : (int)e;
 }

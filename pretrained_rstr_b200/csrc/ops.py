@@ -2515,12 +2515,14 @@ class StateSpace:
             raise KernelArgumentError(f"{what}: shapes do not fit")
         if taps > 1:
             _need(conv_state, torch.float32, "saved inputs", what)
-            if tuple(conv_state.shape) != (state.shape[0], taps - 1, channels):
+            if tuple(conv_state.shape) != (state.shape[0], taps, channels):
                 raise KernelArgumentError(f"{what}: the saved inputs have the wrong shape")
         else:
             conv_state = None
         self.n, self.heads, self.channels, self.out_dtype = n, heads, channels, dtype_code(out.dtype)
         self.vdim, self.dim, self.n_requests = vdim, dim, n_requests
+        # (the calls below hand over addresses: what lies there has to live as long)
+        self._tensors = (proj, conv_w, conv_b, dt_bias, neg_a, direct, norm_w, conv_state, state, raw, out)
         self._args = (_p(proj), proj.stride(0), z, x, dt, _p(conv_w), _p(conv_b), _p(dt_bias), _p(neg_a),
                       _p(direct), _p(conv_state), _p(state), _p(seq_of_token), _p(q_start), _p(state_slot),
                       _p(positions), n, int(n_requests), int(heads), int(vdim), int(dim), int(groups), taps,

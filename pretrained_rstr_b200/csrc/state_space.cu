@@ -16,13 +16,14 @@
 //   w_j = exp(cum_end - cum_j) dt_j; the carry walks a request's segments; outputs are exp(cum_i)
 //   C S_start + sum_(j <= i) (C_i . B_j) exp(cum_i - cum_j) dt_j x_j, cum the running sum of log a.
 //   32-bit runs (and sizes these do not take) use the recurrence of decayed_scan.cu instead.
-// ssm_finish: a CTA per token: norm in parts; the CTA of a request's last token also brings the
-//   convolution's saved inputs up to date.
+// ssm_finish: norm in parts, a warp per (token, part) or a CTA per token; the saved inputs are brought
+//   up to date.
 // ssm_step: a step of single tokens in one launch: CTAs (head and share of its value columns,
 //   request); state, saved inputs and taps are requested before the kernel waits for the
-//   projection; the request's last CTA to arrive norms the token and saves the inputs.
-// The saved inputs are per-request state, [slots, taps - 1, channels] in 32-bit (projected numbers
-// before the convolution's bias).
+//   projection; the request's last CTA to arrive norms the token.
+// The saved inputs are per-request state, [slots, taps, channels] in 32-bit (projected numbers before
+// the convolution's bias): the token at position p lies in row p mod taps, so that saving one never
+// touches a number that any CTA of the same step still reads.
 #include "decayed_scan.cuh"
 
 namespace {
@@ -35,7 +36,7 @@ struct SsmArgs {
     const float* conv_w;             // [taps, channels]
     const float* conv_b;             // [channels]
     const float* dt_bias; const float* neg_a; const float* d;      // [heads]; neg_a = -exp(A_log)
-    float* conv_state;               // [slots, taps - 1, channels], or null (one tap)
+    float* conv_state;               // [slots, taps, channels], or null (one tap)
     float* state;                    // [slots, heads, vdim, dim]
     const int* seq; const int* q_start; const int* state_slot; const int* positions;
     int n_tokens, n_requests, heads, vdim, dim, groups, taps, n_slots;
@@ -54,7 +55,7 @@ __device__ __forceinline__ float past_input(const SsmArgs& a, int channels, int 
                                             int pos, int ch, int m) {
     if (m > pos) return 0.0f;
     if (m <= back) return a.proj[(size_t)(t - m) * a.ld + a.x_col + ch];
-    return a.conv_state[((size_t)slot * (a.taps - 1) + (a.taps - 1 - (m - back))) * channels + ch];
+    return a.conv_state[((size_t)slot * a.taps + (pos - m) % a.taps) * channels + ch];
 }
 
 __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
@@ -62,7 +63,8 @@ __device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __flo
 
 constexpr int SP_TOKENS = 8;
 // grid (tokens / 8, channels / 256 + 1): the last column of CTAs does the step sizes.
-template <typename X>
+// TAPS: the most taps (fewer have weights of zero for the oldest).
+template <typename X, int TAPS>
 __global__ void __launch_bounds__(256) ssm_prepare_kernel(SsmArgs a, X* __restrict__ xbc, long xbc_ld,
                                                           float* __restrict__ dt_out,
                                                           float* __restrict__ decay_out, int as_log) {
@@ -81,9 +83,11 @@ __global__ void __launch_bounds__(256) ssm_prepare_kernel(SsmArgs a, X* __restri
     }
     const int ch = blockIdx.y * blockDim.x + threadIdx.x;
     if (ch >= channels) return;
-    float w[SSM_TAPS], win[SSM_TAPS];                // win[j]: the value taps - 1 - j tokens ago
+    // w[TAPS - 1] is the current token's; win[j] the value TAPS - 1 - j tokens ago
+    float w[TAPS], win[TAPS];
+    const int skip = TAPS - a.taps;
 #pragma unroll
-    for (int j = 0; j < SSM_TAPS; ++j) w[j] = j < a.taps ? a.conv_w[(size_t)j * channels + ch] : 0.0f;
+    for (int j = 0; j < TAPS; ++j) w[j] = j >= skip ? a.conv_w[(size_t)(j - skip) * channels + ch] : 0.0f;
     const float bias = a.conv_b[ch];
     float cur[SP_TOKENS];
 #pragma unroll
@@ -101,20 +105,16 @@ __global__ void __launch_bounds__(256) ssm_prepare_kernel(SsmArgs a, X* __restri
             const bool fine = slot >= 0 && slot < a.n_slots;
             if (!fine && threadIdx.x == 0) prb_set_status(a.status, PRB_S_ROW_RANGE, t, slot, a.n_slots);
 #pragma unroll
-            for (int j = 0; j < SSM_TAPS; ++j)
-                win[j] = j < a.taps - 1 && fine ? past_input(a, channels, t, slot, back, pos, ch, a.taps - 1 - j)
-                                                : 0.0f;
+            for (int j = 0; j < TAPS - 1; ++j)
+                win[j] = j >= skip && fine ? past_input(a, channels, t, slot, back, pos, ch, TAPS - 1 - j) : 0.0f;
         }
+        win[TAPS - 1] = cur[tt];
         float s = bias;
 #pragma unroll
-        for (int j = 0; j < SSM_TAPS; ++j) {
-            if (j == a.taps - 1) win[j] = cur[tt];
-            s = fmaf(w[j], win[j], s);
-        }
+        for (int j = 0; j < TAPS; ++j) s = fmaf(w[j], win[j], s);
         store_as(xbc + (size_t)t * xbc_ld + ch, silu(s));
 #pragma unroll
-        for (int j = 0; j + 1 < SSM_TAPS; ++j) win[j] = win[j + 1];
-        win[SSM_TAPS - 1] = 0.0f;
+        for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
     }
 }
 
@@ -325,9 +325,10 @@ __global__ void ssm_carry_kernel(ChunkArgs c) {
     *reinterpret_cast<float4*>(st) = S;
 }
 
-// Grid (head, segment); 128 threads, a warp per 16 tokens.  VT: 8-column tiles of the value size.
+// Grid (head, segment); 256 threads: warps w and w + 4 share 16 tokens, each with half of the value
+// columns.  VT: 8-column tiles a warp has room for.
 template <int VT>
-__global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
+__global__ void __launch_bounds__(256) ssm_out_kernel(ChunkArgs c) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     prb_grid_launch_dependents();
     const int hd = blockIdx.x;
@@ -356,10 +357,23 @@ __global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
     running_sums(c, t0, nb, hd, cum_s, dt_s);
     copy_wait<0>();
     __syncthreads();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3;
     const int r0 = warp * 16;
-    if (r0 >= nb) return;
+    const int v_lo = (threadIdx.x >> 7) * VT * 8, v_n = min(V - v_lo, VT * 8);   // this warp's columns
+    if (r0 >= nb || v_n <= 0) return;
     const int i0 = r0 + (lane >> 2), i1 = i0 + 8;    // this lane's token rows
+    // the gates, asked for before the products
+    float2 z[VT][2];
+#pragma unroll
+    for (int v = 0; v < VT; ++v)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int i = half ? i1 : i0;
+            z[v][half] = v * 8 < v_n && i < nb
+                ? *reinterpret_cast<const float2*>(c.s.proj + (size_t)(t0 + i) * c.s.ld + c.s.z_col + hd * V + v_lo +
+                                                   v * 8 + (lane & 3) * 2)
+                : make_float2(0.0f, 0.0f);
+        }
     float acc[VT][4];
 #pragma unroll
     for (int i = 0; i < VT; ++i)
@@ -385,8 +399,8 @@ __global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
         if (started) {
 #pragma unroll
             for (int p = 0; p < VT / 2; ++p) {
-                if (p * 16 < V) {
-                    const int at = (p * 16 + (lane & 7) + (lane >> 4) * 8) * np + k0 + ((lane >> 3) & 1) * 8;
+                if (p * 16 < v_n) {
+                    const int at = (v_lo + p * 16 + (lane & 7) + (lane >> 4) * 8) * np + k0 + ((lane >> 3) & 1) * 8;
                     uint32_t hh[4], ll[4];
                     ldsm4(hh, sh + at);
                     ldsm4(ll, sl + at);
@@ -427,9 +441,9 @@ __global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
         mh[3] = pack2(w[1][2], w[1][3]); ml[3] = pack2(low_part(w[1][2]), low_part(w[1][3]));
 #pragma unroll
         for (int v = 0; v < VT / 2; ++v) {
-            if (v * 16 < V) {
+            if (v * 16 < v_n) {
                 uint32_t xx[4];
-                ldsm4t(xx, xs + (p * 16 + (lane & 15)) * vp + v * 16 + (lane >> 4) * 8);
+                ldsm4t(xx, xs + (p * 16 + (lane & 15)) * vp + v_lo + v * 16 + (lane >> 4) * 8);
                 mma16816(acc[2 * v], mh, xx[0], xx[1]);
                 mma16816(acc[2 * v], ml, xx[0], xx[1]);
                 mma16816(acc[2 * v + 1], mh, xx[2], xx[3]);
@@ -440,19 +454,17 @@ __global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
     const float dd = c.s.d[hd];
 #pragma unroll
     for (int v = 0; v < VT; ++v) {
-        if (v * 8 < V) {
-            const int col = v * 8 + (lane & 3) * 2;
+        if (v * 8 < v_n) {
+            const int col = v_lo + v * 8 + (lane & 3) * 2;
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
                 const int i = half ? i1 : i0;
                 if (i < nb) {
                     const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(xs + i * vp + col);
-                    const float2 z = *reinterpret_cast<const float2*>(
-                        c.s.proj + (size_t)(t0 + i) * c.s.ld + c.s.z_col + hd * V + col);
                     const float y0 = fmaf(dd, __bfloat162float(x.x), acc[v][2 * half]);
                     const float y1 = fmaf(dd, __bfloat162float(x.y), acc[v][2 * half + 1]);
                     *reinterpret_cast<float2*>(c.s.raw + (size_t)(t0 + i) * c.s.raw_ld + hd * V + col) =
-                        make_float2(y0 * silu(z.x), y1 * silu(z.y));
+                        make_float2(y0 * silu(z[v][half].x), y1 * silu(z[v][half].y));
                 }
             }
         }
@@ -460,70 +472,105 @@ __global__ void __launch_bounds__(128) ssm_out_kernel(ChunkArgs c) {
 }
 
 // ----------------------------------------------------------------------------- finish
-// The norm of one token's row in equal parts; `row` holds the gated numbers, or (z != null) the
-// ungated ones.  Few parts: the whole CTA a part; many: a warp a part.
+// A part of a token's row by the warp: the gated numbers (or, with z, the ungated ones) stay in
+// registers while they fit (up to 2,048, in pieces of four).
+constexpr int FIN_PIECES = 16;
 template <typename O>
-__device__ __forceinline__ void norm_in_parts(const SsmArgs& a, const float* row, const float* z, int t,
-                                              float* scratch) {
-    const int inner = a.heads * a.vdim, part = inner / a.parts;
-    O* o = (O*)a.out + (size_t)t * a.out_ld;
-    if (a.parts < 4) {
-        for (int p = 0; p < a.parts; ++p) {
-            const int lo = p * part;
-            float ss = 0.0f;
-            for (int i = threadIdx.x; i < part; i += blockDim.x) {
-                const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
-                ss = fmaf(y, y, ss);
-            }
-            ss = prb_block_sum(ss, scratch);
-            const float inv = a.out_scale / sqrtf(ss / (float)part + a.eps);
-            for (int i = threadIdx.x; i < part; i += blockDim.x) {
-                const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
-                o[lo + i] = prb_from_float<O>(y * inv * a.norm_w[lo + i]);
+__device__ __forceinline__ void norm_part_warp(const SsmArgs& a, const float* row, const float* z, O* o, int lo,
+                                               int part, int lane) {
+    if (part % 4 == 0 && part <= FIN_PIECES * 128 && (lo | a.raw_ld) % 4 == 0 && ((uintptr_t)a.raw) % 16 == 0 &&
+        z == nullptr) {
+        float4 y[FIN_PIECES];
+        float ss = 0.0f;
+#pragma unroll
+        for (int p = 0; p < FIN_PIECES; ++p) {
+            const int i = p * 128 + lane * 4;
+            y[p] = i < part ? *reinterpret_cast<const float4*>(row + lo + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+#pragma unroll
+        for (int p = 0; p < FIN_PIECES; ++p)
+            ss = fmaf(y[p].x, y[p].x, fmaf(y[p].y, y[p].y, fmaf(y[p].z, y[p].z, fmaf(y[p].w, y[p].w, ss))));
+        const float inv = a.out_scale / sqrtf(prb_warp_sum(ss) / (float)part + a.eps);
+#pragma unroll
+        for (int p = 0; p < FIN_PIECES; ++p) {
+            const int i = lo + p * 128 + lane * 4;
+            if (p * 128 + lane * 4 < part) {
+                o[i] = prb_from_float<O>(y[p].x * inv * a.norm_w[i]);
+                o[i + 1] = prb_from_float<O>(y[p].y * inv * a.norm_w[i + 1]);
+                o[i + 2] = prb_from_float<O>(y[p].z * inv * a.norm_w[i + 2]);
+                o[i + 3] = prb_from_float<O>(y[p].w * inv * a.norm_w[i + 3]);
             }
         }
         return;
     }
-    const int lane = threadIdx.x & 31;
-    for (int p = threadIdx.x >> 5; p < a.parts; p += blockDim.x >> 5) {
-        const int lo = p * part;
-        float ss = 0.0f;
-        for (int i = lane; i < part; i += 32) {
-            const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
-            ss = fmaf(y, y, ss);
-        }
-        const float inv = a.out_scale / sqrtf(prb_warp_sum(ss) / (float)part + a.eps);
-        for (int i = lane; i < part; i += 32) {
-            const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
-            o[lo + i] = prb_from_float<O>(y * inv * a.norm_w[lo + i]);
-        }
+    float ss = 0.0f;
+    for (int i = lane; i < part; i += 32) {
+        const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
+        ss = fmaf(y, y, ss);
+    }
+    const float inv = a.out_scale / sqrtf(prb_warp_sum(ss) / (float)part + a.eps);
+    for (int i = lane; i < part; i += 32) {
+        const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
+        o[lo + i] = prb_from_float<O>(y * inv * a.norm_w[lo + i]);
     }
 }
 
-// The saved inputs after request b's portion [t0, t1): what is read lies at or behind what is written.
-__device__ __forceinline__ void save_inputs(const SsmArgs& a, int slot, int t0, int t1) {
-    if (a.taps < 2) return;
-    const int channels = a.heads * a.vdim + 2 * a.groups * a.dim, keep = a.taps - 1, n = t1 - t0;
-    for (int ch = threadIdx.x; ch < channels; ch += blockDim.x) {
-        float* st = a.conv_state + (size_t)slot * keep * channels + ch;
-        for (int j = 0; j < keep; ++j) {
-            const int src = j + n;                   // place in [saved inputs | the portion]
-            st[(size_t)j * channels] = src < keep ? st[(size_t)src * channels]
-                                                  : a.proj[(size_t)(t0 + src - keep) * a.ld + a.x_col + ch];
-        }
-    }
-}
-
+// Every part of one token's row by the CTA (few parts: the CTA a part; many: a warp a part).
+constexpr int FIN_KEPT = 8;
 template <typename O>
-__global__ void __launch_bounds__(256) ssm_finish_kernel(SsmArgs a, int gate_here) {
-    __shared__ float scratch[32];
+__device__ __forceinline__ void norm_row_cta(const SsmArgs& a, const float* row, int t, float* scratch) {
+    const int part = a.heads * a.vdim / a.parts;
+    O* o = (O*)a.out + (size_t)t * a.out_ld;
+    if (a.parts >= 4) {
+        for (int p = threadIdx.x >> 5; p < a.parts; p += blockDim.x >> 5)
+            norm_part_warp<O>(a, row, nullptr, o, p * part, part, threadIdx.x & 31);
+        return;
+    }
+    for (int p = 0; p < a.parts; ++p) {
+        const int lo = p * part;
+        float y[FIN_KEPT], ss = 0.0f;
+#pragma unroll
+        for (int k = 0; k < FIN_KEPT; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            y[k] = i < part ? row[lo + i] : 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < FIN_KEPT; ++k) ss = fmaf(y[k], y[k], ss);
+        for (int i = threadIdx.x + FIN_KEPT * blockDim.x; i < part; i += blockDim.x)
+            ss = fmaf(row[lo + i], row[lo + i], ss);
+        ss = prb_block_sum(ss, scratch);
+        const float inv = a.out_scale / sqrtf(ss / (float)part + a.eps);
+#pragma unroll
+        for (int k = 0; k < FIN_KEPT; ++k) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < part) o[lo + i] = prb_from_float<O>(y[k] * inv * a.norm_w[lo + i]);
+        }
+        for (int i = threadIdx.x + FIN_KEPT * blockDim.x; i < part; i += blockDim.x)
+            o[lo + i] = prb_from_float<O>(row[lo + i] * inv * a.norm_w[lo + i]);
+    }
+}
+
+// Warps (token, part); the first part's warp of one of a portion's last `taps` tokens saves the
+// token's inputs.
+constexpr int FIN_WARPS = 4;
+template <typename O>
+__global__ void __launch_bounds__(FIN_WARPS * 32) ssm_finish_kernel(SsmArgs a, int gate_here) {
     prb_grid_launch_dependents();
-    const int t = blockIdx.x, b = a.seq[t];
+    const int lane = threadIdx.x & 31;
+    const long unit = (long)blockIdx.x * FIN_WARPS + (threadIdx.x >> 5);
+    if (unit >= (long)a.n_tokens * a.parts) return;
+    const int t = (int)(unit / a.parts), p = (int)(unit - (long)t * a.parts), b = a.seq[t];
     if (b < 0) return;
-    norm_in_parts<O>(a, a.raw + (size_t)t * a.raw_ld,
-                     gate_here ? a.proj + (size_t)t * a.ld + a.z_col : nullptr, t, scratch);
-    const int t0 = a.q_start[b], t1 = a.q_start[b + 1], slot = a.state_slot[b];
-    if (t == t1 - 1 && t0 >= 0 && slot >= 0 && slot < a.n_slots) save_inputs(a, slot, t0, t1);
+    const int part = a.heads * a.vdim / a.parts;
+    norm_part_warp<O>(a, a.raw + (size_t)t * a.raw_ld, gate_here ? a.proj + (size_t)t * a.ld + a.z_col : nullptr,
+                      (O*)a.out + (size_t)t * a.out_ld, p * part, part, lane);
+    const int slot = a.state_slot[b];
+    if (p != 0 || a.taps < 2 || t < a.q_start[b + 1] - a.taps || slot < 0 || slot >= a.n_slots) return;
+    const int channels = a.heads * a.vdim + 2 * a.groups * a.dim;
+    float* st = a.conv_state + ((size_t)slot * a.taps + a.positions[t] % a.taps) * channels;
+    const float* from = a.proj + (size_t)t * a.ld + a.x_col;
+#pragma unroll 4
+    for (int ch = lane; ch < channels; ch += 32) st[ch] = from[ch];
 }
 
 // ------------------------------------------------------------------- single tokens
@@ -533,6 +580,7 @@ struct StepArgs {
     int* arrived;                    // [requests], zero between launches
 };
 
+constexpr int SS_CC = 4;             // value columns a thread holds
 template <int KPL, typename O>
 __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     extern __shared__ __align__(16) float sm[];
@@ -552,11 +600,11 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     const bool run = t1 > t && t >= 0 && t1 <= a.n_tokens && slot >= 0 && slot < a.n_slots;
     const int pos = run ? a.positions[t] : 0;
     const int ln = threadIdx.x % L, cl = threadIdx.x / L;
-    const int c0 = cg * cols + cl * DS_CC;
-    const bool mine = cl * DS_CC < cols && c0 < V;
+    const int c0 = cg * cols + cl * SS_CC;
+    const bool mine = cl * SS_CC < cols && c0 < V;
     float* sp = a.state + ((size_t)(run ? slot : 0) * a.heads + hd) * V * N;
-    float S[DS_CC][KPL];
-    load_state<KPL>(S, run && pos > 0 && mine ? sp : nullptr, ln, c0, N, V);
+    float S[SS_CC][KPL];
+    load_state<SS_CC, KPL>(S, run && pos > 0 && mine ? sp : nullptr, ln, c0, N, V);
     const int inner = a.heads * V, channels = inner + 2 * a.groups * N, grp = hd / (a.heads / a.groups);
     const int first = cg * cols, live = max(0, min(cols, V - first));
     auto channel_of = [&](int i) {                   // [own x columns | B | C] -> channel
@@ -566,13 +614,16 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     const int todo = live + 2 * N;
     for (int i = threadIdx.x; i < todo; i += blockDim.x) {
         const int ch = channel_of(i);
-        float s = a.conv_b[ch];
-        for (int j = 0; j < a.taps - 1; ++j) {
+        float s = a.conv_b[ch], w[SSM_TAPS - 1], u[SSM_TAPS - 1];
+#pragma unroll
+        for (int j = 0; j < SSM_TAPS - 1; ++j) {
             const int m = a.taps - 1 - j;            // tokens ago
-            if (run && m <= pos)
-                s = fmaf(a.conv_w[(size_t)j * channels + ch],
-                         a.conv_state[((size_t)slot * (a.taps - 1) + j) * channels + ch], s);
+            const bool have = run && m >= 1 && m <= pos;
+            w[j] = have ? a.conv_w[(size_t)j * channels + ch] : 0.0f;
+            u[j] = have ? a.conv_state[((size_t)slot * a.taps + (pos - m) % a.taps) * channels + ch] : 0.0f;
         }
+#pragma unroll
+        for (int j = 0; j < SSM_TAPS - 1; ++j) s = fmaf(w[j], u[j], s);
         h_s[i] = s;
         h_s[todo + i] = a.conv_w[(size_t)(a.taps - 1) * channels + ch];
     }
@@ -584,7 +635,11 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     }
     const float* row = a.proj + (size_t)t * a.ld;
     for (int i = threadIdx.x; i < todo; i += blockDim.x) {   // (the same thread as above)
-        const float u = silu(fmaf(h_s[todo + i], row[a.x_col + channel_of(i)], h_s[i]));
+        const float in = row[a.x_col + channel_of(i)];
+        const float u = silu(fmaf(h_s[todo + i], in, h_s[i]));
+        // (a channel is saved by the one CTA that owns it; B and C by the group's first)
+        if (a.taps > 1 && (i < live || (cg == 0 && hd % (a.heads / a.groups) == 0)))
+            a.conv_state[((size_t)slot * a.taps + pos % a.taps) * channels + channel_of(i)] = in;
         if (i < live) v_s[i] = u;
         else if (i < live + N) k_s[i - live] = u;
         else q_s[i - live - N] = u;
@@ -593,24 +648,24 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     const float dt = softplus(row[a.dt_col + hd] + dtb);
     const float c1 = expm1f(na * dt);
     __syncthreads();
-    float v[DS_CC], x[DS_CC], part[DS_CC];
+    float v[SS_CC], x[SS_CC], part[SS_CC];
 #pragma unroll
-    for (int j = 0; j < DS_CC; ++j) {
-        x[j] = mine && cl * DS_CC + j < live ? v_s[cl * DS_CC + j] : 0.0f;
+    for (int j = 0; j < SS_CC; ++j) {
+        x[j] = mine && cl * SS_CC + j < live ? v_s[cl * SS_CC + j] : 0.0f;
         v[j] = x[j] * dt;
     }
-    advance<KPL, false, true>(S, k_s + ln * KPL, &c1, q_s + ln * KPL, v, part);
-    const float sum = close_columns(part, ln, L);
-    if (mine && (ln & ((L >> 2) - 1)) == 0) {
-        const int j = held_column(ln, L);
-        if (cl * DS_CC + j < live) {
+    advance<SS_CC, KPL, false, true>(S, k_s + ln * KPL, &c1, q_s + ln * KPL, v, part);
+    const float sum = close_columns<SS_CC>(part, ln, L);
+    if (mine && (ln & (L / SS_CC - 1)) == 0) {
+        const int j = held_column<SS_CC>(ln, L);
+        if (cl * SS_CC + j < live) {
             const float xv = j == 0 ? x[0] : j == 1 ? x[1] : j == 2 ? x[2] : x[3];
             const float z = row[a.z_col + hd * V + c0 + j];
             a.raw[(size_t)t * a.raw_ld + hd * V + c0 + j] = fmaf(dd, xv, sum) * silu(z);
         }
     }
-    if (mine) store_state<KPL>(S, sp, ln, c0, N, V);
-    // the request's last CTA to arrive has everything: norm and saved inputs
+    if (mine) store_state<SS_CC, KPL>(S, sp, ln, c0, N, V);
+    // the request's last CTA to arrive norms the token
     __threadfence();
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -621,8 +676,7 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     if (!last_s) return;
     __threadfence();
     if (threadIdx.x == 0) g.arrived[b] = 0;
-    norm_in_parts<O>(a, a.raw + (size_t)t * a.raw_ld, nullptr, t, scratch);
-    save_inputs(a, slot, t, t + 1);
+    norm_row_cta<O>(a, a.raw + (size_t)t * a.raw_ld, t, scratch);
 }
 
 size_t own_smem(int V, int N) {
@@ -668,12 +722,11 @@ PRB_API int prb_ssm_prepare(SSM_PARAMS, void* xbc, long xbc_ld, int xbc_dtype, f
     if (!sizes_ok(a)) return PRB_E_SIZE;
     const int channels = heads * vdim + 2 * groups * dim;
     const dim3 grid((n_tokens + SP_TOKENS - 1) / SP_TOKENS, (channels + 255) / 256 + 1);
-    if (xbc_dtype == PRB_F32)
-        ssm_prepare_kernel<float><<<grid, 256, 0, stream>>>(a, (float*)xbc, xbc_ld, dt, decay, as_log);
-    else if (xbc_dtype == PRB_BF16)
-        ssm_prepare_kernel<bf16><<<grid, 256, 0, stream>>>(a, (bf16*)xbc, xbc_ld, dt, decay, as_log);
-    else
-        return PRB_E_DTYPE;
+#define PREP(XT, TP) ssm_prepare_kernel<XT, TP><<<grid, 256, 0, stream>>>(a, (XT*)xbc, xbc_ld, dt, decay, as_log)
+    if (xbc_dtype == PRB_F32) { if (taps <= 4) PREP(float, 4); else PREP(float, SSM_TAPS); }
+    else if (xbc_dtype == PRB_BF16) { if (taps <= 4) PREP(bf16, 4); else PREP(bf16, SSM_TAPS); }
+    else return PRB_E_DTYPE;
+#undef PREP
     PRB_LAUNCH_CHECK();
     return 0;
 }
@@ -703,11 +756,11 @@ PRB_API int prb_ssm_chunks(SSM_PARAMS, const void* xbc, long xbc_ld, const float
     do {                                                                                                  \
         if (s2 > 40 * 1024)                                                                               \
             cudaFuncSetAttribute(ssm_out_kernel<VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2); \
-        ssm_out_kernel<VT><<<grid, 128, s2, stream>>>(c);                                                 \
+        ssm_out_kernel<VT><<<grid, 256, s2, stream>>>(c);                                                 \
     } while (0)
-    if (vdim <= 32) OUTRUN(4);
-    else if (vdim <= 64) OUTRUN(8);
-    else OUTRUN(16);
+    if (vdim <= 32) OUTRUN(2);
+    else if (vdim <= 64) OUTRUN(4);
+    else OUTRUN(8);
 #undef OUTRUN
     PRB_LAUNCH_CHECK();
     return 0;
@@ -718,8 +771,9 @@ PRB_API int prb_ssm_finish(SSM_PARAMS, int gate_here, int out_dtype, cudaStream_
     const SsmArgs a = SSM_ARGS;
     if (n_tokens <= 0) return 0;
     if (!sizes_ok(a)) return PRB_E_SIZE;
-    if (out_dtype == PRB_F32) ssm_finish_kernel<float><<<n_tokens, 256, 0, stream>>>(a, gate_here);
-    else if (out_dtype == PRB_BF16) ssm_finish_kernel<bf16><<<n_tokens, 256, 0, stream>>>(a, gate_here);
+    const unsigned blocks = (unsigned)(((long)n_tokens * parts + FIN_WARPS - 1) / FIN_WARPS);
+    if (out_dtype == PRB_F32) ssm_finish_kernel<float><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here);
+    else if (out_dtype == PRB_BF16) ssm_finish_kernel<bf16><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here);
     else return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();
     return 0;
@@ -727,10 +781,10 @@ PRB_API int prb_ssm_finish(SSM_PARAMS, int gate_here, int out_dtype, cudaStream_
 
 static int step_cols(int vdim, int dim, int ctas) {
     const int lanes = lanes_of(dim);
-    int cols = (vdim + DS_CC - 1) / DS_CC * DS_CC;
-    while (cols > DS_CC && (cols / DS_CC * lanes > 512 ||
+    int cols = (vdim + SS_CC - 1) / SS_CC * SS_CC;
+    while (cols > SS_CC && (cols / SS_CC * lanes > 512 ||
                             (long)ctas * ((vdim + cols - 1) / cols) < prb_sm_count() / 2))
-        cols = (cols / DS_CC + 1) / 2 * DS_CC;
+        cols = (cols / SS_CC + 1) / 2 * SS_CC;
     return cols;
 }
 
@@ -744,7 +798,7 @@ PRB_API int prb_ssm_step(SSM_PARAMS, int* arrived, int out_dtype, cudaStream_t s
     const int lanes = lanes_of(dim), kpl = keys_per_lane(dim);
     const int cols = step_cols(vdim, dim, heads * n_requests);
     StepArgs g{a, (vdim + cols - 1) / cols, cols, lanes, arrived};
-    const int threads = max((cols / DS_CC * lanes + 31) / 32 * 32, 128);
+    const int threads = max((cols / SS_CC * lanes + 31) / 32 * 32, 256);
     const size_t smem = (size_t)(2 * lanes * kpl + cols + 2 * (cols + 2 * dim)) * sizeof(float);
     const dim3 grid(heads * g.splits, n_requests);
     cudaError_t e;

@@ -10,8 +10,9 @@ rows of ``state`` numbers (head h uses group h / (heads / groups)), dt one numbe
     S_t = a_t S_(t-1) + dt_t B_t x_t^T           y_t = S_t^T C_t + D x_t          (S_(-1) = 0)
 
 y (heads side by side) is multiplied by silu(z), RMS-normed in ``norm_parts`` equal parts, multiplied
-by a weight and projected.  S and the convolution's last ``taps - 1`` inputs are per-request STATE of
-the cache manager (a slot per live request, zero at position 0), so a prompt may be cut anywhere.
+by a weight and projected.  S and the convolution's last inputs are per-request STATE of the cache
+manager (a slot per live request, zero at position 0; the input of position p lies in row p mod
+``taps``), so a prompt may be cut anywhere.
 
 A step of single tokens is one launch.  Steps with portions: convolution, step sizes and decays; the
 recurrence in segments of 64 tokens side by side; the norm.  In bfloat16 the segments' products run
@@ -95,7 +96,7 @@ class StateSpace(Mixer):
     def state_specs(self):
         specs = [StateSpec("ssm_state", (self.heads, self.vdim, self.state_dim), torch.float32)]
         if self.taps > 1:
-            specs.append(StateSpec("ssm_inputs", (self.taps - 1, self.channels), torch.float32))
+            specs.append(StateSpec("ssm_inputs", (self.taps, self.channels), torch.float32))
         return specs
 
     def step_bytes(self, context: int) -> int:

@@ -65,6 +65,16 @@ def log1p_exp(z: torch.Tensor) -> torch.Tensor:
     return torch.clamp(z, min=0.0) + torch.log1p(torch.exp(-z.abs()))
 
 
+def exact(t: torch.Tensor) -> torch.Tensor:
+    return t
+
+
+def to_bfloat16(t: torch.Tensor) -> torch.Tensor:
+    """What storing ``t`` in bfloat16 leaves of it.  Mixers and feed-forwards take ``r``: ``exact``, or
+    this, applied to what serving in bfloat16 stores between two products."""
+    return t.to(torch.bfloat16).to(F64)
+
+
 # ----------------------------------------------------------------------------- attention
 def angle_table(rot: dict):
     """(frequencies, magnitude).  Without ``scaling``: base^(-2i/dims), 1.  With it, pair i keeps
@@ -120,7 +130,7 @@ def sliding_attention(q, k, v, scale: float, window: Optional[int]) -> torch.Ten
     return out
 
 
-def attention_mixer(W, p: str, mx: dict, h, positions) -> torch.Tensor:
+def attention_mixer(W, p: str, mx: dict, h, positions, r=exact) -> torch.Tensor:
     """Biased projections, rotated queries and keys, a window, a gate per head, a biased output."""
     T = h.shape[0]
     H, G, D, V = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
@@ -128,9 +138,9 @@ def attention_mixer(W, p: str, mx: dict, h, positions) -> torch.Tensor:
     k = (h @ W[p + "k"].T + W[p + "k.b"]).reshape(T, G, D)
     v = (h @ W[p + "v"].T + W[p + "v.b"]).reshape(T, G, V)
     q, k = turn_pairs(q, positions, mx.get("rot")), turn_pairs(k, positions, mx.get("rot"))
-    o = sliding_attention(q, k, v, mx["scale"], (mx.get("mask") or {}).get("size"))
+    o = sliding_attention(q, r(k), r(v), mx["scale"], (mx.get("mask") or {}).get("size"))
     o = o * torch.sigmoid(h @ W[p + "g"].T)[:, :, None]
-    return o.reshape(T, H * V) @ W[p + "o"].T + W[p + "o.b"]
+    return r(o).reshape(T, H * V) @ W[p + "o"].T + W[p + "o.b"]
 
 
 # ---------------------------------------------------------------------- recurrent mixers
@@ -146,7 +156,7 @@ def decayed_memory(q, k, v, log_decay) -> torch.Tensor:
     return out
 
 
-def gated_linear_mixer(W, p: str, mx: dict, h, eps: float) -> torch.Tensor:
+def gated_linear_mixer(W, p: str, mx: dict, h, eps: float, r=exact) -> torch.Tensor:
     T = h.shape[0]
     H, D, V = mx["heads"], mx["dim"], mx["vdim"]
     q = (h @ W[p + "q"].T).reshape(T, H, D) * D ** -0.5
@@ -155,7 +165,7 @@ def gated_linear_mixer(W, p: str, mx: dict, h, eps: float) -> torch.Tensor:
     z = (h @ W[p + "a1"].T) @ W[p + "a2"].T + W[p + "a2.b"]
     log_decay = (-log1p_exp(-z) / mx["tau"]).reshape(T, H, D)
     o = unit_rms(decayed_memory(q, k, v, log_decay), eps) * W[p + "norm"]
-    return (o.reshape(T, H * V) * silu(h @ W[p + "g"].T)) @ W[p + "o"].T
+    return r(o.reshape(T, H * V) * silu(h @ W[p + "g"].T)) @ W[p + "o"].T
 
 
 def causal_convolution(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
@@ -169,14 +179,14 @@ def causal_convolution(x: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor) 
     return out
 
 
-def state_space_mixer(W, p: str, mx: dict, h, eps: float) -> torch.Tensor:
+def state_space_mixer(W, p: str, mx: dict, h, eps: float, r=exact) -> torch.Tensor:
     """A scalar decay per head and token, keys B and queries C shared by a group's heads, step
     sizes on the keys, a direct path D, the gate before a norm in equal parts."""
     T = h.shape[0]
     H, V, N, G = mx["heads"], mx["vdim"], mx["state"], mx["groups"]
     inner = H * V
     z, xbc, dt = torch.split(h @ W[p + "in"].T, [inner, inner + 2 * G * N, H], dim=1)
-    xbc = silu(causal_convolution(xbc, W[p + "conv"], W[p + "conv.b"]))
+    xbc = r(silu(causal_convolution(xbc, W[p + "conv"], W[p + "conv.b"])))
     x, B, C = torch.split(xbc, [inner, G * N, G * N], dim=1)
     x = x.reshape(T, H, V)
     B = B.reshape(T, G, N).repeat_interleave(H // G, dim=1)
@@ -185,66 +195,71 @@ def state_space_mixer(W, p: str, mx: dict, h, eps: float) -> torch.Tensor:
     log_decay = (-torch.exp(W[p + "A_log"]) * dt)[:, :, None].expand(T, H, N)
     y = decayed_memory(C, B * dt[:, :, None], x, log_decay) + W[p + "D"][:, None] * x
     y = (y.reshape(T, inner) * silu(z)).reshape(T, mx["norm_groups"], -1)
-    return (unit_rms(y, eps).reshape(T, inner) * W[p + "norm"]) @ W[p + "o"].T
+    return r(unit_rms(y, eps).reshape(T, inner) * W[p + "norm"]) @ W[p + "o"].T
 
 
 # ------------------------------------------------------------------------- feed-forwards
-def gated_unit(W, p: str, h) -> torch.Tensor:
-    return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+def gated_unit(W, p: str, h, r=exact) -> torch.Tensor:
+    return r(silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
-def routed_unit(W, p: str, mlp: dict, h) -> torch.Tensor:
+def routed_unit(W, p: str, mlp: dict, h, margins: Optional[list] = None, r=exact) -> torch.Tensor:
     """Softmax scores over all experts; chosen by score + correction, weighted by the score
-    alone; the last ``identity`` experts give back their input; a gated shared expert."""
-    r = mlp["router"]
-    real = r["experts"]
+    alone; the last ``identity`` experts give back their input; a gated shared expert.
+    ``margins`` collects how far the last chosen and the first unchosen expert lie apart [T]."""
+    router = mlp["router"]
+    real, top = router["experts"], router["top"]
     scores = torch.softmax(h @ W[p + "router"].T, dim=-1)
-    chosen = torch.topk(scores + W[p + "correction"], r["top"], dim=-1).indices
+    choice = scores + W[p + "correction"]
+    chosen = torch.topk(choice, top, dim=-1).indices
+    if margins is not None and top < choice.shape[1]:
+        ranked = choice.sort(dim=-1, descending=True).values
+        margins.append(ranked[:, top - 1] - ranked[:, top])
     weight = torch.zeros_like(scores).scatter(1, chosen, scores.gather(1, chosen))
     out = weight[:, real:].sum(-1, keepdim=True) * h
     for e in range(real):
-        out = out + weight[:, e:e + 1] * gated_unit(W, f"{p}e{e}.", h)
+        out = out + weight[:, e:e + 1] * gated_unit(W, f"{p}e{e}.", h, r)
     if mlp.get("shared"):
-        out = out + torch.sigmoid(h @ W[p + "shared.sg"].T) * gated_unit(W, p + "shared.", h)
+        out = out + torch.sigmoid(h @ W[p + "shared.sg"].T) * gated_unit(W, p + "shared.", h, r)
     return out
 
 
-def feed_forward(W, p: str, mlp: dict, h) -> torch.Tensor:
+def feed_forward(W, p: str, mlp: dict, h, margins: Optional[list] = None, r=exact) -> torch.Tensor:
     if mlp["kind"] == "dense":
-        return torch.relu(h @ W[p + "up"].T).pow(2) @ W[p + "down"].T
-    return routed_unit(W, p, mlp, h)
+        return r(torch.relu(h @ W[p + "up"].T).pow(2)) @ W[p + "down"].T
+    return routed_unit(W, p, mlp, h, margins, r)
 
 
 # ------------------------------------------------------------------------------ the model
-def mixer(W, p: str, layer: dict, h, positions, eps: float) -> torch.Tensor:
+def mixer(W, p: str, layer: dict, h, positions, eps: float, r=exact) -> torch.Tensor:
     mx = layer["mixer"]
     if layer["type"] == "mamba2":
-        return state_space_mixer(W, p, mx, h, eps)
-    return mx["left_scale"] * attention_mixer(W, p + "left.", mx["left"], h, positions) + \
-        mx["right_scale"] * gated_linear_mixer(W, p + "right.", mx["right"], h, eps)
+        return state_space_mixer(W, p, mx, h, eps, r)
+    return mx["left_scale"] * attention_mixer(W, p + "left.", mx["left"], h, positions, r) + \
+        mx["right_scale"] * gated_linear_mixer(W, p + "right.", mx["right"], h, eps, r)
 
 
 def forward(tokens: List[int], W: Dict[str, torch.Tensor], cfg: dict,
-            taps: Optional[list] = None, rounded: bool = False) -> torch.Tensor:
-    """Logits [T, vocab] of one sequence; ``taps`` collects the stream after every layer.
-    ``rounded``: every layer's normed input is rounded to bfloat16 (the least that serving in
-    bfloat16 does to it); the difference to the exact run says how far rounding alone moves a
-    row."""
+            taps: Optional[list] = None, rounded: bool = False,
+            margins: Optional[list] = None) -> torch.Tensor:
+    """Logits [T, vocab] of one sequence; ``taps`` collects the stream after every layer,
+    ``margins`` the routers' margins (see ``routed_unit``).
+    ``rounded``: what serving in bfloat16 stores between two products is rounded to it; the
+    difference to the exact run says how far rounding alone moves a row."""
     eps = cfg["norm"]["eps"]
+    r = to_bfloat16 if rounded else exact
     positions = torch.arange(len(tokens))
     x = offset_norm(W["embed"][tokens], W["embed.norm"], eps)
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
-        h = offset_norm(x, W[p + "norm1"], eps)
-        if rounded:
-            h = h.to(torch.bfloat16).to(F64)
-        y = mixer(W, p + "mix.", layer, h, positions, eps)
+        h = r(offset_norm(x, W[p + "norm1"], eps))
+        y = mixer(W, p + "mix.", layer, h, positions, eps, r)
         if layer.get("mlp"):
-            y = y + feed_forward(W, p + "mlp.", layer["mlp"], h)
+            y = y + feed_forward(W, p + "mlp.", layer["mlp"], h, margins, r)
         x = x + y
         if taps is not None:
             taps.append(x.clone())
-    return offset_norm(x, W["final.norm"], eps) @ W["head"].T
+    return r(offset_norm(x, W["final.norm"], eps)) @ W["head"].T
 
 
 def greedy(prompt: List[int], n_new: int, W: Dict[str, torch.Tensor], cfg: dict) -> List[int]:
