@@ -51,6 +51,16 @@ template <> __device__ __forceinline__ __nv_bfloat16 prb_from_float<__nv_bfloat1
     return __float2bfloat16_rn(v);
 }
 
+// Four neighbouring numbers in one piece (o aligned to 4 elements).
+__device__ __forceinline__ void prb_store4(float* o, float a, float b, float c, float d) {
+    *reinterpret_cast<float4*>(o) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ void prb_store4(__nv_bfloat16* o, float a, float b, float c, float d) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    *reinterpret_cast<uint2*>(o) =
+        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
 __device__ __forceinline__ float prb_warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

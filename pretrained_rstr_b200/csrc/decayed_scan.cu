@@ -183,7 +183,7 @@ __global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
         const float* d_s = v_s - cl + DS_TB * cols;
         const int nb = min(DS_TB, t1 - tb);
         float* o_at = o_to + (a.fin.out ? 0 : (size_t)tb * o_ld);
-#pragma unroll 2
+#pragma unroll 4
         for (int tok = 0; tok < nb; ++tok) {
             float v[DS_CC], part[DS_CC];
 #pragma unroll

@@ -134,7 +134,7 @@ __device__ __forceinline__ int held_column(int ln, int L) {
 }
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 
 // Portions in segments of DS_SEG tokens; segment z of the launch is segment s of request b
 // (requests' segments are numbered in request order).

@@ -11,7 +11,7 @@
 #include "common.cuh"
 
 namespace {
-__device__ __forceinline__ float ea_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float ea_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 __device__ __forceinline__ float ea_gate(float g, int act) {     // 0: silu, 1: gelu (tanh form)
     return act == 1 ? prb_activate(g, PRB_ACT_GELU_TANH) : g * ea_sigmoid(g);
 }
@@ -29,17 +29,6 @@ struct ExpertArgs {
     const float* norm_w;
     float eps;
 };
-
-template <typename O>
-__device__ __forceinline__ void store4(O* o, const float (&v)[4]) {
-    if constexpr (sizeof(O) == 4) {
-        *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
-    } else {
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-        *reinterpret_cast<uint2*>(o) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo),
-                                                  *reinterpret_cast<const uint32_t*>(&hi));
-    }
-}
 
 // Scores, choice and weights of one row, by a warp: wt[e] of every expert, own[0] the identity experts'
 // weight together, own[1] the shared expert's.
@@ -103,88 +92,155 @@ __device__ __forceinline__ void choose(const ExpertArgs& a, const float* row, fl
     }
 }
 
-// x += weight * input of one row, by the CTA.
+struct Columns {
+    int n_exp, n_all, lo, hi;        // the routed experts' columns, all, and this CTA's slice
+    bool vec;
+    __device__ __forceinline__ explicit Columns(const ExpertArgs& a, int esz) {
+        n_exp = a.experts * a.group;
+        n_all = n_exp + a.shared;
+        const int per = ((n_all + (int)gridDim.y - 1) / (int)gridDim.y + 3) / 4 * 4;
+        lo = blockIdx.y * per;
+        hi = min(n_all, lo + per);
+        vec = a.group % 4 == 0 && (a.gate_col | a.up_col | a.in_ld | a.out_ld) % 4 == 0 &&
+              (a.shared == 0 || (a.shared_gate_col | a.shared_up_col | a.shared) % 4 == 0) &&
+              ((uintptr_t)a.in) % 16 == 0 && ((uintptr_t)a.out) % (4 * esz) == 0;
+    }
+    __device__ __forceinline__ int gate(const ExpertArgs& a, int i) const {
+        return i < n_exp ? a.gate_col + i : a.shared_gate_col + i - n_exp;
+    }
+    __device__ __forceinline__ int up(const ExpertArgs& a, int i) const {
+        return i < n_exp ? a.up_col + i : a.shared_up_col + i - n_exp;
+    }
+};
+
+// Few rows: CTAs (row, slice of its columns); every CTA of a row chooses for itself.  Columns are
+// the experts' (experts * group), then the shared expert's.
 template <typename O>
-__device__ __forceinline__ void add_input(const ExpertArgs& a, int t, float w, float* scratch) {
+__global__ void __launch_bounds__(256) expert_act_row_kernel(ExpertArgs a) {
+    extern __shared__ float sh[];                    // [all] scores, [all] choice, [all] weights
+    __shared__ float scratch[32];
+    __shared__ float own_s[2];
+    const int all = a.experts + a.identity, t = blockIdx.x;
+    prb_grid_launch_dependents();
+    const Columns c(a, sizeof(O));
+    const float* row = a.in + (size_t)t * a.in_ld;
+    const float* wt = sh + 2 * all;
+    prb_grid_wait();
+    // the first columns are asked for before anyone knows which experts the row chooses
+    const int first = c.lo + (int)threadIdx.x * 4;
+    float4 g0 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), u0 = g0;
+    if (c.vec && first < c.hi) {
+        g0 = *reinterpret_cast<const float4*>(row + c.gate(a, first));
+        u0 = *reinterpret_cast<const float4*>(row + c.up(a, first));
+    }
+    if (threadIdx.x < 32) choose(a, row, sh, sh + all, sh + 2 * all, own_s);
+    __syncthreads();
+    O* o = (O*)a.out + (size_t)t * a.out_ld;
+    if (c.vec) {
+        for (int i = first; i < c.hi; i += blockDim.x * 4) {
+            const float w = i < c.n_exp ? wt[i / a.group] : own_s[1];
+            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if (w != 0.0f) {                         // (columns of experts not chosen are not read)
+                float4 g = g0, u = u0;
+                if (i != first) {
+                    g = *reinterpret_cast<const float4*>(row + c.gate(a, i));
+                    u = *reinterpret_cast<const float4*>(row + c.up(a, i));
+                }
+                v[0] = w * ea_gate(g.x, a.act) * u.x;
+                v[1] = w * ea_gate(g.y, a.act) * u.y;
+                v[2] = w * ea_gate(g.z, a.act) * u.z;
+                v[3] = w * ea_gate(g.w, a.act) * u.w;
+            }
+            prb_store4(o + i, v[0], v[1], v[2], v[3]);
+        }
+    } else {
+        for (int i = c.lo + threadIdx.x; i < c.hi; i += blockDim.x) {
+            const float w = i < c.n_exp ? wt[i / a.group] : own_s[1];
+            o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(row[c.gate(a, i)], a.act) * row[c.up(a, i)] : 0.0f);
+        }
+    }
+    if (a.identity == 0 || blockIdx.y != 0 || own_s[0] == 0.0f) return;
     float* x = a.x + (size_t)t * a.x_ld;
     if (a.h != nullptr) {
         const O* h = (const O*)a.h + (size_t)t * a.h_ld;
-        for (int i = threadIdx.x; i < a.width; i += blockDim.x) x[i] = fmaf(w, prb_to_float<O>(h[i]), x[i]);
+        for (int i = threadIdx.x; i < a.width; i += blockDim.x)
+            x[i] = fmaf(own_s[0], prb_to_float<O>(h[i]), x[i]);
         return;
     }
     float ss = 0.0f;
     for (int i = threadIdx.x; i < a.width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
     ss = prb_block_sum(ss, scratch);
-    const float inv = w / sqrtf(ss / (float)a.width + a.eps);
+    const float inv = own_s[0] / sqrtf(ss / (float)a.width + a.eps);
     for (int i = threadIdx.x; i < a.width; i += blockDim.x)
         x[i] = fmaf(x[i] * inv, a.norm_w ? a.norm_w[i] : 1.0f, x[i]);
 }
 
-// CTAs (ROWS rows, slice of their columns); every CTA of a row chooses for itself, a warp a row.
-// Columns: the experts' (experts * group), then the shared expert's.
-constexpr int EA_ROWS = 8;
-template <typename O, int ROWS>
-__global__ void __launch_bounds__(256) expert_act_kernel(ExpertArgs a) {
-    extern __shared__ float sh[];                    // per row: [all] scores, [all] choice, [all] weights
-    __shared__ float scratch[32];
-    __shared__ float own_s[ROWS][2];
-    const int all = a.experts + a.identity;
-    prb_grid_launch_dependents();
-    const int t0 = blockIdx.x * ROWS, nt = min(ROWS, a.n_rows - t0);
-    const int n_exp = a.experts * a.group, n_all = n_exp + a.shared;
-    const int per = ((n_all + (int)gridDim.y - 1) / (int)gridDim.y + 3) / 4 * 4;
-    const int lo = blockIdx.y * per, hi = min(n_all, lo + per);
-    const bool vec = a.group % 4 == 0 && (a.gate_col | a.up_col | a.in_ld | a.out_ld) % 4 == 0 &&
-                     (a.shared == 0 || (a.shared_gate_col | a.shared_up_col | a.shared) % 4 == 0) &&
-                     ((uintptr_t)a.in) % 16 == 0 && ((uintptr_t)a.out) % (4 * sizeof(O)) == 0;
-    auto gate_at = [&](int i) { return i < n_exp ? a.gate_col + i : a.shared_gate_col + i - n_exp; };
-    auto up_at = [&](int i) { return i < n_exp ? a.up_col + i : a.shared_up_col + i - n_exp; };
-    prb_grid_wait();
-    // a single row's first columns are asked for before anyone knows which experts it chooses
-    float4 g0 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), u0 = g0;
-    const int first = lo + (int)threadIdx.x * 4;
-    if (ROWS == 1 && vec && first < hi) {
-        const float* row = a.in + (size_t)t0 * a.in_ld;
-        g0 = *reinterpret_cast<const float4*>(row + gate_at(first));
-        u0 = *reinterpret_cast<const float4*>(row + up_at(first));
-    }
-    const int warp = threadIdx.x >> 5;
-    if (warp < nt) {
-        float* mine = sh + (size_t)warp * 3 * all;
-        choose(a, a.in + (size_t)(t0 + warp) * a.in_ld, mine, mine + all, mine + 2 * all, own_s[warp]);
-    }
-    __syncthreads();
-    for (int r = 0; r < nt; ++r) {
-        const float* row = a.in + (size_t)(t0 + r) * a.in_ld;
-        const float* wt = sh + (size_t)r * 3 * all + 2 * all;
-        O* o = (O*)a.out + (size_t)(t0 + r) * a.out_ld;
-        const float shared_w = own_s[r][1];
-        if (vec) {
-            for (int i = first; i < hi; i += blockDim.x * 4) {
-                const float w = i < n_exp ? wt[i / a.group] : shared_w;
-                float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-                if (w != 0.0f) {                     // (columns of experts not chosen are not read)
-                    float4 g = g0, u = u0;
-                    if (ROWS > 1 || i != first) {
-                        g = *reinterpret_cast<const float4*>(row + gate_at(i));
-                        u = *reinterpret_cast<const float4*>(row + up_at(i));
-                    }
-                    v[0] = w * ea_gate(g.x, a.act) * u.x;
-                    v[1] = w * ea_gate(g.y, a.act) * u.y;
-                    v[2] = w * ea_gate(g.z, a.act) * u.z;
-                    v[3] = w * ea_gate(g.w, a.act) * u.w;
-                }
-                store4(o + i, v);
-            }
-        } else {
-            for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) {
-                const float w = i < n_exp ? wt[i / a.group] : shared_w;
-                o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(row[gate_at(i)], a.act) * row[up_at(i)] : 0.0f);
-            }
+// `n` columns of a row by a warp: w * f(gate) * up, or zeros without reading anything.
+template <typename O>
+__device__ __forceinline__ void act_run(O* o, const float* gate, const float* up, int n, float w, int act, bool vec,
+                                        int lane) {
+    if (vec) {
+        if (w == 0.0f) {
+            for (int i = lane * 4; i < n; i += 128) prb_store4(o + i, 0.0f, 0.0f, 0.0f, 0.0f);
+            return;
         }
-        if (a.identity > 0 && blockIdx.y == 0 && own_s[r][0] != 0.0f)
-            add_input<O>(a, t0 + r, own_s[r][0], scratch);
+#pragma unroll 4
+        for (int i = lane * 4; i < n; i += 128) {
+            const float4 g = *reinterpret_cast<const float4*>(gate + i);
+            const float4 u = *reinterpret_cast<const float4*>(up + i);
+            prb_store4(o + i, w * ea_gate(g.x, act) * u.x, w * ea_gate(g.y, act) * u.y, w * ea_gate(g.z, act) * u.z,
+                       w * ea_gate(g.w, act) * u.w);
+        }
+        return;
     }
+    for (int i = lane; i < n; i += 32)
+        o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(gate[i], act) * up[i] : 0.0f);
+}
+
+// Many rows: a warp a row and slice, no barrier.  A slice is every gridDim.y-th expert, the shared
+// expert (in shares) and a share of the identity experts' width.
+constexpr int EA_ROWS = 8;
+template <typename O>
+__global__ void __launch_bounds__(EA_ROWS * 32) expert_act_kernel(ExpertArgs a) {
+    extern __shared__ float sh[];                    // per row: [all] scores, [all] choice, [all] weights
+    __shared__ float own_s[EA_ROWS][2];
+    const int all = a.experts + a.identity, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    prb_grid_launch_dependents();
+    const int t = blockIdx.x * EA_ROWS + warp;
+    if (t >= a.n_rows) return;
+    const bool vec = Columns(a, sizeof(O)).vec;
+    const float* row = a.in + (size_t)t * a.in_ld;
+    float* mine = sh + (size_t)warp * 3 * all;
+    const float* wt = mine + 2 * all;
+    choose(a, row, mine, mine + all, mine + 2 * all, own_s[warp]);
+    __syncwarp();
+    const float identity = own_s[warp][0], shared_w = own_s[warp][1];
+    O* o = (O*)a.out + (size_t)t * a.out_ld;
+    for (int e = blockIdx.y; e < a.experts; e += gridDim.y)
+        act_run<O>(o + (size_t)e * a.group, row + a.gate_col + (size_t)e * a.group,
+                   row + a.up_col + (size_t)e * a.group, a.group, wt[e], a.act, vec, lane);
+    if (a.shared > 0) {
+        const int per = ((a.shared + (int)gridDim.y - 1) / (int)gridDim.y + 3) / 4 * 4;
+        const int lo = blockIdx.y * per, n = min(a.shared - lo, per);
+        if (n > 0)
+            act_run<O>(o + (size_t)a.experts * a.group + lo, row + a.shared_gate_col + lo,
+                       row + a.shared_up_col + lo, n, shared_w, a.act, vec, lane);
+    }
+    if (a.identity == 0 || identity == 0.0f) return;
+    float* x = a.x + (size_t)t * a.x_ld;
+    if (a.h != nullptr) {                            // (every slice a share of the width)
+        const O* h = (const O*)a.h + (size_t)t * a.h_ld;
+        const int per = (a.width + (int)gridDim.y - 1) / (int)gridDim.y;
+        const int end = min(a.width, ((int)blockIdx.y + 1) * per);
+#pragma unroll 4
+        for (int i = blockIdx.y * per + lane; i < end; i += 32) x[i] = fmaf(identity, prb_to_float<O>(h[i]), x[i]);
+        return;
+    }
+    if (blockIdx.y != 0) return;
+    float ss = 0.0f;
+    for (int i = lane; i < a.width; i += 32) ss = fmaf(x[i], x[i], ss);
+    const float inv = identity / sqrtf(prb_warp_sum(ss) / (float)a.width + a.eps);
+    for (int i = lane; i < a.width; i += 32) x[i] = fmaf(x[i] * inv, a.norm_w ? a.norm_w[i] : 1.0f, x[i]);
 }
 
 __device__ __forceinline__ float column_act(float v, int act) {
@@ -207,8 +263,8 @@ __global__ void act_columns_kernel(O* __restrict__ out, long out_ld, const float
         if (idx >= (size_t)n_rows * n4) return;
         const int t = (int)(idx / n4), i = (int)(idx - (size_t)t * n4) * 4;
         const float4 u = *reinterpret_cast<const float4*>(in + (size_t)t * in_ld + i);
-        const float v[4] = {column_act(u.x, act), column_act(u.y, act), column_act(u.z, act), column_act(u.w, act)};
-        store4(out + (size_t)t * out_ld + i, v);
+        prb_store4(out + (size_t)t * out_ld + i, column_act(u.x, act), column_act(u.y, act), column_act(u.z, act),
+                   column_act(u.w, act));
     } else {
         if (idx >= (size_t)n_rows * n) return;
         const int t = (int)(idx / n), i = (int)(idx - (size_t)t * n);
@@ -239,25 +295,25 @@ PRB_API int prb_expert_act(void* out, long out_ld, const float* in, long in_ld, 
         const int slices = columns < 1024 ? 1 : (columns + 1023) / 1024 > 64 ? 64 : (columns + 1023) / 1024;
         const dim3 grid(n_rows, slices);
         const size_t smem = (size_t)3 * all * sizeof(float);
-        if (dtype == PRB_F32) e = prb_launch_dependent(expert_act_kernel<float, 1>, grid, dim3(256), smem, stream, a);
+        if (dtype == PRB_F32) e = prb_launch_dependent(expert_act_row_kernel<float>, grid, dim3(256), smem, stream, a);
         else if (dtype == PRB_BF16)
-            e = prb_launch_dependent(expert_act_kernel<__nv_bfloat16, 1>, grid, dim3(256), smem, stream, a);
+            e = prb_launch_dependent(expert_act_row_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, a);
         else return PRB_E_DTYPE;
     } else {
         const int groups = (n_rows + EA_ROWS - 1) / EA_ROWS;
         int slices = (columns + 1023) / 1024;
         if (slices < 1) slices = 1;
-        while (slices > 1 && (long)groups * slices > 8L * prb_sm_count()) slices = (slices + 1) / 2;
+        while (slices > 1 && (long)groups * slices > 6L * prb_sm_count()) slices = (slices + 1) / 2;
         const dim3 grid(groups, slices);
         const size_t smem = (size_t)3 * EA_ROWS * all * sizeof(float);
         if (smem > 40 * 1024) {
-            cudaFuncSetAttribute(expert_act_kernel<float, EA_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-            cudaFuncSetAttribute(expert_act_kernel<__nv_bfloat16, EA_ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            cudaFuncSetAttribute(expert_act_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            cudaFuncSetAttribute(expert_act_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         }
         if (dtype == PRB_F32)
-            e = prb_launch_maybe_early(false, expert_act_kernel<float, EA_ROWS>, grid, dim3(256), smem, stream, a);
+            e = prb_launch_maybe_early(false, expert_act_kernel<float>, grid, dim3(256), smem, stream, a);
         else if (dtype == PRB_BF16)
-            e = prb_launch_maybe_early(false, expert_act_kernel<__nv_bfloat16, EA_ROWS>, grid, dim3(256), smem, stream, a);
+            e = prb_launch_maybe_early(false, expert_act_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, a);
         else return PRB_E_DTYPE;
     }
     return e == cudaSuccess ? 0 : (int)e;

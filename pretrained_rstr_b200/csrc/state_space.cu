@@ -478,8 +478,8 @@ constexpr int FIN_PIECES = 16;
 template <typename O>
 __device__ __forceinline__ void norm_part_warp(const SsmArgs& a, const float* row, const float* z, O* o, int lo,
                                                int part, int lane) {
-    if (part % 4 == 0 && part <= FIN_PIECES * 128 && (lo | a.raw_ld) % 4 == 0 && ((uintptr_t)a.raw) % 16 == 0 &&
-        z == nullptr) {
+    if (part % 4 == 0 && part <= FIN_PIECES * 128 && (lo | a.raw_ld | a.out_ld) % 4 == 0 && z == nullptr &&
+        (((uintptr_t)a.raw | (uintptr_t)a.norm_w) % 16) == 0 && ((uintptr_t)a.out) % (4 * sizeof(O)) == 0) {
         float4 y[FIN_PIECES];
         float ss = 0.0f;
 #pragma unroll
@@ -493,12 +493,11 @@ __device__ __forceinline__ void norm_part_warp(const SsmArgs& a, const float* ro
         const float inv = a.out_scale / sqrtf(prb_warp_sum(ss) / (float)part + a.eps);
 #pragma unroll
         for (int p = 0; p < FIN_PIECES; ++p) {
-            const int i = lo + p * 128 + lane * 4;
-            if (p * 128 + lane * 4 < part) {
-                o[i] = prb_from_float<O>(y[p].x * inv * a.norm_w[i]);
-                o[i + 1] = prb_from_float<O>(y[p].y * inv * a.norm_w[i + 1]);
-                o[i + 2] = prb_from_float<O>(y[p].z * inv * a.norm_w[i + 2]);
-                o[i + 3] = prb_from_float<O>(y[p].w * inv * a.norm_w[i + 3]);
+            const int i = p * 128 + lane * 4;
+            if (i < part) {
+                const float4 w = *reinterpret_cast<const float4*>(a.norm_w + lo + i);
+                prb_store4(o + lo + i, y[p].x * inv * w.x, y[p].y * inv * w.y, y[p].z * inv * w.z,
+                           y[p].w * inv * w.w);
             }
         }
         return;
@@ -516,7 +515,7 @@ __device__ __forceinline__ void norm_part_warp(const SsmArgs& a, const float* ro
 }
 
 // Every part of one token's row by the CTA (few parts: the CTA a part; many: a warp a part).
-constexpr int FIN_KEPT = 8;
+constexpr int FIN_KEPT = 4;
 template <typename O>
 __device__ __forceinline__ void norm_row_cta(const SsmArgs& a, const float* row, int t, float* scratch) {
     const int part = a.heads * a.vdim / a.parts;
@@ -550,27 +549,38 @@ __device__ __forceinline__ void norm_row_cta(const SsmArgs& a, const float* row,
     }
 }
 
-// Warps (token, part); the first part's warp of one of a portion's last `taps` tokens saves the
-// token's inputs.
-constexpr int FIN_WARPS = 4;
+// Warps (token, part); behind them CTAs that save inputs: (request, one of its portion's last `taps`
+// tokens, 512 channels).
+constexpr int FIN_WARPS = 4, SAVE_CHANNELS = 512;
 template <typename O>
-__global__ void __launch_bounds__(FIN_WARPS * 32) ssm_finish_kernel(SsmArgs a, int gate_here) {
+__global__ void __launch_bounds__(FIN_WARPS * 32) ssm_finish_kernel(SsmArgs a, int gate_here, int norm_blocks) {
     prb_grid_launch_dependents();
+    if ((int)blockIdx.x >= norm_blocks) {
+        const int channels = a.heads * a.vdim + 2 * a.groups * a.dim;
+        const int pieces = (channels + SAVE_CHANNELS - 1) / SAVE_CHANNELS;
+        int e = blockIdx.x - norm_blocks;
+        const int piece = e % pieces;
+        e /= pieces;
+        const int back = e % a.taps, b = e / a.taps;
+        const int t = a.q_start[b + 1] - 1 - back, slot = a.state_slot[b];
+        if (t < a.q_start[b] || t < 0 || t >= a.n_tokens || slot < 0 || slot >= a.n_slots) return;
+        float* st = a.conv_state + ((size_t)slot * a.taps + a.positions[t] % a.taps) * channels;
+        const float* from = a.proj + (size_t)t * a.ld + a.x_col;
+#pragma unroll
+        for (int k = 0; k < SAVE_CHANNELS / (FIN_WARPS * 32); ++k) {
+            const int ch = piece * SAVE_CHANNELS + k * FIN_WARPS * 32 + (int)threadIdx.x;
+            if (ch < channels) st[ch] = from[ch];
+        }
+        return;
+    }
     const int lane = threadIdx.x & 31;
     const long unit = (long)blockIdx.x * FIN_WARPS + (threadIdx.x >> 5);
     if (unit >= (long)a.n_tokens * a.parts) return;
-    const int t = (int)(unit / a.parts), p = (int)(unit - (long)t * a.parts), b = a.seq[t];
-    if (b < 0) return;
+    const int t = (int)(unit / a.parts), p = (int)(unit - (long)t * a.parts);
+    if (a.seq[t] < 0) return;
     const int part = a.heads * a.vdim / a.parts;
     norm_part_warp<O>(a, a.raw + (size_t)t * a.raw_ld, gate_here ? a.proj + (size_t)t * a.ld + a.z_col : nullptr,
                       (O*)a.out + (size_t)t * a.out_ld, p * part, part, lane);
-    const int slot = a.state_slot[b];
-    if (p != 0 || a.taps < 2 || t < a.q_start[b + 1] - a.taps || slot < 0 || slot >= a.n_slots) return;
-    const int channels = a.heads * a.vdim + 2 * a.groups * a.dim;
-    float* st = a.conv_state + ((size_t)slot * a.taps + a.positions[t] % a.taps) * channels;
-    const float* from = a.proj + (size_t)t * a.ld + a.x_col;
-#pragma unroll 4
-    for (int ch = lane; ch < channels; ch += 32) st[ch] = from[ch];
 }
 
 // ------------------------------------------------------------------- single tokens
@@ -581,8 +591,8 @@ struct StepArgs {
 };
 
 constexpr int SS_CC = 4;             // value columns a thread holds
-template <int KPL, typename O>
-__global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
+template <int KPL, int TAPS, typename O>
+__global__ void __launch_bounds__(512, KPL == 4 ? 2 : 1) ssm_step_kernel(StepArgs g) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float scratch[32];
     __shared__ int last_s;
@@ -614,16 +624,16 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     const int todo = live + 2 * N;
     for (int i = threadIdx.x; i < todo; i += blockDim.x) {
         const int ch = channel_of(i);
-        float s = a.conv_b[ch], w[SSM_TAPS - 1], u[SSM_TAPS - 1];
+        float s = a.conv_b[ch], w[TAPS - 1], u[TAPS - 1];
 #pragma unroll
-        for (int j = 0; j < SSM_TAPS - 1; ++j) {
+        for (int j = 0; j < TAPS - 1; ++j) {
             const int m = a.taps - 1 - j;            // tokens ago
             const bool have = run && m >= 1 && m <= pos;
             w[j] = have ? a.conv_w[(size_t)j * channels + ch] : 0.0f;
             u[j] = have ? a.conv_state[((size_t)slot * a.taps + (pos - m) % a.taps) * channels + ch] : 0.0f;
         }
 #pragma unroll
-        for (int j = 0; j < SSM_TAPS - 1; ++j) s = fmaf(w[j], u[j], s);
+        for (int j = 0; j < TAPS - 1; ++j) s = fmaf(w[j], u[j], s);
         h_s[i] = s;
         h_s[todo + i] = a.conv_w[(size_t)(a.taps - 1) * channels + ch];
     }
@@ -634,6 +644,10 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
         return;
     }
     const float* row = a.proj + (size_t)t * a.ld;
+    // the column of this lane's sum, and its gate
+    const int held = held_column<SS_CC>(ln, L);
+    const bool writes = mine && (ln & (L / SS_CC - 1)) == 0 && cl * SS_CC + held < live;
+    const float z = writes ? row[a.z_col + hd * V + c0 + held] : 0.0f;
     for (int i = threadIdx.x; i < todo; i += blockDim.x) {   // (the same thread as above)
         const float in = row[a.x_col + channel_of(i)];
         const float u = silu(fmaf(h_s[todo + i], in, h_s[i]));
@@ -648,22 +662,13 @@ __global__ void __launch_bounds__(512) ssm_step_kernel(StepArgs g) {
     const float dt = softplus(row[a.dt_col + hd] + dtb);
     const float c1 = expm1f(na * dt);
     __syncthreads();
-    float v[SS_CC], x[SS_CC], part[SS_CC];
+    float v[SS_CC], part[SS_CC];
 #pragma unroll
-    for (int j = 0; j < SS_CC; ++j) {
-        x[j] = mine && cl * SS_CC + j < live ? v_s[cl * SS_CC + j] : 0.0f;
-        v[j] = x[j] * dt;
-    }
+    for (int j = 0; j < SS_CC; ++j) v[j] = mine && cl * SS_CC + j < live ? v_s[cl * SS_CC + j] * dt : 0.0f;
     advance<SS_CC, KPL, false, true>(S, k_s + ln * KPL, &c1, q_s + ln * KPL, v, part);
     const float sum = close_columns<SS_CC>(part, ln, L);
-    if (mine && (ln & (L / SS_CC - 1)) == 0) {
-        const int j = held_column<SS_CC>(ln, L);
-        if (cl * SS_CC + j < live) {
-            const float xv = j == 0 ? x[0] : j == 1 ? x[1] : j == 2 ? x[2] : x[3];
-            const float z = row[a.z_col + hd * V + c0 + j];
-            a.raw[(size_t)t * a.raw_ld + hd * V + c0 + j] = fmaf(dd, xv, sum) * silu(z);
-        }
-    }
+    if (writes)
+        a.raw[(size_t)t * a.raw_ld + hd * V + c0 + held] = fmaf(dd, v_s[cl * SS_CC + held], sum) * silu(z);
     if (mine) store_state<SS_CC, KPL>(S, sp, ln, c0, N, V);
     // the request's last CTA to arrive norms the token
     __threadfence();
@@ -771,9 +776,14 @@ PRB_API int prb_ssm_finish(SSM_PARAMS, int gate_here, int out_dtype, cudaStream_
     const SsmArgs a = SSM_ARGS;
     if (n_tokens <= 0) return 0;
     if (!sizes_ok(a)) return PRB_E_SIZE;
-    const unsigned blocks = (unsigned)(((long)n_tokens * parts + FIN_WARPS - 1) / FIN_WARPS);
-    if (out_dtype == PRB_F32) ssm_finish_kernel<float><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here);
-    else if (out_dtype == PRB_BF16) ssm_finish_kernel<bf16><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here);
+    const int norm_blocks = (int)(((long)n_tokens * parts + FIN_WARPS - 1) / FIN_WARPS);
+    const int channels = heads * vdim + 2 * groups * dim;
+    const int save_blocks = taps > 1 ? n_requests * taps * ((channels + SAVE_CHANNELS - 1) / SAVE_CHANNELS) : 0;
+    const unsigned blocks = (unsigned)(norm_blocks + save_blocks);
+    if (out_dtype == PRB_F32)
+        ssm_finish_kernel<float><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here, norm_blocks);
+    else if (out_dtype == PRB_BF16)
+        ssm_finish_kernel<bf16><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here, norm_blocks);
     else return PRB_E_DTYPE;
     PRB_LAUNCH_CHECK();
     return 0;
@@ -802,13 +812,14 @@ PRB_API int prb_ssm_step(SSM_PARAMS, int* arrived, int out_dtype, cudaStream_t s
     const size_t smem = (size_t)(2 * lanes * kpl + cols + 2 * (cols + 2 * dim)) * sizeof(float);
     const dim3 grid(heads * g.splits, n_requests);
     cudaError_t e;
-#define SSTEP(OT)                                                                                          \
-    e = kpl == 4   ? prb_launch_dependent(ssm_step_kernel<4, OT>, grid, dim3(threads), smem, stream, g)     \
-        : kpl == 8 ? prb_launch_dependent(ssm_step_kernel<8, OT>, grid, dim3(threads), smem, stream, g)     \
-                   : prb_launch_dependent(ssm_step_kernel<16, OT>, grid, dim3(threads), smem, stream, g)
+#define SSTEP1(KP, TP, OT) prb_launch_dependent(ssm_step_kernel<KP, TP, OT>, grid, dim3(threads), smem, stream, g)
+#define SSTEP2(KP, OT) (taps <= 4 ? SSTEP1(KP, 4, OT) : SSTEP1(KP, SSM_TAPS, OT))
+#define SSTEP(OT) e = kpl == 4 ? SSTEP2(4, OT) : kpl == 8 ? SSTEP2(8, OT) : SSTEP2(16, OT)
     if (out_dtype == PRB_F32) { SSTEP(float); }
     else if (out_dtype == PRB_BF16) { SSTEP(bf16); }
     else return PRB_E_DTYPE;
 #undef SSTEP
+#undef SSTEP2
+#undef SSTEP1
     return e == cudaSuccess ? 0 : (int)e;
 }
