@@ -51,18 +51,17 @@ struct SegArgs {
     Finish fin;
 };
 
-// A token's row of a finish: a warp; src the head's sums (shared or global memory).
+// A token's row of a finish: a warp; src the head's sums, gp its gates (shared or global memory).
 template <typename O>
-__device__ __forceinline__ void finish_row(const Finish& f, const float* src, int t, int hd, int vdim,
-                                           int lane) {
+__device__ __forceinline__ void finish_row(const Finish& f, const float* src, const float* gp, int t, int hd,
+                                           int vdim, int lane) {
     float ss = 0.0f;
     for (int j = lane; j < vdim; j += 32) ss = fmaf(src[j], src[j], ss);
     ss = prb_warp_sum(ss);
     const float inv = f.out_scale / sqrtf(ss / (float)vdim + f.eps);
-    const float* gp = f.gate + (size_t)t * f.gate_ld + (size_t)hd * vdim;
     O* o = (O*)f.out + (size_t)t * f.out_ld + (size_t)hd * vdim;
     for (int j = lane; j < vdim; j += 32)
-        o[j] = prb_from_float<O>(src[j] * inv * f.norm_w[j] * silu(gp[j]));
+        o[j] = prb_from_float<O>(src[j] * inv * f.norm_w[j] * silu<O>(gp[j]));
 }
 
 // MODE 1: a segment's own sums from zero; 2: a segment from its start with outputs.  Scales of the
@@ -88,7 +87,8 @@ __global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
     const int L = a.lanes, dp = L * KPL, dim = a.dim, vdim = a.vdim, cols = a.cols;
     const int cw = PER_KEY ? dp : 4;
     const int stage = DS_TB * (2 * dp + cw + cols + 4);
-    float* o_s = sm + 2 * stage;                     // [DS_TB][vdim], with the finish inside
+    float* o_s = sm + 2 * stage;                     // [DS_TB][vdim], with the finish inside,
+    float* g_s = o_s + DS_TB * vdim;                 // and twice [DS_TB][vdim] gates
     const int ln = threadIdx.x % L, cl = min((int)threadIdx.x / L * DS_CC, cols - DS_CC);
     const int c0 = cg * cols + cl;                   // this thread's first value column
     const bool mine = (int)threadIdx.x / L * DS_CC < cols;       // (threads beyond work along, and store nothing)
@@ -106,6 +106,9 @@ __global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
     const bool vec = dim % 4 == 0 && vdim % 4 == 0 &&
                      (a.q_ld | a.k_ld | a.v_ld) % 4 == 0 && (!PER_KEY || a.c_ld % 4 == 0) &&
                      ((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (PER_KEY ? (uintptr_t)a.c : 0)) % 16 == 0;
+    const bool inside = MODE == 2 && a.fin.out != nullptr;
+    const float* gb = inside ? a.fin.gate + (size_t)hd * vdim : nullptr;
+    const bool gvec = inside && vdim % 4 == 0 && a.fin.gate_ld % 4 == 0 && ((uintptr_t)a.fin.gate) % 16 == 0;
     const float dd = !PER_KEY && a.direct ? a.direct[hd] : 0.0f;
     if (dp > dim) {                                  // keys beyond the head: zero in both stages
         for (int e = threadIdx.x; e < 2 * DS_TB * (dp - dim); e += blockDim.x) {
@@ -153,6 +156,20 @@ __global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
             for (int e = threadIdx.x; e < nb * vcols; e += blockDim.x) {
                 const int tok = e / vcols, i = e - tok * vcols;
                 v_s[tok * cols + i] = vb[(size_t)(tb + tok) * a.v_ld + i];
+            }
+        }
+        if (inside) {
+            float* to = g_s + into * DS_TB * vdim;
+            if (gvec) {
+                for (int e = threadIdx.x; e < nb * (vdim / 4); e += blockDim.x) {
+                    const int tok = e / (vdim / 4), i = (e - tok * (vdim / 4)) * 4;
+                    copy16(to + tok * vdim + i, gb + (size_t)(tb + tok) * a.fin.gate_ld + i);
+                }
+            } else {
+                for (int e = threadIdx.x; e < nb * vdim; e += blockDim.x) {
+                    const int tok = e / vdim, i = e - tok * vdim;
+                    to[e] = gb[(size_t)(tb + tok) * a.fin.gate_ld + i];
+                }
             }
         }
         if (!PER_KEY) {
@@ -216,9 +233,10 @@ __global__ void __launch_bounds__(ds_threads(KPL)) dscan_seg_kernel(SegArgs a) {
             }
         }
         __syncthreads();
-        if (MODE == 2 && a.fin.out) {
+        if (inside) {
             for (int tok = threadIdx.x >> 5; tok < nb; tok += blockDim.x >> 5)
-                finish_row<O>(a.fin, o_s + tok * vdim, tb + tok, hd, vdim, threadIdx.x & 31);
+                finish_row<O>(a.fin, o_s + tok * vdim, g_s + (turn * DS_TB + tok) * vdim, tb + tok, hd, vdim,
+                              threadIdx.x & 31);
         }
     }
     if (mine) {
@@ -294,7 +312,8 @@ __global__ void gla_finish_kernel(Finish f, const float* __restrict__ raw, long 
     if (unit >= (long)n_tokens * heads) return;
     const int t = (int)(unit / heads), hd = (int)(unit - (long)t * heads);
     if (seq_of_token[t] < 0) return;
-    finish_row<O>(f, raw + (size_t)t * raw_ld + (size_t)hd * vdim, t, hd, vdim, lane);
+    finish_row<O>(f, raw + (size_t)t * raw_ld + (size_t)hd * vdim, f.gate + (size_t)t * f.gate_ld + (size_t)hd * vdim,
+                  t, hd, vdim, lane);
 }
 
 __device__ __forceinline__ float decay_minus_one(float z, float inv_tau) {
@@ -355,6 +374,7 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     float* c_s = k_s + dp;
     float* v_s = c_s + dp;                           // [vdim rounded to GS_CC]
     float* o_s = v_s + (vdim + GS_CC - 1) / GS_CC * GS_CC;
+    float* g_s = o_s + (vdim + GS_CC - 1) / GS_CC * GS_CC;
     prb_grid_launch_dependents();
     const int hd = blockIdx.x, b = blockIdx.y;
     // (the step's description and the state of the step before lie behind launches that have
@@ -388,6 +408,8 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     }
     for (int i = threadIdx.x; i < (vdim + GS_CC - 1) / GS_CC * GS_CC; i += blockDim.x)
         v_s[i] = i < vdim ? row[a.v_col + hd * vdim + i] : 0.0f;
+    for (int i = threadIdx.x; i < vdim; i += blockDim.x)
+        g_s[i] = a.fin.gate[(size_t)t * a.fin.gate_ld + (size_t)hd * vdim + i];
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
         float z = 0.0f;
         if (i == (int)threadIdx.x) {
@@ -415,7 +437,7 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     }
     if (c0 < vdim) store_state<GS_CC, KPL>(S, sp, ln, c0, dim, vdim);
     __syncthreads();
-    if (threadIdx.x < 32) finish_row<O>(a.fin, o_s, t, hd, vdim, threadIdx.x);
+    if (threadIdx.x < 32) finish_row<O>(a.fin, o_s, g_s, t, hd, vdim, threadIdx.x);
 }
 
 int seg_cols(int dim, int vdim) {
@@ -427,7 +449,7 @@ int seg_cols(int dim, int vdim) {
 size_t seg_smem(int dim, int vdim, bool per_key, bool fin) {
     const int dp = lanes_of(dim) * keys_per_lane(dim);
     return (size_t)(2 * DS_TB * (2 * dp + (per_key ? dp : 4) + seg_cols(dim, vdim) + 4) +
-                    (fin ? DS_TB * vdim : 0)) * sizeof(float);
+                    (fin ? 3 * DS_TB * vdim : 0)) * sizeof(float);
 }
 }  // namespace
 
@@ -552,7 +574,7 @@ PRB_API int prb_gla_step(void* out, long out_ld, const float* proj, long ld, int
     const int lanes = lanes_of(dim), kpl = keys_per_lane(dim);
     const int vp = (vdim + GS_CC - 1) / GS_CC * GS_CC;
     const int threads = (vp / GS_CC * lanes + 31) / 32 * 32;
-    const size_t smem = (size_t)(3 * lanes * kpl + 2 * vp) * sizeof(float);
+    const size_t smem = (size_t)(3 * lanes * kpl + 3 * vp) * sizeof(float);
     GlaStepArgs a{proj, ld, q_col, k_col, v_col, lr_col, w2t, bias, inv_tau, q_scale, state, q_start,
                   state_slot, positions, n_tokens, n_requests, heads, dim, vdim, rank, lanes, n_slots,
                   status, Finish{out, out_ld, proj + g_col, ld, norm_w, eps, out_scale}};

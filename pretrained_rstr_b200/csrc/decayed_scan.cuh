@@ -134,7 +134,12 @@ __device__ __forceinline__ int held_column(int ln, int L) {
 }
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
+// T: the type the result is stored in; one that keeps 8 bits of mantissa is content with the
+// hardware's exponential.
+template <typename T>
+__device__ __forceinline__ float silu(float z) {
+    return __fdividef(z, 1.0f + (sizeof(T) == 2 ? __expf(-z) : expf(-z)));
+}
 
 // Portions in segments of DS_SEG tokens; segment z of the launch is segment s of request b
 // (requests' segments are numbered in request order).

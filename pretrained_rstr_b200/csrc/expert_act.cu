@@ -11,9 +11,22 @@
 #include "common.cuh"
 
 namespace {
-__device__ __forceinline__ float ea_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
-__device__ __forceinline__ float ea_gate(float g, int act) {     // 0: silu, 1: gelu (tanh form)
-    return act == 1 ? prb_activate(g, PRB_ACT_GELU_TANH) : g * ea_sigmoid(g);
+__device__ __forceinline__ float ea_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// 0: silu, 1: gelu (tanh form).  O: the type the result is stored in; one that keeps 8 bits of
+// mantissa is content with the hardware's exponential.
+template <typename O>
+__device__ __forceinline__ float ea_gate(float g, int act) {
+    if (act == 1) return prb_activate(g, PRB_ACT_GELU_TANH);
+    return __fdividef(g, 1.0f + (sizeof(O) == 2 ? __expf(-g) : expf(-g)));
+}
+
+// Floats in an order that unsigned integers keep (for the warp's integer reductions).
+__device__ __forceinline__ unsigned ordered(float v) {
+    const unsigned b = __float_as_uint(v);
+    return (b & 0x80000000u) ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ float from_ordered(unsigned k) {
+    return __uint_as_float((k & 0x80000000u) ? k & 0x7fffffffu : ~k);
 }
 
 struct ExpertArgs {
@@ -41,7 +54,7 @@ __device__ __forceinline__ void choose(const ExpertArgs& a, const float* row, fl
         sc[e] = z;
         top_z = fmaxf(top_z, z);
     }
-    top_z = prb_warp_max(top_z);
+    top_z = from_ordered(__reduce_max_sync(0xffffffffu, ordered(top_z)));
     float sum = 0.0f;
     for (int e = lane; e < all; e += 32) {
         const float p = expf(sc[e] - top_z);
@@ -59,17 +72,14 @@ __device__ __forceinline__ void choose(const ExpertArgs& a, const float* row, fl
     float chosen = 0.0f;
     for (int k = 0; k < a.top; ++k) {                // the largest left; ties: the lower index
         float best = -INFINITY;
-        int arg = all;
+        unsigned arg = all;
         for (int e = lane; e < all; e += 32) {
             const float v = pick[e];
             if (v > best) { best = v; arg = e; }
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, best, o);
-            const int w = __shfl_xor_sync(0xffffffffu, arg, o);
-            if (w < all && (arg >= all || v > best || (v == best && w < arg))) { best = v; arg = w; }
-        }
+        const unsigned key = ordered(best);
+        const unsigned top_key = __reduce_max_sync(0xffffffffu, key);
+        arg = __reduce_min_sync(0xffffffffu, key == top_key ? arg : (unsigned)all);
         if (arg >= all) break;                       // (a row of NaNs: padding, or a fault upstream)
         chosen += sc[arg];
         if (lane == 0) {
@@ -146,17 +156,17 @@ __global__ void __launch_bounds__(256) expert_act_row_kernel(ExpertArgs a) {
                     g = *reinterpret_cast<const float4*>(row + c.gate(a, i));
                     u = *reinterpret_cast<const float4*>(row + c.up(a, i));
                 }
-                v[0] = w * ea_gate(g.x, a.act) * u.x;
-                v[1] = w * ea_gate(g.y, a.act) * u.y;
-                v[2] = w * ea_gate(g.z, a.act) * u.z;
-                v[3] = w * ea_gate(g.w, a.act) * u.w;
+                v[0] = w * ea_gate<O>(g.x, a.act) * u.x;
+                v[1] = w * ea_gate<O>(g.y, a.act) * u.y;
+                v[2] = w * ea_gate<O>(g.z, a.act) * u.z;
+                v[3] = w * ea_gate<O>(g.w, a.act) * u.w;
             }
             prb_store4(o + i, v[0], v[1], v[2], v[3]);
         }
     } else {
         for (int i = c.lo + threadIdx.x; i < c.hi; i += blockDim.x) {
             const float w = i < c.n_exp ? wt[i / a.group] : own_s[1];
-            o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(row[c.gate(a, i)], a.act) * row[c.up(a, i)] : 0.0f);
+            o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate<O>(row[c.gate(a, i)], a.act) * row[c.up(a, i)] : 0.0f);
         }
     }
     if (a.identity == 0 || blockIdx.y != 0 || own_s[0] == 0.0f) return;
@@ -177,8 +187,8 @@ __global__ void __launch_bounds__(256) expert_act_row_kernel(ExpertArgs a) {
 
 // `n` columns of a row by a warp: w * f(gate) * up, or zeros without reading anything.
 template <typename O>
-__device__ __forceinline__ void act_run(O* o, const float* gate, const float* up, int n, float w, int act, bool vec,
-                                        int lane) {
+__device__ __forceinline__ void act_run(O* __restrict__ o, const float* __restrict__ gate,
+                                        const float* __restrict__ up, int n, float w, int act, bool vec, int lane) {
     if (vec) {
         if (w == 0.0f) {
             for (int i = lane * 4; i < n; i += 128) prb_store4(o + i, 0.0f, 0.0f, 0.0f, 0.0f);
@@ -188,13 +198,13 @@ __device__ __forceinline__ void act_run(O* o, const float* gate, const float* up
         for (int i = lane * 4; i < n; i += 128) {
             const float4 g = *reinterpret_cast<const float4*>(gate + i);
             const float4 u = *reinterpret_cast<const float4*>(up + i);
-            prb_store4(o + i, w * ea_gate(g.x, act) * u.x, w * ea_gate(g.y, act) * u.y, w * ea_gate(g.z, act) * u.z,
-                       w * ea_gate(g.w, act) * u.w);
+            prb_store4(o + i, w * ea_gate<O>(g.x, act) * u.x, w * ea_gate<O>(g.y, act) * u.y, w * ea_gate<O>(g.z, act) * u.z,
+                       w * ea_gate<O>(g.w, act) * u.w);
         }
         return;
     }
     for (int i = lane; i < n; i += 32)
-        o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate(gate[i], act) * up[i] : 0.0f);
+        o[i] = prb_from_float<O>(w != 0.0f ? w * ea_gate<O>(gate[i], act) * up[i] : 0.0f);
 }
 
 // Many rows: a warp a row and slice, no barrier.  A slice is every gridDim.y-th expert, the shared
@@ -230,10 +240,20 @@ __global__ void __launch_bounds__(EA_ROWS * 32) expert_act_kernel(ExpertArgs a) 
     float* x = a.x + (size_t)t * a.x_ld;
     if (a.h != nullptr) {                            // (every slice a share of the width)
         const O* h = (const O*)a.h + (size_t)t * a.h_ld;
-        const int per = (a.width + (int)gridDim.y - 1) / (int)gridDim.y;
+        const int per = ((a.width + (int)gridDim.y - 1) / (int)gridDim.y + 127) / 128 * 128;
         const int end = min(a.width, ((int)blockIdx.y + 1) * per);
-#pragma unroll 4
-        for (int i = blockIdx.y * per + lane; i < end; i += 32) x[i] = fmaf(identity, prb_to_float<O>(h[i]), x[i]);
+        for (int i0 = blockIdx.y * per + lane; i0 < end; i0 += 128) {
+            float xv[4], hv[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int i = i0 + 32 * k;
+                xv[k] = i < end ? x[i] : 0.0f;
+                hv[k] = i < end ? prb_to_float<O>(h[i]) : 0.0f;
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (i0 + 32 * k < end) x[i0 + 32 * k] = fmaf(identity, hv[k], xv[k]);
+        }
         return;
     }
     if (blockIdx.y != 0) return;

@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(256) ssm_prepare_kernel(SsmArgs a, X* __restri
         float s = bias;
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) s = fmaf(w[j], win[j], s);
-        store_as(xbc + (size_t)t * xbc_ld + ch, silu(s));
+        store_as(xbc + (size_t)t * xbc_ld + ch, silu<X>(s));
 #pragma unroll
         for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
     }
@@ -152,7 +152,7 @@ struct ChunkArgs {
     float* seg_decay;                                // [segments, heads]: product of decays minus one
 };
 
-// Running sums of log a over a segment's tokens, cum_s[64] (zero steps beyond nb), and dt_s.
+// Running sums of log2 a over a segment's tokens, cum_s[64] (zero steps beyond nb), and dt_s.
 __device__ __forceinline__ void running_sums(const ChunkArgs& c, int t0, int nb, int hd, float* cum_s,
                                              float* dt_s) {
     if (threadIdx.x < 32) {
@@ -167,8 +167,9 @@ __device__ __forceinline__ void running_sums(const ChunkArgs& c, int t0, int nb,
             const float up = __shfl_up_sync(0xffffffffu, sum, o);
             if (lane >= o) sum += up;
         }
-        cum_s[i1] = sum;
-        cum_s[i0] = sum - a1;
+        const float log2e = 1.4426950408889634f;
+        cum_s[i1] = sum * log2e;
+        cum_s[i0] = (sum - a1) * log2e;
     }
 }
 
@@ -214,10 +215,10 @@ __global__ void __launch_bounds__(128) ssm_own_kernel(ChunkArgs c) {
     copy_wait<0>();
     __syncthreads();
     const float end = cum_s[DS_SEG - 1];
-    if (threadIdx.x == 0) c.seg_decay[(size_t)blockIdx.y * c.s.heads + hd] = expm1f(end);
+    if (threadIdx.x == 0) c.seg_decay[(size_t)blockIdx.y * c.s.heads + hd] = expm1f(end * 0.6931471805599453f);
     for (int e = threadIdx.x; e < DS_SEG * (V / 2); e += blockDim.x) {
         const int r = e / (V / 2), i = (e - r * (V / 2)) * 2;
-        const float w = r < nb ? expf(end - cum_s[r]) * dt_s[r] : 0.0f;
+        const float w = r < nb ? exp2f(end - cum_s[r]) * dt_s[r] : 0.0f;
         const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(xh + r * vp + i);
         const float x0 = w * __bfloat162float(x.x), x1 = w * __bfloat162float(x.y);
         *reinterpret_cast<uint32_t*>(xh + r * vp + i) = pack2(x0, x1);
@@ -414,7 +415,7 @@ __global__ void __launch_bounds__(256) ssm_out_kernel(ChunkArgs c) {
     }
     const float cum0 = cum_s[i0], cum1 = cum_s[i1];
     if (started) {
-        const float e0 = expf(cum0), e1 = expf(cum1);
+        const float e0 = exp2f(cum0), e1 = exp2f(cum1);
 #pragma unroll
         for (int i = 0; i < VT; ++i) {
             acc[i][0] *= e0; acc[i][1] *= e0;
@@ -430,10 +431,10 @@ __global__ void __launch_bounds__(256) ssm_out_kernel(ChunkArgs c) {
         for (int q = 0; q < 2; ++q) {
             const int j0 = p * 16 + q * 8 + (lane & 3) * 2, j1 = j0 + 1;
             const float* gq = gm[2 * p + q];
-            w[q][0] = j0 <= i0 ? gq[0] * expf(cum0 - cum_s[j0]) * dt_s[j0] : 0.0f;
-            w[q][1] = j1 <= i0 ? gq[1] * expf(cum0 - cum_s[j1]) * dt_s[j1] : 0.0f;
-            w[q][2] = j0 <= i1 ? gq[2] * expf(cum1 - cum_s[j0]) * dt_s[j0] : 0.0f;
-            w[q][3] = j1 <= i1 ? gq[3] * expf(cum1 - cum_s[j1]) * dt_s[j1] : 0.0f;
+            w[q][0] = j0 <= i0 ? gq[0] * exp2f(cum0 - cum_s[j0]) * dt_s[j0] : 0.0f;
+            w[q][1] = j1 <= i0 ? gq[1] * exp2f(cum0 - cum_s[j1]) * dt_s[j1] : 0.0f;
+            w[q][2] = j0 <= i1 ? gq[2] * exp2f(cum1 - cum_s[j0]) * dt_s[j0] : 0.0f;
+            w[q][3] = j1 <= i1 ? gq[3] * exp2f(cum1 - cum_s[j1]) * dt_s[j1] : 0.0f;
         }
         mh[0] = pack2(w[0][0], w[0][1]); ml[0] = pack2(low_part(w[0][0]), low_part(w[0][1]));
         mh[1] = pack2(w[0][2], w[0][3]); ml[1] = pack2(low_part(w[0][2]), low_part(w[0][3]));
@@ -464,7 +465,7 @@ __global__ void __launch_bounds__(256) ssm_out_kernel(ChunkArgs c) {
                     const float y0 = fmaf(dd, __bfloat162float(x.x), acc[v][2 * half]);
                     const float y1 = fmaf(dd, __bfloat162float(x.y), acc[v][2 * half + 1]);
                     *reinterpret_cast<float2*>(c.s.raw + (size_t)(t0 + i) * c.s.raw_ld + hd * V + col) =
-                        make_float2(y0 * silu(z[v][half].x), y1 * silu(z[v][half].y));
+                        make_float2(y0 * silu<bf16>(z[v][half].x), y1 * silu<bf16>(z[v][half].y));
                 }
             }
         }
@@ -504,12 +505,12 @@ __device__ __forceinline__ void norm_part_warp(const SsmArgs& a, const float* ro
     }
     float ss = 0.0f;
     for (int i = lane; i < part; i += 32) {
-        const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
+        const float y = z ? row[lo + i] * silu<O>(z[lo + i]) : row[lo + i];
         ss = fmaf(y, y, ss);
     }
     const float inv = a.out_scale / sqrtf(prb_warp_sum(ss) / (float)part + a.eps);
     for (int i = lane; i < part; i += 32) {
-        const float y = z ? row[lo + i] * silu(z[lo + i]) : row[lo + i];
+        const float y = z ? row[lo + i] * silu<O>(z[lo + i]) : row[lo + i];
         o[lo + i] = prb_from_float<O>(y * inv * a.norm_w[lo + i]);
     }
 }
@@ -650,7 +651,7 @@ __global__ void __launch_bounds__(512, KPL == 4 ? 2 : 1) ssm_step_kernel(StepArg
     const float z = writes ? row[a.z_col + hd * V + c0 + held] : 0.0f;
     for (int i = threadIdx.x; i < todo; i += blockDim.x) {   // (the same thread as above)
         const float in = row[a.x_col + channel_of(i)];
-        const float u = silu(fmaf(h_s[todo + i], in, h_s[i]));
+        const float u = silu<O>(fmaf(h_s[todo + i], in, h_s[i]));
         // (a channel is saved by the one CTA that owns it; B and C by the group's first)
         if (a.taps > 1 && (i < live || (cg == 0 && hd % (a.heads / a.groups) == 0)))
             a.conv_state[((size_t)slot * a.taps + pos % a.taps) * channels + channel_of(i)] = in;
@@ -668,7 +669,7 @@ __global__ void __launch_bounds__(512, KPL == 4 ? 2 : 1) ssm_step_kernel(StepArg
     advance<SS_CC, KPL, false, true>(S, k_s + ln * KPL, &c1, q_s + ln * KPL, v, part);
     const float sum = close_columns<SS_CC>(part, ln, L);
     if (writes)
-        a.raw[(size_t)t * a.raw_ld + hd * V + c0 + held] = fmaf(dd, v_s[cl * SS_CC + held], sum) * silu(z);
+        a.raw[(size_t)t * a.raw_ld + hd * V + c0 + held] = fmaf(dd, v_s[cl * SS_CC + held], sum) * silu<O>(z);
     if (mine) store_state<SS_CC, KPL>(S, sp, ln, c0, N, V);
     // the request's last CTA to arrive norms the token
     __threadfence();

@@ -241,6 +241,11 @@ class StepContext:
         self.feedback = False               # token ids below zero name tokens chosen last
         self.used_words: Optional[int] = None      # words of the step's buffer that go to the device
 
+    def side(self, index: int) -> "SideStream":
+        """The ``index``-th stream beside the step's main one (see :class:`SideStream`).  Scratch memory
+        that both branches fill has to exist before they part."""
+        return SideStream(self.runtime.device, index)
+
     @property
     def dtype(self) -> torch.dtype:
         return self.runtime.dtype
@@ -267,6 +272,35 @@ class StepContext:
         """Scratch that is zero when first handed out; whoever uses it leaves it zero
         (counters that their kernel resets)."""
         return self._scratch.get(key, shape, dtype, zero=True)
+
+
+_SIDE_STREAMS: Dict[Tuple[str, int], "torch.cuda.Stream"] = {}
+
+
+class SideStream:
+    """Work beside a step's main stream: ``with side:`` launches inside go to a stream that has waited
+    for everything launched before the ``with``; :meth:`join` makes the current stream wait for
+    them.  A step that is recorded as a CUDA graph records the two branches.  The first kernel of a
+    branch, and the first behind a join, must not be placed early (``ops.plain_launch``)."""
+
+    def __init__(self, device: torch.device, index: int):
+        key = (str(device), index)
+        if key not in _SIDE_STREAMS:
+            _SIDE_STREAMS[key] = torch.cuda.Stream(device=device)
+        self.stream = _SIDE_STREAMS[key]
+        self._inside = None
+
+    def __enter__(self):
+        self.stream.wait_stream(torch.cuda.current_stream())
+        self._inside = torch.cuda.stream(self.stream)
+        self._inside.__enter__()
+        return self
+
+    def __exit__(self, *exc):
+        return self._inside.__exit__(*exc)
+
+    def join(self) -> None:
+        torch.cuda.current_stream().wait_stream(self.stream)
 
 
 class ScratchPool:

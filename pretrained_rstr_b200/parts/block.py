@@ -8,6 +8,7 @@ from typing import Dict
 import torch
 
 from ..csrc import ops
+from ..settings import SETTINGS
 from .interfaces import Block, FeedForward, LayerCache, Mixer, Norm
 from .linear import LazyNorm, Linear
 from .registry import register_part
@@ -172,6 +173,18 @@ class ParallelBlock(Block):
         norm = self.norms["shared"]
         if self.result is not None or not self.has_ff:
             h_in = PreNormBlock._normed(ctx, self.mixer, norm, x, h)
+            if self.has_ff and SETTINGS.side_streams and getattr(self.feed_forward, "worth_a_branch", False):
+                # the feed-forward's activations beside the mixer: both start from the first product
+                self.mixer.products()[0].run_ahead(ctx, h_in)
+                self.result.buffer(ctx, x.shape[0])        # (there before the branches part)
+                side = ctx.side(1)
+                with side, ops.plain_launch():
+                    self.feed_forward.forward(ctx, h_in, x)
+                self.mixer.forward(ctx, h_in, x, cache)
+                side.join()
+                with ops.plain_launch():
+                    self.result.close(ctx, x)
+                return
             self.mixer.forward(ctx, h_in, x, cache)
             if self.has_ff:
                 self.feed_forward.forward(ctx, h_in, x)

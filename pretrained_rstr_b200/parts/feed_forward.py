@@ -206,6 +206,11 @@ class GatedMoE(FeedForward):
     def fused_rows(self, name: str):
         return self.input.view(self._proj, name)
 
+    @property
+    def worth_a_branch(self) -> bool:
+        """The activations take long enough that running them beside a mixer pays for the branch."""
+        return self.one_launch
+
     def _forward_one_launch(self, ctx, h, x, accumulate: bool) -> None:
         proj = self._proj = self.input.run(ctx, h)
         at = lambda name: self.input.cols[name][0]

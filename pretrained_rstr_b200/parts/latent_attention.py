@@ -70,6 +70,7 @@ class FusedInput:
         self.host: Optional["FusedInput"] = None            # whose product this one's rows ride in
         self._guests: List[Tuple[str, "FusedInput"]] = []   # (prefix of its segments' names, guest)
         self._result: Optional[torch.Tensor] = None         # of the step that runs
+        self._ahead = False                                 # the next run() has been done already
 
     def absorb(self, other: "FusedInput") -> None:
         """Take over ``other``'s segments (and what is added to it from now on)."""
@@ -114,9 +115,27 @@ class FusedInput:
                                    if name.startswith(prefix)})
         return self._linear
 
+    @property
+    def ahead(self) -> bool:
+        return self._ahead
+
+    @property
+    def result(self) -> torch.Tensor:
+        """What the product of this step left."""
+        return self._result if self.host is None else self.host._result
+
+    def run_ahead(self, ctx, h) -> None:
+        """Run the product now; the next :meth:`run` hands out its result (whoever lets several parts
+        start from it side by side does that)."""
+        self.run(ctx, h)
+        self._ahead = True
+
     def run(self, ctx, h) -> torch.Tensor:
         if self.host is not None:
             return self.host._result
+        if self._ahead:
+            self._ahead = False
+            return self._result
         lin = self.linear()
         t = h.shape[0]
         out = ctx.scratch(self.key, (ctx.token_capacity, lin.n_out), torch.float32)[:t]

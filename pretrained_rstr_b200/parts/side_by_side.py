@@ -13,6 +13,8 @@ it).  ``share_product`` False keeps the products apart.  Children that end in a
 brings both results to the stream."""
 from __future__ import annotations
 
+from ..csrc import ops
+from ..settings import SETTINGS
 from .interfaces import LayerCache, Mixer
 from .registry import build_part, register_part
 
@@ -72,10 +74,26 @@ class SideBySide(Mixer):
 
     def forward(self, ctx, h, x, cache: LayerCache, accumulate: bool = True) -> None:
         first, second = self.children
+        if self.products() is None or not SETTINGS.side_streams:
+            first.forward(ctx, h, x, cache, accumulate=accumulate)
+            second.forward(ctx, h, x, cache, accumulate=True)
+            if self.result is not None and self.result.closer is self:
+                self.result.close(ctx, x, accumulate)
+            return
+        # both start from the same product and meet in the same last one: side by side in between
+        # (on the GPU too: neither fills it)
+        product, _result = self.products()
+        if not product.ahead:
+            product.run_ahead(ctx, h)
+        self.result.buffer(ctx, x.shape[0])        # (there before the branches part)
+        side = ctx.side(0)
+        with side, ops.plain_launch():
+            second.forward(ctx, h, x, cache, accumulate=True)
         first.forward(ctx, h, x, cache, accumulate=accumulate)
-        second.forward(ctx, h, x, cache, accumulate=True)
-        if self.result is not None and self.result.closer is self:
-            self.result.close(ctx, x, accumulate)
+        side.join()
+        if self.result.closer is self:
+            with ops.plain_launch():
+                self.result.close(ctx, x, accumulate)
 
 
 register_part("mixer", "side_by_side", lambda p, store, rt: SideBySide(p, store, rt))

@@ -91,7 +91,7 @@ class StateSpace(Mixer):
     def fused_product(self):
         """(the fused product's 32-bit result of this step, first column by segment name): for a
         mixer beside this one whose projections ride in the product."""
-        return self._proj, self.input.cols
+        return self.input.result, self.input.cols
 
     def state_specs(self):
         specs = [StateSpec("ssm_state", (self.heads, self.vdim, self.state_dim), torch.float32)]

@@ -8,6 +8,7 @@ Python side (``SETTINGS``):
 
 ``PRB200_GRAPHS=0``        small steps are launched kernel by kernel instead of as CUDA graphs
 ``PRB200_PDL=0``           no programmatic dependent launch between the kernels of a step
+``PRB200_SIDE_STREAMS=0``  parts that read the same product run one after the other instead of side by side
 ``PRB200_ATTN_TC=0``       prompt attention on ``mma.sync`` even where the tcgen05 kernel applies
 ``PRB200_PREFILL_PART=N``  key blocks per part of the tcgen05 prompt attention (-1: the kernel's rule)
 ``PRB200_DECODE_CTAS=N``   CTAs a decode attention launch aims for (0: about five per SM)
@@ -44,6 +45,7 @@ def _int(name: str, default: int) -> int:
 class Settings:
     graphs: bool = True
     pdl: bool = True
+    side_streams: bool = True
     attention_tcgen05: bool = True
     prefill_part: int = -1
     decode_ctas: int = 0
@@ -53,6 +55,7 @@ class Settings:
     @classmethod
     def from_environment(cls) -> "Settings":
         return cls(graphs=_flag("PRB200_GRAPHS", True), pdl=_flag("PRB200_PDL", True),
+                   side_streams=_flag("PRB200_SIDE_STREAMS", True),
                    attention_tcgen05=_flag("PRB200_ATTN_TC", True),
                    prefill_part=_int("PRB200_PREFILL_PART", -1),
                    decode_ctas=_int("PRB200_DECODE_CTAS", 0),
