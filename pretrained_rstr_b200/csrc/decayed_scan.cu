@@ -440,15 +440,17 @@ __global__ void __launch_bounds__(KPL == 4 ? 1024 : 512) gla_step_kernel(GlaStep
     if (threadIdx.x < 32) finish_row<O>(a.fin, o_s, g_s, t, hd, vdim, threadIdx.x);
 }
 
-int seg_cols(int dim, int vdim) {
+// Value columns a CTA of a pass takes (the pass with outputs likes whole heads, for the finish; the
+// other several CTAs an SM).
+int seg_cols(int dim, int vdim, int mode = 2) {
     const int lanes = lanes_of(dim);
-    int cols = ds_threads(keys_per_lane(dim)) / lanes * DS_CC;
+    int cols = min(ds_threads(keys_per_lane(dim)), mode == 1 ? 256 : 1024) / lanes * DS_CC;
     if (cols > vdim) cols = (vdim + DS_CC - 1) / DS_CC * DS_CC;
     return cols;
 }
-size_t seg_smem(int dim, int vdim, bool per_key, bool fin) {
+size_t seg_smem(int dim, int vdim, int cols, bool per_key, bool fin) {
     const int dp = lanes_of(dim) * keys_per_lane(dim);
-    return (size_t)(2 * DS_TB * (2 * dp + (per_key ? dp : 4) + seg_cols(dim, vdim) + 4) +
+    return (size_t)(2 * DS_TB * (2 * dp + (per_key ? dp : 4) + cols + 4) +
                     (fin ? 3 * DS_TB * vdim : 0)) * sizeof(float);
 }
 }  // namespace
@@ -458,8 +460,9 @@ PRB_API int prb_dscan_max_segments(int t_cap, int b_cap) { return t_cap / DS_SEG
 // 0: not at all; 1: raw sums; 3: also with the finish inside pass 2 (a CTA holds a whole head).
 PRB_API int prb_dscan_supports(int dim, int vdim) {
     if (lanes_of(dim) == 0 || vdim <= 0 || vdim > 4096) return 0;
-    if (seg_smem(dim, vdim, true, false) > 200 * 1024) return 0;
-    return seg_cols(dim, vdim) >= vdim && seg_smem(dim, vdim, true, true) <= 200 * 1024 ? 3 : 1;
+    const int cols = seg_cols(dim, vdim);
+    if (seg_smem(dim, vdim, cols, true, false) > 200 * 1024) return 0;
+    return cols >= vdim && seg_smem(dim, vdim, cols, true, true) <= 200 * 1024 ? 3 : 1;
 }
 
 // Three launches.  Workspaces: seg_own, seg_start [segments, heads, vdim, dim], seg_decay
@@ -487,11 +490,12 @@ PRB_API int prb_dscan_segments(float* raw, long raw_ld, const float* q, long q_l
               state, q_start, state_slot, positions, n_tokens, n_requests, heads, dim, vdim, lanes,
               cols, n_slots, seg_own, seg_start, seg_decay, status,
               Finish{out, out_ld, gate, gate_ld, norm_w, eps, out_scale}};
-    const int threads = (cols / DS_CC * lanes + 31) / 32 * 32;
-    const size_t smem = seg_smem(dim, vdim, per_key != 0, out != nullptr);
-    const dim3 grid(heads, need, (vdim + cols - 1) / cols);
 #define SEGRUN(KP, PK, MD, OT)                                                                     \
     do {                                                                                           \
+        a.cols = MD == 1 ? seg_cols(dim, vdim, 1) : cols;                                          \
+        const int threads = (a.cols / DS_CC * lanes + 31) / 32 * 32;                               \
+        const size_t smem = seg_smem(dim, vdim, a.cols, PK, MD == 2 && out != nullptr);            \
+        const dim3 grid(heads, need, (vdim + a.cols - 1) / a.cols);                                \
         if (smem > 40 * 1024)                                                                      \
             cudaFuncSetAttribute(dscan_seg_kernel<KP, PK, MD, OT>,                                 \
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);          \

@@ -550,11 +550,40 @@ __device__ __forceinline__ void norm_row_cta(const SsmArgs& a, const float* row,
     }
 }
 
-// Warps (token, part); behind them CTAs that save inputs: (request, one of its portion's last `taps`
-// tokens, 512 channels).
-constexpr int FIN_WARPS = 4, SAVE_CHANNELS = 512;
+// A long part of a token's row by a CTA of FIN_WIDE threads.
+constexpr int FIN_WIDE = 256;
 template <typename O>
-__global__ void __launch_bounds__(FIN_WARPS * 32) ssm_finish_kernel(SsmArgs a, int gate_here, int norm_blocks) {
+__device__ __forceinline__ void norm_part_cta(const SsmArgs& a, const float* row, const float* z, O* o, int lo,
+                                              int part, float* scratch) {
+    constexpr int KEPT = 16;
+    float y[KEPT], ss = 0.0f;
+    auto value = [&](int i) { return z ? row[lo + i] * silu<O>(z[lo + i]) : row[lo + i]; };
+#pragma unroll
+    for (int k = 0; k < KEPT; ++k) {
+        const int i = threadIdx.x + k * FIN_WIDE;
+        y[k] = i < part ? value(i) : 0.0f;
+    }
+#pragma unroll
+    for (int k = 0; k < KEPT; ++k) ss = fmaf(y[k], y[k], ss);
+    for (int i = threadIdx.x + KEPT * FIN_WIDE; i < part; i += FIN_WIDE) ss = fmaf(value(i), value(i), ss);
+    ss = prb_block_sum(ss, scratch);
+    const float inv = a.out_scale / sqrtf(ss / (float)part + a.eps);
+#pragma unroll
+    for (int k = 0; k < KEPT; ++k) {
+        const int i = threadIdx.x + k * FIN_WIDE;
+        if (i < part) o[lo + i] = prb_from_float<O>(y[k] * inv * a.norm_w[lo + i]);
+    }
+    for (int i = threadIdx.x + KEPT * FIN_WIDE; i < part; i += FIN_WIDE)
+        o[lo + i] = prb_from_float<O>(value(i) * inv * a.norm_w[lo + i]);
+}
+
+// Warps (token, part), or CTAs where a part is longer than a warp keeps; behind them CTAs that save
+// inputs: (request, one of its portion's last `taps` tokens, 512 channels).
+constexpr int FIN_WARPS = 4, SAVE_CHANNELS = 512;
+template <typename O, bool WIDE>
+__global__ void __launch_bounds__(WIDE ? FIN_WIDE : FIN_WARPS * 32)
+ssm_finish_kernel(SsmArgs a, int gate_here, int norm_blocks) {
+    __shared__ float scratch[32];
     prb_grid_launch_dependents();
     if ((int)blockIdx.x >= norm_blocks) {
         const int channels = a.heads * a.vdim + 2 * a.groups * a.dim;
@@ -567,21 +596,21 @@ __global__ void __launch_bounds__(FIN_WARPS * 32) ssm_finish_kernel(SsmArgs a, i
         if (t < a.q_start[b] || t < 0 || t >= a.n_tokens || slot < 0 || slot >= a.n_slots) return;
         float* st = a.conv_state + ((size_t)slot * a.taps + a.positions[t] % a.taps) * channels;
         const float* from = a.proj + (size_t)t * a.ld + a.x_col;
-#pragma unroll
-        for (int k = 0; k < SAVE_CHANNELS / (FIN_WARPS * 32); ++k) {
-            const int ch = piece * SAVE_CHANNELS + k * FIN_WARPS * 32 + (int)threadIdx.x;
-            if (ch < channels) st[ch] = from[ch];
-        }
+        const int end = min(channels, (piece + 1) * SAVE_CHANNELS);
+#pragma unroll 4
+        for (int ch = piece * SAVE_CHANNELS + (int)threadIdx.x; ch < end; ch += blockDim.x) st[ch] = from[ch];
         return;
     }
-    const int lane = threadIdx.x & 31;
-    const long unit = (long)blockIdx.x * FIN_WARPS + (threadIdx.x >> 5);
+    const long unit = WIDE ? blockIdx.x : (long)blockIdx.x * FIN_WARPS + (threadIdx.x >> 5);
     if (unit >= (long)a.n_tokens * a.parts) return;
     const int t = (int)(unit / a.parts), p = (int)(unit - (long)t * a.parts);
     if (a.seq[t] < 0) return;
     const int part = a.heads * a.vdim / a.parts;
-    norm_part_warp<O>(a, a.raw + (size_t)t * a.raw_ld, gate_here ? a.proj + (size_t)t * a.ld + a.z_col : nullptr,
-                      (O*)a.out + (size_t)t * a.out_ld, p * part, part, lane);
+    const float* row = a.raw + (size_t)t * a.raw_ld;
+    const float* z = gate_here ? a.proj + (size_t)t * a.ld + a.z_col : nullptr;
+    O* o = (O*)a.out + (size_t)t * a.out_ld;
+    if (WIDE) norm_part_cta<O>(a, row, z, o, p * part, part, scratch);
+    else norm_part_warp<O>(a, row, z, o, p * part, part, threadIdx.x & 31);
 }
 
 // ------------------------------------------------------------------- single tokens
@@ -777,15 +806,21 @@ PRB_API int prb_ssm_finish(SSM_PARAMS, int gate_here, int out_dtype, cudaStream_
     const SsmArgs a = SSM_ARGS;
     if (n_tokens <= 0) return 0;
     if (!sizes_ok(a)) return PRB_E_SIZE;
-    const int norm_blocks = (int)(((long)n_tokens * parts + FIN_WARPS - 1) / FIN_WARPS);
+    const bool wide = heads * vdim / parts > FIN_PIECES * 128;
+    const long units = (long)n_tokens * parts;
+    const int norm_blocks = (int)(wide ? units : (units + FIN_WARPS - 1) / FIN_WARPS);
     const int channels = heads * vdim + 2 * groups * dim;
     const int save_blocks = taps > 1 ? n_requests * taps * ((channels + SAVE_CHANNELS - 1) / SAVE_CHANNELS) : 0;
     const unsigned blocks = (unsigned)(norm_blocks + save_blocks);
-    if (out_dtype == PRB_F32)
-        ssm_finish_kernel<float><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here, norm_blocks);
-    else if (out_dtype == PRB_BF16)
-        ssm_finish_kernel<bf16><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here, norm_blocks);
+#define FINISH(OT)                                                                                              \
+    do {                                                                                                        \
+        if (wide) ssm_finish_kernel<OT, true><<<blocks, FIN_WIDE, 0, stream>>>(a, gate_here, norm_blocks);       \
+        else ssm_finish_kernel<OT, false><<<blocks, FIN_WARPS * 32, 0, stream>>>(a, gate_here, norm_blocks);     \
+    } while (0)
+    if (out_dtype == PRB_F32) FINISH(float);
+    else if (out_dtype == PRB_BF16) FINISH(bf16);
     else return PRB_E_DTYPE;
+#undef FINISH
     PRB_LAUNCH_CHECK();
     return 0;
 }

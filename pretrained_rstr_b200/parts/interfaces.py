@@ -68,6 +68,11 @@ class StreamJoin:
 
 
 class Mixer:
+    """``products()`` (optional, a feed-forward's too): (the fused first product, the product that
+    ends the part), for arrangements whose branches share them (``FusedInput.absorb``,
+    ``ResultProduct.absorb``); the part then hands its columns over and leaves running the last product
+    to whoever joined them."""
+
     def kv_spec(self) -> Optional[KVSpec]:
         return None
 

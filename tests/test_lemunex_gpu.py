@@ -394,7 +394,7 @@ class StateSpaceCase:
 
 @pytest.mark.parametrize("heads,vdim,dim,groups,taps,parts", [
     (4, 16, 32, 2, 4, 1), (6, 32, 16, 1, 3, 3), (2, 64, 128, 1, 4, 2), (2, 128, 64, 2, 2, 1), (3, 20, 10, 3, 1, 1),
-    (5, 8, 136, 1, 7, 5), (8, 16, 48, 4, 8, 8), (1, 7, 3, 1, 2, 1)])
+    (5, 8, 136, 1, 7, 5), (8, 16, 48, 4, 8, 8), (1, 7, 3, 1, 2, 1), (36, 64, 16, 2, 4, 1), (20, 128, 8, 4, 2, 1)])
 def test_state_space_mixer(heads, vdim, dim, groups, taps, parts):
     """Whole, in portions down to one token, and token by token in one launch each, beside another
     request; the three ways agree with the plain mixer, and states left by one are carried on by
